@@ -11,8 +11,8 @@ equal shape, which gives ``[page][run][k|v][kv_head][slot][head_dim]``.
 
 Pages are taken before a step for the tokens the step brings
 (:meth:`KVCacheManager.reserve`), and given back when the request ends
-(:meth:`free_request`) or, in a group with a window, once no later token can
-see them (:meth:`advance`).  The manager is host-side bookkeeping and has no
+(:meth:`free_request`) or, in a group with a window or with chunks, once no
+later token can see them (:meth:`advance`).  The manager is host-side bookkeeping and has no
 GPU dependency; :class:`KVCacheStorage` owns the device tensors.
 
 The reference sizes a dense buffer ``[max_batch][layers][2][max_seq][kv_dim]``
@@ -76,8 +76,11 @@ class KVCacheManager:
         return (seq.serial, seq.version)
 
     def _first_needed_block(self, group: int, length: int) -> int:
-        """Blocks below this one lie wholly behind the window of every token at
-        position >= length."""
+        """Blocks below this one lie wholly behind the window, or ahead of the
+        chunk, of every token at position >= length."""
+        chunk = getattr(self.needs[group], "chunk", None)
+        if chunk:
+            return (length - length % chunk) // self.page_size
         w = self.needs[group].window
         if not w:
             return 0
@@ -129,7 +132,8 @@ class KVCacheManager:
 
     def advance(self, rid: Hashable, n_new: int) -> None:
         """The step wrote ``n_new`` tokens: move the length on and give back the
-        pages that a window has passed (never those of kept first tokens)."""
+        pages that a window has passed (never those of kept first tokens) or
+        whose chunk is over."""
         seq = self._seqs[rid]
         if seq.length + n_new > seq.reserved:
             raise RuntimeError(f"request {rid!r}: advance beyond the reserved pages")

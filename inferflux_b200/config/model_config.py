@@ -815,3 +815,165 @@ class MalazenConfig(ModelConfig):
         if self.loop_times:
             out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
         return out
+
+
+@dataclass(frozen=True)
+class ZetivikLayer:
+    """One layer of a Zetivik model as config.json gives it: the mixer's sizes and constants (checked, defaults
+    filled in) and its feed-forward (``None`` = none; ``kind`` ``dense`` with ``ff`` and ``limit``)."""
+
+    type: str = ""
+    mixer: Dict[str, Any] = field(default_factory=dict)
+    mlp: Optional[Dict[str, Any]] = None
+
+
+@dataclass(frozen=True)
+class ZetivikConfig(ModelConfig):
+    """``Zetivik``: a decoder whose layers are listed one by one in config.json (``layers``: ``type``, the mixer's
+    sizes under ``mixer``, the feed-forward under ``mlp`` or null), pre-norm with RMS norms whose weights are stored
+    around zero.  The mixer ``parallel`` is a weighted sum of a pair of mixers on one input: ``left`` grouped-query
+    attention inside chunks of ``mask.size`` positions (biases, every query and key head normed, rotate-half positions,
+    one output gate a head) and ``right`` the gated delta rule (short convolutions, unit queries and keys, one decay
+    and one rate a head).  The mixer ``lightning`` is linear attention with a fixed decay per head.  Feed-forwards are
+    gated with clamped inputs.  A stretch of layers (``loop``: ``start``, ``stop``, ``times``) may run several times in a
+    row on the same weights; a stored vector joins the stream ahead of every pass, and the embedding's output ahead of
+    every pass but the first.  The output head is the embedding table, its logits optionally capped
+    (``logit_softcap``)."""
+
+    width: int = 0
+    vocab: int = 0
+    norm_eps: float = 1e-6
+    logit_softcap: Optional[float] = None
+    layers: List[ZetivikLayer] = field(default_factory=list)
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0              # 0 = the model has no loop
+
+    ARCHITECTURE = "Zetivik"
+    MODEL_TYPE = "zetivik"
+    MIXERS = ("lightning", "parallel")
+
+    @staticmethod
+    def _heads(m: Dict[str, Any], where: str, dim_max: int = 256) -> Dict[str, Any]:
+        """heads, kv_heads (default: as many), dim, vdim (default: dim)."""
+        heads, dim = _require_int(m, "heads"), _require_int(m, "dim")
+        out = {"heads": heads, "kv_heads": _require_int(m, "kv_heads") if m.get("kv_heads") is not None else heads,
+               "dim": dim, "vdim": _require_int(m, "vdim") if m.get("vdim") is not None else dim}
+        if heads % out["kv_heads"]:
+            raise ConfigError(f"{where}: heads {heads} is not a multiple of kv_heads {out['kv_heads']}")
+        if dim > dim_max:
+            raise ConfigError(f"{where}: dim {dim} is not supported (at most {dim_max})")
+        return out
+
+    @classmethod
+    def _left(cls, m: Dict[str, Any], where: str) -> Dict[str, Any]:
+        out = cls._heads(m, where)
+        if out["vdim"] > 256:
+            raise ConfigError(f"{where}: vdim {out['vdim']} is not supported (at most 256)")
+        out["scale"] = _require_number(m, "scale", where) if m.get("scale") is not None else float(out["dim"]) ** -0.5
+        mask = _sub(m, "mask", where, optional=True)
+        out["chunk"] = _require_int(mask, "size") if mask is not None and mask.get("size") is not None else None
+        rot = _sub(m, "rot", where, optional=True)
+        out["rot"] = {"dims": 0, "base": 10000.0}
+        if rot is not None:
+            out["rot"] = {"dims": _require_int(rot, "dims", 0), "base": _require_number(rot, "base", where + " rot")}
+            if out["rot"]["dims"] % 2 or out["rot"]["dims"] > out["dim"]:
+                raise ConfigError(f"{where}: rot.dims {out['rot']['dims']} must be even and at most dim {out['dim']}")
+            if out["rot"]["base"] <= 0.0:
+                raise ConfigError(f"{where}: rot.base must be positive")
+        return out
+
+    @classmethod
+    def _right(cls, m: Dict[str, Any], where: str) -> Dict[str, Any]:
+        out = cls._heads(m, where)
+        out["conv"] = _require_int(m, "conv")
+        if out["conv"] > 16:
+            raise ConfigError(f"{where}: a convolution of {out['conv']} taps is not supported (at most 16)")
+        return out
+
+    @classmethod
+    def _lightning(cls, m: Dict[str, Any], where: str) -> Dict[str, Any]:
+        out = cls._heads(m, where)
+        del out["kv_heads"]
+        decay = m.get("decay")
+        if not isinstance(decay, list) or len(decay) != out["heads"] or any(
+                isinstance(x, bool) or not isinstance(x, (int, float)) or not 0.0 <= float(x) <= 1.0 for x in decay):
+            raise ConfigError(f"{where}: 'decay' must list one number in [0, 1] for each of the {out['heads']} heads")
+        out["decay"] = [float(x) for x in decay]
+        return out
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "ZetivikConfig":
+        width, vocab = _require_int(d, "width"), _require_int(d, "vocab")
+        eps = _require_number(_sub(d, "norm", "config.json"), "eps", "config.json norm")
+        if eps <= 0:
+            raise ConfigError(f"norm eps must be positive, got {eps}")
+        cap = _require_number(d, "logit_softcap") if d.get("logit_softcap") is not None else None
+        if cap is not None and cap <= 0:
+            raise ConfigError("config.json: logit_softcap must be positive")
+        raw = d.get("layers")
+        if not isinstance(raw, list) or not raw:
+            raise ConfigError("config.json: 'layers' must be a non-empty list")
+        layers = []
+        for i, entry in enumerate(raw):
+            where = f"config.json layers[{i}]"
+            if not isinstance(entry, dict):
+                raise ConfigError(f"{where}: must be an object")
+            kind = entry.get("type")
+            if kind not in cls.MIXERS:
+                raise ConfigError(f"{where}: type {kind!r} is not one of {list(cls.MIXERS)}")
+            mixer = _sub(entry, "mixer", where)
+            if kind == "parallel":
+                sizes = {"left": cls._left(_sub(mixer, "left", where + " mixer"), where + " mixer.left"),
+                         "right": cls._right(_sub(mixer, "right", where + " mixer"), where + " mixer.right"),
+                         "left_scale": _opt_number(mixer, "left_scale", 1.0), "right_scale": _opt_number(mixer, "right_scale", 1.0)}
+            else:
+                sizes = cls._lightning(mixer, where + " mixer")
+            mlp = _sub(entry, "mlp", where, optional=True)
+            ff = None
+            if mlp is not None:
+                if mlp.get("kind") != "dense":
+                    raise ConfigError(f"{where}: mlp kind {mlp.get('kind')!r} is not one of ['dense']")
+                ff = {"kind": "dense", "ff": _require_int(mlp, "ff"), "limit": _require_number(mlp, "limit", where + " mlp")}
+                if ff["limit"] <= 0:
+                    raise ConfigError(f"{where}: mlp limit must be positive")
+            layers.append(ZetivikLayer(type=kind, mixer=sizes, mlp=ff))
+        start = stop = times = 0
+        loop = _sub(d, "loop", "config.json", optional=True)
+        if loop is not None:
+            start, stop = _require_int(loop, "start", 0), _require_int(loop, "stop", 0)
+            times = _require_int(loop, "times", 1)
+            if not 0 <= start < stop <= len(layers):
+                raise ConfigError(f"config.json: loop {start}..{stop} does not lie within the {len(layers)} layers")
+        arch = d.get("architecture") or (d.get("architectures") or [cls.ARCHITECTURE])[0]
+        return cls(architectures=[str(arch)], model_type=str(d.get("model_type", "") or cls.MODEL_TYPE), width=width,
+                   vocab=vocab, norm_eps=eps, logit_softcap=cap, layers=layers, loop_start=start, loop_stop=stop,
+                   loop_times=times)
+
+    @property
+    def vocab_size(self) -> int:
+        return self.vocab
+
+    @property
+    def eos_token_id(self) -> Optional[int]:
+        return None
+
+    def to_dict(self) -> Dict[str, Any]:
+        """The config.json this configuration was read from (its own keys)."""
+        layers = []
+        for l in self.layers:
+            m = {k: (dict(v) if isinstance(v, dict) else v) for k, v in l.mixer.items()}
+            if l.type == "parallel":
+                chunk, rot = m["left"].pop("chunk"), m["left"].pop("rot")
+                if chunk:
+                    m["left"]["mask"] = {"size": chunk}
+                if rot["dims"]:
+                    m["left"]["rot"] = dict(rot)
+            layers.append({"type": l.type, "mixer": m, "mlp": dict(l.mlp) if l.mlp else None})
+        out = {"architecture": self.architecture, "width": self.width, "vocab": self.vocab, "norm": {"eps": self.norm_eps},
+               "layers": layers}
+        if self.logit_softcap is not None:
+            out["logit_softcap"] = self.logit_softcap
+        if self.loop_times:
+            out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return out

@@ -148,12 +148,13 @@ struct AttnMeta {
 // What newer attention designs add to the prompt kernel (all off for plain attention): a cap on the scores,
 // s <- cap * tanh(s / cap); first tokens that stay visible behind the window; a sink (one more term exp(0) in
 // the softmax's denominator, without a value); an output gate (the result times the sigmoid of float32 sums
-// given beside it, [parts][N][gate_stride], first n_heads * HD columns).
+// given beside it, [parts][N][gate_stride], first n_heads * HD columns, or one column per head).  A negative window
+// hides the keys ahead of the query's chunk (first_visible in common.cuh).
 struct PrefillOptions {
   float softcap;
   int keep_first;
   int sink;
-  const float* gate; int gate_parts; long long gate_part_stride; int gate_stride;
+  HeadGate gate;
   // a query temperature (the query at position p counts 1 + coef * ln(floor((p + 1) / every) + 1) times; every = 0:
   // none) and a toll on distance (the score of key j loses r1[head] * ln(1 + r2[head] * (p - j)), after the cap;
   // null: none)
@@ -225,7 +226,7 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
   const float toll1 = opt.dist_r1 ? opt.dist_r1[head] : 0.0f, toll2 = opt.dist_r1 ? opt.dist_r2[head] : 0.0f;
 
   const int kend = pos0 + rows;                                  // keys [.., kend) may be seen
-  const int kfirst = window > 0 ? max(0, pos0 - window + 1) : 0; // first key the first row may see
+  const int kfirst = first_visible(pos0, window);                // first key the first row may see
   const int t_begin = kfirst / BK, t_end = (kend - 1) / BK;
   // kept first tokens: their tiles come first when the window has passed them (tiles [0, n_keep), then
   // [t_begin, t_end]); otherwise the window's tiles hold them anyway
@@ -244,6 +245,8 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
     }
   }
   const int pa_row = pos0 + wr0 + g, pb_row = pa_row + 8;        // positions of this thread's two rows
+  const int lo_a = first_visible(pa_row, window), lo_b = first_visible(pb_row, window);
+  const int warp_lo = first_visible(pos0 + wr0, window), warp_lo_end = first_visible(pos0 + wr0 + 15, window);
   const int warp_last = pos0 + min(wr0 + 15, rows - 1);
 
   // shared-memory byte offsets of this lane's ldmatrix rows, swizzle included (they do not depend on the tile)
@@ -273,8 +276,7 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
     }
     __syncthreads();
     const int key0 = t * BK;
-    const bool active = wr0 < rows && key0 <= warp_last &&
-                        (window <= 0 || key0 + BK > pos0 + wr0 - window + 1 || key0 < keep);
+    const bool active = wr0 < rows && key0 <= warp_last && (key0 + BK > warp_lo || key0 < keep);
     if (active) {
       const unsigned kt = ks_addr + (unsigned)(st * BK * HD * 2);
       const unsigned vt = vs_addr + (unsigned)(st * BK * HD * 2);
@@ -320,7 +322,7 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
       // a tile needs no mask when every row of the warp sees all of it: it ends at or before the warp's first
       // position and starts inside the window of the warp's last one (or lies wholly among the kept first tokens)
       const bool need_mask = key0 + BK - 1 > pos0 + wr0 || key0 + BK > kend ||
-                             (window > 0 && key0 <= pos0 + wr0 + 15 - window && key0 + BK > keep);
+                             (key0 < warp_lo_end && key0 + BK > keep);
       if (need_mask) {
 #pragma unroll
         for (int n = 0; n < BK / 8; ++n) {
@@ -328,7 +330,7 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
           for (int c = 0; c < 4; ++c) {
             const int key = key0 + n * 8 + t4 * 2 + (c & 1);
             const int p = (c & 2) ? pb_row : pa_row;
-            const bool vis = key <= p && key < kend && (window <= 0 || key > p - window || key < keep);
+            const bool vis = key <= p && key < kend && (key >= ((c & 2) ? lo_b : lo_a) || key < keep);
             if (!vis) s[n][c] = -INFINITY;
           }
         }
@@ -403,16 +405,18 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
   const int ra = wr0 + g, rb = ra + 8;
   bf16* oa = out + (size_t)(tok0 + ra) * out_stride + (size_t)head * HD;
   bf16* ob = out + (size_t)(tok0 + rb) * out_stride + (size_t)head * HD;
-  if (opt.gate) {
+  if (opt.gate.p && opt.gate.per_head) {
+    const float fa = ra < rows ? opt.gate.factor(tok0 + ra, head, HD, 0) : 0.0f;
+    const float fb = rb < rows ? opt.gate.factor(tok0 + rb, head, HD, 0) : 0.0f;
+#pragma unroll
+    for (int d = 0; d < DT; ++d) { o[d][0] *= fa; o[d][1] *= fa; o[d][2] *= fb; o[d][3] *= fb; }
+  } else if (opt.gate.p) {
 #pragma unroll
     for (int d = 0; d < DT; ++d) {
-      const int col = head * HD + d * 8 + t4 * 2;
+      const int col = d * 8 + t4 * 2;
       float ga[2] = {0.0f, 0.0f}, gb[2] = {0.0f, 0.0f};
-      for (int sl = 0; sl < opt.gate_parts; ++sl) {
-        const float* gp = opt.gate + (size_t)sl * opt.gate_part_stride + col;
-        if (ra < rows) { ga[0] += gp[(size_t)(tok0 + ra) * opt.gate_stride]; ga[1] += gp[(size_t)(tok0 + ra) * opt.gate_stride + 1]; }
-        if (rb < rows) { gb[0] += gp[(size_t)(tok0 + rb) * opt.gate_stride]; gb[1] += gp[(size_t)(tok0 + rb) * opt.gate_stride + 1]; }
-      }
+      if (ra < rows) { ga[0] = opt.gate.sums(tok0 + ra, head, HD, col); ga[1] = opt.gate.sums(tok0 + ra, head, HD, col + 1); }
+      if (rb < rows) { gb[0] = opt.gate.sums(tok0 + rb, head, HD, col); gb[1] = opt.gate.sums(tok0 + rb, head, HD, col + 1); }
       o[d][0] *= 1.0f / (1.0f + __expf(-ga[0])); o[d][1] *= 1.0f / (1.0f + __expf(-ga[1]));
       o[d][2] *= 1.0f / (1.0f + __expf(-gb[0])); o[d][3] *= 1.0f / (1.0f + __expf(-gb[1]));
     }
@@ -459,6 +463,7 @@ struct QkvPrep {
 // distance (the score of key j loses r1[head] * ln(1 + r2[head] * (p - j)); null: none).
 struct ScoreShape {
   float q_temp_coef; int q_temp_every; const float* dist_r1; const float* dist_r2;
+  HeadGate gate;            // the heads' results times the sigmoid of sums beside them
 };
 
 // PREP: the kernel takes the place of the bias/rotation/cache-write kernel for the token it decodes.  Every
@@ -488,7 +493,7 @@ attn_decode_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __
   const int nrows = min(8, ratio - hc * 8);                     // query heads of this block
   const int tok = m.entry_q_start[e];
   const int len = m.entry_ctx_start[e] + 1;                     // keys [0, len) exist; the query sits at len - 1
-  const int kfirst = window > 0 ? max(0, len - window) : 0;
+  const int kfirst = first_visible(len - 1, window);
   const int total = len - kfirst;
   int chunk = (total + n_splits - 1) / n_splits;
   chunk = (chunk + BK - 1) / BK * BK;
@@ -721,7 +726,9 @@ attn_decode_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __
     }
     const int head = h0 + row;
     if (n_splits == 1) {
-      out[(size_t)tok * out_stride + (size_t)head * HD + d] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+      float y = l > 0.0f ? acc / l : 0.0f;
+      if (shape.gate.p) y *= shape.gate.factor(tok, head, HD, d);
+      out[(size_t)tok * out_stride + (size_t)head * HD + d] = __float2bfloat16_rn(y);
     } else {
       const size_t p = ((size_t)dec * n_heads + head) * n_splits + split;
       part_o[p * HD + d] = acc;
@@ -734,7 +741,8 @@ attn_decode_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __
 // batch sizes) are loaded in one go, maxima, sums and outputs together, so the block waits for memory once.
 __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          bf16* __restrict__ out, long long out_stride, const int* __restrict__ dec_entries,
-                                         const int* __restrict__ entry_q_start, int n_heads, int head_dim, int n_splits) {
+                                         const int* __restrict__ entry_q_start, int n_heads, int head_dim, int n_splits,
+                                         HeadGate gate) {
   pdl_launch_dependents();
   const int dec = blockIdx.x, head = blockIdx.y;
   const int tok = entry_q_start[dec_entries[dec]];            // the step's metadata: read before the wait
@@ -762,7 +770,9 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const
           l += ml[s].y * f;
           acc += po[s] * f;
         }
-      out[(size_t)tok * out_stride + (size_t)head * head_dim + d] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+      float y = l > 0.0f ? acc / l : 0.0f;
+      if (gate.p) y *= gate.factor(tok, head, head_dim, d);
+      out[(size_t)tok * out_stride + (size_t)head * head_dim + d] = __float2bfloat16_rn(y);
     }
     return;
   }
@@ -778,7 +788,9 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const
       l += part_ml[(p0 + s) * 2 + 1] * f;
       acc += part_o[(p0 + s) * head_dim + d] * f;
     }
-    out[(size_t)tok * out_stride + (size_t)head * head_dim + d] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+    float y = l > 0.0f ? acc / l : 0.0f;
+    if (gate.p) y *= gate.factor(tok, head, head_dim, d);
+    out[(size_t)tok * out_stride + (size_t)head * head_dim + d] = __float2bfloat16_rn(y);
   }
 }
 
@@ -1189,7 +1201,7 @@ int launch_decode(const void* q, long long q_stride, void* out, long long out_st
       head_chunks, scale, window, n_splits, prep, shape);
   if (!rc) rc = IFX_LAUNCH_CHECK();
   if (rc || n_splits == 1) return rc;
-  rc = launch_pdl(attn_decode_merge_kernel, dim3(n_dec, n_heads), dim3(HD < 128 ? HD : 128), 0, stream, part_o, part_ml, (bf16*)out, out_stride, dec_entries, m.entry_q_start, n_heads, HD, n_splits);
+  rc = launch_pdl(attn_decode_merge_kernel, dim3(n_dec, n_heads), dim3(HD < 128 ? HD : 128), 0, stream, part_o, part_ml, (bf16*)out, out_stride, dec_entries, m.entry_q_start, n_heads, HD, n_splits, shape.gate);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 // Blocks of the even-share decode kernel that the GPU holds at once (asked once per head size); negative: a CUDA error.
@@ -1240,22 +1252,24 @@ int launch_decode_even(const void* q, long long q_stride, void* out, long long o
 
 // head_dim 64 or 128; page_size a power of two; q rows 4-byte aligned.
 // Query tiles are 64 tokens of one entry (tile_entry / tile_q0).
-// q_temp_every > 0: a query temperature; dist_r1 / dist_r2 ([n_heads] float32 or null): a toll on distance.
+// q_temp_every > 0: a query temperature; dist_r1 / dist_r2 ([n_heads] float32 or null): a toll on distance; gate_per_head:
+// one gate column per head instead of one per element; window < 0: chunks of -window positions.
 IFX_API int ifx_attn_prefill_bf16_ex2(const void* q, long long q_stride, void* out, long long out_stride,
                                   void* k_layer, void* v_layer, long long page_stride, int page_size,
                                   const int* block_tables, int bt_stride, const int* tile_entry, const int* tile_q0,
                                   int n_tiles, const int* entry_q_start, const int* entry_q_len,
                                   const int* entry_ctx_start, int n_heads, int n_kv, int head_dim, float scale,
                                   int window, float softcap, int keep_first, int sink, const float* gate, int gate_parts,
-                                  long long gate_part_stride, int gate_stride, float q_temp_coef, int q_temp_every,
-                                  const float* dist_r1, const float* dist_r2, cudaStream_t stream) {
+                                  long long gate_part_stride, int gate_stride, int gate_per_head, float q_temp_coef,
+                                  int q_temp_every, const float* dist_r1, const float* dist_r2, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (n_kv < 1 || n_heads % n_kv || n_tiles > 65535) return IFX_ERR_UNSUPPORTED;
   if (page_size <= 0 || (page_size & (page_size - 1))) return IFX_ERR_UNSUPPORTED;
   if ((q_stride & 1) || (out_stride & 1) || ((uintptr_t)q & 3) || ((uintptr_t)out & 3)) return IFX_ERR_ALIGNMENT;
   if ((page_stride & 7) || ((uintptr_t)k_layer & 15) || ((uintptr_t)v_layer & 15)) return IFX_ERR_ALIGNMENT;
   if (softcap < 0.0f || keep_first < 0 || q_temp_every < 0 || (dist_r1 != nullptr) != (dist_r2 != nullptr)) return IFX_ERR_UNSUPPORTED;
-  PrefillOptions opt{softcap, keep_first, sink, gate, gate_parts, gate_part_stride, gate_stride, q_temp_coef, q_temp_every, dist_r1, dist_r2};
+  PrefillOptions opt{softcap, keep_first, sink, HeadGate{gate, gate_parts, gate_part_stride, gate_stride, gate_per_head},
+                     q_temp_coef, q_temp_every, dist_r1, dist_r2};
   PagedKV kv = make_kv(k_layer, v_layer, page_stride, page_size, head_dim);
   AttnMeta m{block_tables, bt_stride, entry_q_start, entry_q_len, entry_ctx_start};
   if (head_dim == 128)
@@ -1275,7 +1289,7 @@ IFX_API int ifx_attn_prefill_bf16_ex(const void* q, long long q_stride, void* ou
   return ifx_attn_prefill_bf16_ex2(q, q_stride, out, out_stride, k_layer, v_layer, page_stride, page_size, block_tables, bt_stride,
                                    tile_entry, tile_q0, n_tiles, entry_q_start, entry_q_len, entry_ctx_start, n_heads, n_kv,
                                    head_dim, scale, window, softcap, keep_first, sink, gate, gate_parts, gate_part_stride,
-                                   gate_stride, 0.0f, 0, nullptr, nullptr, stream);
+                                   gate_stride, 0, 0.0f, 0, nullptr, nullptr, stream);
 }
 
 IFX_API int ifx_attn_prefill_bf16(const void* q, long long q_stride, void* out, long long out_stride,
@@ -1291,17 +1305,20 @@ IFX_API int ifx_attn_prefill_bf16(const void* q, long long q_stride, void* out, 
 
 // Scratch: part_o float32 [n_dec * n_heads * n_splits * head_dim], part_ml float32
 // [n_dec * n_heads * n_splits * 2] (unused when n_splits == 1).
-// q_temp_every > 0: a query temperature; dist_r1 / dist_r2 ([n_heads] float32 or null): a toll on distance.
+// q_temp_every > 0: a query temperature; dist_r1 / dist_r2 ([n_heads] float32 or null): a toll on distance; gate: float32
+// slices [gate_parts][N][gate_stride] or null, a column per element or (gate_per_head) per head; window < 0: chunks.
 IFX_API int ifx_attn_decode_bf16_ex(const void* q, long long q_stride, void* out, long long out_stride,
                                     void* k_layer, void* v_layer, long long page_stride, int page_size,
                                     const int* block_tables, int bt_stride, const int* dec_entries, int n_dec,
                                     const int* entry_q_start, const int* entry_q_len, const int* entry_ctx_start,
                                     float* part_o, float* part_ml, int n_heads, int n_kv, int head_dim, float scale,
                                     int window, int n_splits, float q_temp_coef, int q_temp_every, const float* dist_r1,
-                                    const float* dist_r2, cudaStream_t stream) {
+                                    const float* dist_r2, const float* gate, int gate_parts, long long gate_part_stride,
+                                    int gate_stride, int gate_per_head, cudaStream_t stream) {
   if (n_dec <= 0) return 0;
   if (q_temp_every < 0 || (dist_r1 != nullptr) != (dist_r2 != nullptr)) return IFX_ERR_UNSUPPORTED;
-  const ScoreShape shape{q_temp_coef, q_temp_every, dist_r1, dist_r2};
+  const ScoreShape shape{q_temp_coef, q_temp_every, dist_r1, dist_r2,
+                         HeadGate{gate, gate_parts, gate_part_stride, gate_stride, gate_per_head}};
   if (n_kv < 1 || n_heads % n_kv || n_splits < 1 || n_splits > 65535) return IFX_ERR_UNSUPPORTED;
   if (page_size <= 0 || (page_size & (page_size - 1))) return IFX_ERR_UNSUPPORTED;
   if ((q_stride & 1) || ((uintptr_t)q & 3)) return IFX_ERR_ALIGNMENT;
@@ -1324,7 +1341,7 @@ IFX_API int ifx_attn_decode_bf16(const void* q, long long q_stride, void* out, l
                                  int window, int n_splits, cudaStream_t stream) {
   return ifx_attn_decode_bf16_ex(q, q_stride, out, out_stride, k_layer, v_layer, page_stride, page_size, block_tables, bt_stride,
                                  dec_entries, n_dec, entry_q_start, entry_q_len, entry_ctx_start, part_o, part_ml, n_heads, n_kv,
-                                 head_dim, scale, window, n_splits, 0.0f, 0, nullptr, nullptr, stream);
+                                 head_dim, scale, window, n_splits, 0.0f, 0, nullptr, nullptr, nullptr, 0, 0, 0, 0, stream);
 }
 
 // The same for a step of single tokens only, with the work of ifx_qkv_rope_kv_write folded in: qkv is the

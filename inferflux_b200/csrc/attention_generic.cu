@@ -16,7 +16,8 @@
 // the scores, s <- cap * tanh(s / cap); kept first tokens, which stay visible behind the window
 // (key j visible iff j <= p and (p - j < w or j < keep_first)); a sink, one more term of score 0 and no value
 // in the softmax's denominator, p_j = exp(s_j) / (1 + sum exp(s_j)); an output gate, every element of a
-// head's result times sigmoid of a float32 row given beside it.
+// head's result times sigmoid of a float32 row given beside it, or every head's result times one such number.
+// A negative window hides the keys ahead of the query's chunk (first_visible in common.cuh).
 //
 // Tiles start at multiples of 32 keys and keys are added in index order, so in
 // float32 the result for a token does not depend on how the prompt was cut.
@@ -42,8 +43,7 @@ struct AttnOptions {
   float softcap;              // 0 = none
   int keep_first;             // first tokens that stay visible behind the window
   int sink;                   // 1 = the denominator has one more term exp(0)
-  const float* gate;          // [N][gate_stride] float32 or null: out *= sigmoid(gate[row][head * v_dim + d])
-  int gate_parts; long long gate_part_stride; int gate_stride;
+  HeadGate gate;              // float32 rows: out *= sigmoid(gate[row][head * v_dim + d]), or of gate[row][head]
   float q_temp_coef;          // the query at position p counts 1 + coef * ln(floor((p + 1) / every) + 1) times; every = 0: none
   int q_temp_every;
   const float* dist_r1;       // [n_heads] or null: the score of key j loses r1[head] * ln(1 + r2[head] * (p - j))
@@ -102,7 +102,9 @@ attn_paged_generic_kernel(const T* __restrict__ q, long long q_stride, T* __rest
 
   const int kend = pos0 + rows - 1;               // last key any row of the tile may see
   int kstart = 0;
-  if (window > 0) kstart = max(0, pos0 - window + 1) & ~(BKEYS - 1);
+  if (window != 0) kstart = first_visible(pos0, window) & ~(BKEYS - 1);
+  const int lo0 = first_visible(pos0 + r0, window), lo1 = first_visible(pos0 + r1, window);
+  const int kept = window > 0 ? opt.keep_first : 0;
   // with kept first tokens the tiles [0, keep_end) come first, then those from kstart on
   const int keep_end = window > 0 ? min((opt.keep_first + BKEYS - 1) & ~(BKEYS - 1), kstart) : 0;
 
@@ -148,7 +150,7 @@ attn_paged_generic_kernel(const T* __restrict__ q, long long q_stride, T* __rest
       for (int rr = 0; rr < 2; ++rr) {
         if (rr == 1 && !two) break;
         const int p = pos0 + r0 + rr;
-        const bool visible = key <= p && (window <= 0 || key > p - window || key < opt.keep_first);
+        const bool visible = key <= p && (key >= (rr ? lo1 : lo0) || key < kept);
         const float sc = shaped_score(opt, rr ? s1 : s0, scale * query_temperature(opt, p), toll1, toll2, visible ? p - key : 0);
         const float s = visible ? sc : -INFINITY;
         const float m_new = fmaxf(m[rr], warp_max(s));
@@ -182,12 +184,7 @@ attn_paged_generic_kernel(const T* __restrict__ q, long long q_stride, T* __rest
       const int d = lane + 32 * a;
       if (d >= v_dim) continue;
       float y = o[rr][a] * inv;
-      if (opt.gate) {
-        float g = 0.0f;
-        for (int s = 0; s < opt.gate_parts; ++s)
-          g += opt.gate[(size_t)s * opt.gate_part_stride + (size_t)(tok0 + r) * opt.gate_stride + (size_t)head * v_dim + d];
-        y *= 1.0f / (1.0f + expf(-g));
-      }
+      if (opt.gate.p) y *= opt.gate.factor(tok0 + r, head, v_dim, d);
       orow[d] = Num<T>::from_f(y);
     }
   }
@@ -221,7 +218,8 @@ attn_single_token_kernel(const T* __restrict__ q, long long q_stride, T* __restr
   for (int d = tid; d < head_dim; d += blockDim.x) qs[d] = Num<T>::to_f(q[(size_t)tok * q_stride + (size_t)head * head_dim + d]);
   __syncthreads();
   int kstart = 0;
-  if (window > 0) kstart = max(0, p - window + 1) & ~(BKEYS - 1);
+  const int lo = first_visible(p, window), kept = window > 0 ? opt.keep_first : 0;
+  if (window != 0) kstart = lo & ~(BKEYS - 1);
   const int keep_end = window > 0 ? min((opt.keep_first + BKEYS - 1) & ~(BKEYS - 1), kstart) : 0;
   const int n_keep = keep_end / BKEYS, n_tiles = n_keep + (p - kstart) / BKEYS + 1;
   const float scale_temp = scale * query_temperature(opt, p);
@@ -236,7 +234,7 @@ attn_single_token_kernel(const T* __restrict__ q, long long q_stride, T* __restr
   for (int it = warp; it < n_tiles; it += DEC_WARPS) {
     const int k0 = it < n_keep ? it * BKEYS : kstart + (it - n_keep) * BKEYS;
     const int key = k0 + lane;
-    const bool visible = key <= p && (window <= 0 || key > p - window || key < opt.keep_first);
+    const bool visible = key <= p && (key >= lo || key < kept);
     const int page = key <= p ? bt[key >> kv.page_shift] : -1;
     float sc = -INFINITY;
     if (visible && page >= 0) {
@@ -338,12 +336,7 @@ attn_single_token_kernel(const T* __restrict__ q, long long q_stride, T* __restr
       float y = 0.0f;
       for (int w = 0; w < DEC_WARPS; ++w) y = fmaf(wo[w * v_dim + d], f[w], y);
       y *= inv;
-      if (opt.gate) {
-        float g = 0.0f;
-        for (int sl = 0; sl < opt.gate_parts; ++sl)
-          g += opt.gate[(size_t)sl * opt.gate_part_stride + (size_t)tok * opt.gate_stride + (size_t)head * v_dim + d];
-        y *= 1.0f / (1.0f + expf(-g));
-      }
+      if (opt.gate.p) y *= opt.gate.factor(tok, head, v_dim, d);
       orow[d] = Num<T>::from_f(y);
     }
   }
@@ -409,7 +402,8 @@ int dispatch_generic(const void* q, long long q_stride, void* out, long long out
 
 // Query tiles are 16 tokens of one entry: tile_entry / tile_q0 list them.
 // head_dim and v_dim: any positive size up to 256; n_heads must be a multiple of n_kv.  The options are
-// those of AttnOptions; gate: float32 slices [gate_parts][N][gate_stride] whose sum is the gate's argument.
+// those of AttnOptions; gate: float32 slices [gate_parts][N][gate_stride] whose sum is the gate's argument, a column per
+// element or (gate_per_head) per head.  window: > 0 the last so many positions, < 0 chunks of so many, 0 everything.
 // q_temp_every > 0: the query at position p is multiplied by 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1);
 // dist_r1, dist_r2 ([n_heads] float32 or null): the score of key j loses r1 * ln(1 + r2 * (p - j)), after the cap;
 // sink_value ([n_heads] float32 or null): the sink's score where it is not 0.
@@ -421,7 +415,7 @@ IFX_API int ifx_attn_paged_generic_ex2(const void* q, long long q_stride, void* 
                                        int n_heads, int n_kv, int head_dim, float scale, int window,
                                        int v_dim, float softcap, int keep_first, int sink,
                                        const float* gate, int gate_parts, long long gate_part_stride, int gate_stride,
-                                       int single_tokens, float q_temp_coef, int q_temp_every, const float* dist_r1,
+                                       int gate_per_head, int single_tokens, float q_temp_coef, int q_temp_every, const float* dist_r1,
                                        const float* dist_r2, const float* sink_value, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (head_dim < 1 || head_dim > 256 || v_dim < 1 || v_dim > 256 || n_kv < 1 || n_heads % n_kv) return IFX_ERR_UNSUPPORTED;
@@ -433,7 +427,7 @@ IFX_API int ifx_attn_paged_generic_ex2(const void* q, long long q_stride, void* 
   while ((1 << kv.page_shift) < page_size) ++kv.page_shift;
   AttnBatch b{block_tables, bt_stride, tile_entry, tile_q0, entry_q_start, entry_q_len, entry_ctx_start};
   if (q_temp_every < 0 || (dist_r1 != nullptr) != (dist_r2 != nullptr)) return IFX_ERR_UNSUPPORTED;
-  AttnOptions opt{v_dim, page_size * v_dim, softcap, keep_first, sink, gate, gate_parts, gate_part_stride, gate_stride,
+  AttnOptions opt{v_dim, page_size * v_dim, softcap, keep_first, sink, HeadGate{gate, gate_parts, gate_part_stride, gate_stride, gate_per_head},
                   q_temp_coef, q_temp_every, dist_r1, dist_r2, sink_value};
   if (single_tokens) {            // every tile is one token (tile_q0 = its place in its entry): the kernel for those
     if (dtype == IFX_F32)
@@ -461,7 +455,7 @@ IFX_API int ifx_attn_paged_generic_ex(const void* q, long long q_stride, void* o
   return ifx_attn_paged_generic_ex2(q, q_stride, out, out_stride, dtype, k_layer, v_layer, page_stride, page_size,
                                     block_tables, bt_stride, tile_entry, tile_q0, n_tiles, entry_q_start, entry_q_len,
                                     entry_ctx_start, n_heads, n_kv, head_dim, scale, window, v_dim, softcap, keep_first,
-                                    sink, gate, gate_parts, gate_part_stride, gate_stride, single_tokens, 0.0f, 0,
+                                    sink, gate, gate_parts, gate_part_stride, gate_stride, 0, single_tokens, 0.0f, 0,
                                     nullptr, nullptr, nullptr, stream);
 }
 

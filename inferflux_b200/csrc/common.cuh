@@ -85,6 +85,29 @@ struct PagedKV {
   int page_shift;          // log2(page_size)
 };
 
+// How far back attention reaches is one int: 0 = to the sequence's start, w > 0 = the last w positions (the token's
+// own among them), -c < 0 = to the start of the token's chunk of c positions, chunks counted from position 0.
+// The first position that the query at position p sees; it never falls as p grows.
+__device__ __forceinline__ int first_visible(int p, int window) {
+  if (window > 0) return max(0, p - window + 1);
+  return window < 0 ? p - p % -window : 0;
+}
+
+// An output gate of attention: a head's result times the sigmoid of float32 sums given beside it, one number per
+// element (column head * v_dim + d of a row) or, with per_head, one per head (column head).  p null: none.
+struct HeadGate {
+  const float* p; int parts; long long part_stride; int stride; int per_head;
+  __device__ __forceinline__ float sums(int row, int head, int v_dim, int d) const {
+    const float* g = p + (size_t)row * stride + (per_head ? head : head * v_dim + d);
+    float v = 0.0f;
+    for (int s = 0; s < parts; ++s) v += g[(size_t)s * part_stride];
+    return v;
+  }
+  __device__ __forceinline__ float factor(int row, int head, int v_dim, int d) const {
+    return 1.0f / (1.0f + expf(-sums(row, head, v_dim, d)));
+  }
+};
+
 #define IFX_LAUNCH_CHECK() ((int)cudaGetLastError())
 
 // Programmatic dependent launch.  Every kernel of the library starts with pdl_enter(): it lets the kernel

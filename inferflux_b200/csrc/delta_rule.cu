@@ -283,6 +283,32 @@ head_norm_gate_kernel(const float* __restrict__ o, long long o_stride, const flo
     dst[i] = Num<TO>::from_f(v);
   }
 }
+
+// The same with a block a (token, head), for heads wide enough that a warp would walk long rows (a norm over all heads of
+// a token together, say).
+template <typename TO>
+__global__ void __launch_bounds__(512)
+wide_norm_gate_kernel(const float* __restrict__ o, long long o_stride, const float* __restrict__ g, long long g_stride,
+                      const float* __restrict__ w, TO* __restrict__ out, long long out_stride, int heads, int vdim,
+                      float eps, int gate) {
+  __shared__ float scratch[32];
+  pdl_enter();
+  const int t = blockIdx.x / heads, h = blockIdx.x - t * heads;
+  const float* src = o + (size_t)t * o_stride + (size_t)h * vdim;
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < vdim; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)vdim + eps);
+  const float* gr = g ? g + (size_t)t * g_stride + (size_t)h * vdim : nullptr;
+  TO* dst = out + (size_t)t * out_stride + (size_t)h * vdim;
+  for (int i = threadIdx.x; i < vdim; i += blockDim.x) {
+    float v = src[i] * inv;
+    if (w) v *= w[h * vdim + i];
+    if (gate == 1) v *= 1.0f / (1.0f + expf(-gr[i]));
+    else if (gate == 2) v *= gr[i] / (1.0f + expf(-gr[i]));
+    dst[i] = Num<TO>::from_f(v);
+  }
+}
+constexpr int WIDE_HEAD = 512;          // from this width on
 }  // namespace
 
 // proj float32 rows hold r, k, v heads and the raw removal rates from the given columns on; wraw float32 rows the raw
@@ -343,6 +369,15 @@ IFX_API int ifx_head_norm_gate(const float* o, long long o_stride, const float* 
   const long long warps = (long long)n_rows * heads;
   const int blocks = (int)((warps + 7) / 8);
   int rc;
+  if (vdim >= WIDE_HEAD && (out_dtype == IFX_BF16 || out_dtype == IFX_F32)) {
+    const dim3 block(vdim >= 2048 ? 512 : 256);
+    rc = out_dtype == IFX_BF16
+        ? launch_pdl(wide_norm_gate_kernel<bf16>, dim3((unsigned)warps), block, 0, stream, o, o_stride, g, g_stride, w, (bf16*)out,
+                     out_stride, heads, vdim, eps, gate)
+        : launch_pdl(wide_norm_gate_kernel<float>, dim3((unsigned)warps), block, 0, stream, o, o_stride, g, g_stride, w, (float*)out,
+                     out_stride, heads, vdim, eps, gate);
+    return rc ? rc : IFX_LAUNCH_CHECK();
+  }
   if (out_dtype == IFX_BF16)
     rc = launch_pdl(head_norm_gate_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, o, o_stride, g, g_stride, w, (bf16*)out,
                     out_stride, n_rows, heads, vdim, eps, gate);

@@ -571,3 +571,21 @@ IFX_API int ifx_activation(const float* z, long long z_stride, int parts, long l
     return IFX_ERR_UNSUPPORTED;
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
+
+namespace {
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long total, float cap) {
+  pdl_enter();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+}  // namespace
+
+// x <- cap * tanh(x / cap) in place, float32.
+IFX_API int ifx_softcap(float* x, long long total, float cap, cudaStream_t stream) {
+  if (total <= 0) return 0;
+  if (!(cap > 0.0f)) return IFX_ERR_UNSUPPORTED;
+  long long blocks = (total + 255) / 256;
+  if (blocks > 148 * 8) blocks = 148 * 8;
+  const int rc = launch_pdl(softcap_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, total, cap);
+  return rc ? rc : IFX_LAUNCH_CHECK();
+}

@@ -1,16 +1,17 @@
 // RMS norm over equal consecutive parts of a row, fused with the sum into the float32 stream:
 //
-//   r = residual + sa * (a_0 + a_1 + ...) + sb * (b_0 + b_1 + ...)        (either addend may be absent)
+//   r = residual + sa * (a_0 + a_1 + ...) + sb * (b_0 + b_1 + ...) + x + v        (each addend may be absent)
 //   out[i] = r[i] / sqrt(mean(r[part of i]^2) + eps) * weight[i]
 //
 // The row is cut into `groups` parts of hidden / groups elements; every part is divided by its own root mean
 // square.  groups = 1 is the plain RMS norm.  The two addends, each given as float32 or bfloat16 slices whose sum
 // it is and each with a factor of its own, are what a layer with two mixers side by side hands on
-// (sa * left + sb * right): the weighted sum, the sum into the stream and the norm are one pass.
+// (sa * left + sb * right): the weighted sum, the sum into the stream and the norm are one pass.  x (float32 rows) and
+// v (one float32 vector for all rows) are what joins the stream where a pass over a stretch of layers begins.
 //
 // One block per output row; the row lies in shared memory between the passes.  A part's squares are added by one
-// warp, lane by lane and then over the warp, so the order of additions depends on the part's length alone, never on
-// what else is in the batch.  Source row = rows ? rows[blockIdx.x] : blockIdx.x; in that gather mode the stream is
+// warp, lane by lane and then over the warp, or, where the row is one part, by the whole block, so the order of
+// additions depends on the part's length alone, never on what else is in the batch.  Source row = rows ? rows[blockIdx.x] : blockIdx.x; in that gather mode the stream is
 // left untouched.
 #include "common.cuh"
 
@@ -41,7 +42,7 @@ __global__ void add_group_rmsnorm_kernel(float* __restrict__ residual, const TD*
                                          long long a_stride, float a_scale, const TD* __restrict__ b, int b_parts,
                                          long long b_stride, float b_scale, const float* __restrict__ weight, float eps,
                                          int groups, TO* __restrict__ out, const int* __restrict__ rows, int hidden,
-                                         int write_residual) {
+                                         int write_residual, const float* __restrict__ x, const float* __restrict__ vec) {
   pdl_enter();
   extern __shared__ __align__(16) float gn_smem[];
   float* row_buf = gn_smem;                 // [hidden]
@@ -49,12 +50,13 @@ __global__ void add_group_rmsnorm_kernel(float* __restrict__ residual, const TD*
   const int src = rows ? rows[blockIdx.x] : blockIdx.x;
   float* r = residual + (size_t)src * hidden;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  const bool adds = a || b || x || vec;
   if (VEC) {                                // hidden a multiple of 4, float32 addends, everything on 16-byte boundaries
     const float* ar = a ? reinterpret_cast<const float*>(a) + (size_t)src * hidden : nullptr;
     const float* br = b ? reinterpret_cast<const float*>(b) + (size_t)src * hidden : nullptr;
     for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
       float4 v = *reinterpret_cast<const float4*>(r + i);
-      if (a || b) {
+      if (adds) {
         float4 sa = make_float4(0.f, 0.f, 0.f, 0.f), sb = sa;
         for (int p = 0; ar && p < a_parts; ++p) {
           const float4 t = *reinterpret_cast<const float4*>(ar + (size_t)p * a_stride + i);
@@ -66,6 +68,14 @@ __global__ void add_group_rmsnorm_kernel(float* __restrict__ residual, const TD*
         }
         v.x += fmaf(b_scale, sb.x, a_scale * sa.x); v.y += fmaf(b_scale, sb.y, a_scale * sa.y);
         v.z += fmaf(b_scale, sb.z, a_scale * sa.z); v.w += fmaf(b_scale, sb.w, a_scale * sa.w);
+        if (x) {
+          const float4 t = *reinterpret_cast<const float4*>(x + (size_t)src * hidden + i);
+          v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w;
+        }
+        if (vec) {
+          const float4 t = *reinterpret_cast<const float4*>(vec + i);
+          v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w;
+        }
         if (write_residual) *reinterpret_cast<float4*>(r + i) = v;
       }
       *reinterpret_cast<float4*>(row_buf + i) = v;
@@ -77,19 +87,29 @@ __global__ void add_group_rmsnorm_kernel(float* __restrict__ residual, const TD*
       if (a) add = a_scale * slices_sum<TD>(a + (size_t)src * hidden + i, a_parts, a_stride);
       if (b) add = fmaf(b_scale, slices_sum<TD>(b + (size_t)src * hidden + i, b_parts, b_stride), add);
       if (a || b) v += add;
+      if (x) v += x[(size_t)src * hidden + i];
+      if (vec) v += vec[i];
       row_buf[i] = v;
-      if (write_residual && (a || b)) r[i] = v;
+      if (write_residual && adds) r[i] = v;
     }
   }
   __syncthreads();
   if (!out) return;
   const int gs = hidden / groups;
-  for (int g = warp; g < groups; g += nwarps) {
-    const float* part = row_buf + (size_t)g * gs;
+  if (groups == 1) {
+    __shared__ float scratch[32];
     float ss = 0.0f;
-    for (int i = lane; i < gs; i += 32) ss = fmaf(part[i], part[i], ss);
-    ss = warp_sum(ss);
-    if (lane == 0) rstd[g] = 1.0f / sqrtf(ss / (float)gs + eps);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) ss = fmaf(row_buf[i], row_buf[i], ss);
+    ss = block_sum(ss, scratch);
+    if (threadIdx.x == 0) rstd[0] = 1.0f / sqrtf(ss / (float)hidden + eps);
+  } else {
+    for (int g = warp; g < groups; g += nwarps) {
+      const float* part = row_buf + (size_t)g * gs;
+      float ss = 0.0f;
+      for (int i = lane; i < gs; i += 32) ss = fmaf(part[i], part[i], ss);
+      ss = warp_sum(ss);
+      if (lane == 0) rstd[g] = 1.0f / sqrtf(ss / (float)gs + eps);
+    }
   }
   __syncthreads();
   TO* o = out + (size_t)blockIdx.x * hidden;
@@ -107,12 +127,14 @@ __global__ void add_group_rmsnorm_kernel(float* __restrict__ residual, const TD*
 template <typename TD, typename TO>
 int launch_group_norm(float* residual, const void* a, int a_parts, long long a_stride, float a_scale, const void* b,
                       int b_parts, long long b_stride, float b_scale, const float* weight, float eps, int groups,
-                      void* out, const int* rows, int n_rows, int hidden, int write_residual, cudaStream_t stream) {
+                      void* out, const int* rows, int n_rows, int hidden, int write_residual, const float* x,
+                      const float* vec_add, cudaStream_t stream) {
   const size_t smem = ((size_t)hidden + groups) * sizeof(float);
   if (smem > 200 * 1024) return IFX_ERR_UNSUPPORTED;
   // 16-byte accesses where everything allows them; the order of every addition is the same in both shapes
   const bool vec = sizeof(TD) == 4 && hidden % 4 == 0 && (a_stride & 3) == 0 && (b_stride & 3) == 0 &&
-                   (((uintptr_t)residual | (uintptr_t)a | (uintptr_t)b | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+                   (((uintptr_t)residual | (uintptr_t)a | (uintptr_t)b | (uintptr_t)weight | (uintptr_t)out | (uintptr_t)x |
+                     (uintptr_t)vec_add) & 15) == 0;
   auto kern = vec ? add_group_rmsnorm_kernel<TD, TO, true> : add_group_rmsnorm_kernel<TD, TO, false>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -121,24 +143,27 @@ int launch_group_norm(float* residual, const void* a, int a_parts, long long a_s
   int threads = 128;
   while (threads < 1024 && threads * 4 < hidden) threads <<= 1;
   const int rc = launch_pdl(kern, dim3(n_rows), dim3(threads), smem, stream, residual, (const TD*)a, a_parts, a_stride, a_scale,
-                            (const TD*)b, b_parts, b_stride, b_scale, weight, eps, groups, (TO*)out, rows, hidden, write_residual);
+                            (const TD*)b, b_parts, b_stride, b_scale, weight, eps, groups, (TO*)out, rows, hidden, write_residual,
+                            x, vec_add);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 }  // namespace
 
 // delta_dtype (of a and b) / out_dtype: IFX_F32 or IFX_BF16.  a, b and out may be null; a_parts / b_parts slices
-// lie a_stride / b_stride elements apart.  groups must divide hidden.
+// lie a_stride / b_stride elements apart.  x float32 [N][hidden] and vec_add float32 [hidden] may be null.  groups must
+// divide hidden.
 IFX_API int ifx_add_group_rmsnorm(float* residual, const void* a, int a_parts, long long a_stride, float a_scale,
                                   const void* b, int b_parts, long long b_stride, float b_scale, int delta_dtype,
                                   const float* weight, float eps, int groups, void* out, int out_dtype, const int* rows,
-                                  int n_rows, int hidden, int write_residual, cudaStream_t stream) {
+                                  int n_rows, int hidden, int write_residual, const float* x, const float* vec_add,
+                                  cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (rows && write_residual) return IFX_ERR_UNSUPPORTED;
   if (groups < 1 || hidden < 1 || hidden % groups) return IFX_ERR_UNSUPPORTED;
   if (a_parts < 1) a_parts = 1;
   if (b_parts < 1) b_parts = 1;
 #define IFX_GN(TD, TO) return launch_group_norm<TD, TO>(residual, a, a_parts, a_stride, a_scale, b, b_parts, b_stride, b_scale, weight, \
-                                                        eps, groups, out, rows, n_rows, hidden, write_residual, stream)
+                                                        eps, groups, out, rows, n_rows, hidden, write_residual, x, vec_add, stream)
   if (delta_dtype == IFX_F32 && out_dtype == IFX_F32) IFX_GN(float, float);
   if (delta_dtype == IFX_F32 && out_dtype == IFX_BF16) IFX_GN(float, bf16);
   if (delta_dtype == IFX_BF16 && out_dtype == IFX_BF16) IFX_GN(bf16, bf16);

@@ -8,6 +8,13 @@
 //   value mixing: mode 1 stores the token's values in v_first; mode 2 computes v <- (1 - lambda) v + lambda v_first
 //   q goes to q_out, k and v into the paged cache at slot_map.
 //
+// A second kernel serves designs that norm every query and key head by itself, with one weight of the head's size for
+// all query heads and one for all key heads, and whose projections may have biases that are added here:
+//
+//   q_h <- N(q_h + b) * wq,  k_g <- N(k_g + b) * wk,  the same rotation,  v_g <- v_g + b
+//
+// There no head waits for another: a warp a (token, head), the head in shared memory between norm and rotation.
+//
 // The projection arrives as float32 sums [N][W] (or slices [P][N][W] to be added): q heads, k heads, v heads side by side.
 #include "common.cuh"
 
@@ -93,7 +100,89 @@ qkv_norm_rope_kernel(QkvNormArgs p) {
     vc[((size_t)h * p.page_size + off) * p.vdim + d] = Num<T>::from_f(row[qw + kw + c]);
   }
 }
+
+struct HeadNormArgs {
+  const float* proj; int parts; long long part_stride; int width; const float* bias;      // bias [channels] or null
+  const float* wq; const float* wk; float eps;                                            // [dim] each
+  const float* cos_t; const float* sin_t; int rot_half; int layout;
+  int n_heads, n_kv, dim, vdim, n_tokens;
+  void* q_out; const int* slot_map; void* k_cache; void* v_cache; long long page_stride; int page_size, page_shift;
+};
+
+constexpr int HN_WARPS = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(HN_WARPS * 32)
+head_norm_rope_kernel(HeadNormArgs p) {
+  extern __shared__ float heads_s[];                 // [HN_WARPS][max(dim, vdim)]
+  pdl_enter();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int per_token = p.n_heads + 2 * p.n_kv;
+  const long long item = (long long)blockIdx.x * HN_WARPS + warp;
+  if (item >= (long long)p.n_tokens * per_token) return;         // warps never wait for one another
+  const int t = (int)(item / per_token), h = (int)(item - (long long)t * per_token);
+  const bool is_q = h < p.n_heads, is_v = h >= p.n_heads + p.n_kv;
+  const int size = is_v ? p.vdim : p.dim;
+  const int col = is_v ? (p.n_heads + p.n_kv) * p.dim + (h - p.n_heads - p.n_kv) * p.vdim : h * p.dim;
+  float* row = heads_s + warp * (p.dim > p.vdim ? p.dim : p.vdim);
+  const float* src = p.proj + (size_t)t * p.width + col;
+  float ss = 0.0f;
+  for (int i = lane; i < size; i += 32) {
+    float v = 0.0f;
+    for (int s = 0; s < p.parts; ++s) v += src[(size_t)s * p.part_stride + i];
+    if (p.bias) v += p.bias[col + i];
+    row[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (!is_v) {
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)size + p.eps);
+    const float* w = is_q ? p.wq : p.wk;
+    for (int i = lane; i < size; i += 32) row[i] = row[i] * inv * w[i];
+    __syncwarp();
+    const float* ct = p.cos_t + (size_t)t * p.rot_half;
+    const float* st = p.sin_t + (size_t)t * p.rot_half;
+    for (int j = lane; j < p.rot_half; j += 32) {
+      const int a = p.layout == 0 ? j : 2 * j, b = p.layout == 0 ? j + p.rot_half : 2 * j + 1;
+      const float cs = ct[j], sn = st[j], u = row[a], v = row[b];
+      row[a] = u * cs - v * sn;
+      row[b] = v * cs + u * sn;
+    }
+  }
+  __syncwarp();
+  T* dst;
+  if (is_q) {
+    dst = (T*)p.q_out + ((size_t)t * p.n_heads + h) * p.dim;
+  } else {
+    const int where = p.slot_map ? p.slot_map[t] : -1;
+    if (where < 0) return;
+    const int g = is_v ? h - p.n_heads - p.n_kv : h - p.n_heads;
+    dst = (T*)(is_v ? p.v_cache : p.k_cache) + (size_t)(where >> p.page_shift) * p.page_stride +
+          ((size_t)g * p.page_size + (where & (p.page_size - 1))) * size;
+  }
+  for (int i = lane; i < size; i += 32) dst[i] = Num<T>::from_f(row[i]);
+}
 }  // namespace
+
+// proj float32 [parts][N][width]: q, k and v heads side by side; bias [channels] or null; wq, wk [dim].
+IFX_API int ifx_head_norm_rope_write(const float* proj, int parts, long long part_stride, int width, const float* bias,
+                                     const float* wq, const float* wk, float eps, const float* cos_t, const float* sin_t,
+                                     int rot_half, int layout, int n_heads, int n_kv, int dim, int vdim, void* q_out,
+                                     int dtype, const int* slot_map, void* k_cache, void* v_cache, long long page_stride,
+                                     int page_size, int n_tokens, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (page_size <= 0 || (page_size & (page_size - 1)) || n_heads < 1 || n_kv < 1 || dim < 1 || vdim < 1) return IFX_ERR_UNSUPPORTED;
+  if (rot_half < 0 || 2 * rot_half > dim || !wq || !wk || dim > 1024 || vdim > 1024) return IFX_ERR_UNSUPPORTED;
+  if ((n_heads + n_kv) * dim + n_kv * vdim > width) return IFX_ERR_UNSUPPORTED;
+  if (dtype != IFX_BF16 && dtype != IFX_F32) return IFX_ERR_UNSUPPORTED;
+  HeadNormArgs p{proj, parts, part_stride, width, bias, wq, wk, eps, cos_t, sin_t, rot_half, layout, n_heads, n_kv, dim, vdim,
+                 n_tokens, q_out, slot_map, k_cache, v_cache, page_stride, page_size, 0};
+  while ((1 << p.page_shift) < page_size) ++p.page_shift;
+  const long long items = (long long)n_tokens * (n_heads + 2 * n_kv);
+  const size_t smem = (size_t)HN_WARPS * (dim > vdim ? dim : vdim) * sizeof(float);
+  const int rc = launch_pdl(dtype == IFX_BF16 ? head_norm_rope_kernel<bf16> : head_norm_rope_kernel<float>,
+                            dim3((unsigned)((items + HN_WARPS - 1) / HN_WARPS)), dim3(HN_WARPS * 32), smem, stream, p);
+  return rc ? rc : IFX_LAUNCH_CHECK();
+}
 
 IFX_API int ifx_qkv_norm_rope_write(const float* proj, int parts, long long part_stride, int width, const float* wq,
                                     const float* wk, float eps, const float* cos_t, const float* sin_t, int rot_half,

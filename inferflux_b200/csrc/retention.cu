@@ -1,7 +1,8 @@
 // Retention: linear attention with a fixed decay per head, no softmax and no denominator,
 //
 //   S_t = g S_{t-1} + k_t v_t^T          S: [dim x vdim] per head, float32, in the request's state slot
-//   o_t = S_t^T q_t                      g = the head's decay, k already scaled
+//   o_t = S_t^T q_t                      g = the head's decay, k already scaled; q, k and v through silu on the way in
+//                                        where a design asks for it
 //
 // so o_t = g^(i+1) S_start^T q_t + sum_{j <= i} g^(i-j) (q_t . k_j) v_j for the i-th token of a segment that
 // starts from S_start.  A portion is cut into segments of IFX_RETENTION_SEGMENT tokens that run side by side:
@@ -9,8 +10,8 @@
 //   2. per entry and head the segments' starting states one after the other, S <- g^n S + B; the last one
 //      goes into the slot                                                                 (carry)
 //   3. every segment's outputs from its starting state                                    (outputs)
-// A step whose entries all fit one segment (single tokens, short portions) runs 3 alone: it reads the slot
-// and writes the new state itself.  A block owns a tile of 64 value columns of one (segment, head); the
+// A step whose entries all fit one segment (short portions) runs 3 alone: it reads the slot and writes the new
+// state itself; a step of single tokens has a kernel of its own, which streams the state through registers.  A block owns a tile of 64 value columns of one (segment, head); the
 // state tile, the segment's q, k, v and the decayed scores live in shared memory.  All of it is float32
 // FFMA: the state, what enters it and the scores are 32-bit by the mixer's definition.
 // `finish` divides each head's output by its root mean square, multiplies by silu(gate) and rounds once.
@@ -31,6 +32,7 @@ struct RetStep {
   int heads, dim, vdim;
   const float* decay;                  // [heads]
   float k_scale;
+  int silu;                            // q, k and v are silu(projection)
   const int* seg_entry; const int* seg_t0;
   const int* entry_q_start; const int* entry_q_len; const int* entry_slot;
   float* state;                        // [slots][heads][dim][vdim]
@@ -44,16 +46,21 @@ __device__ __forceinline__ void decay_powers(float* pw, float g, int tid) {
 // 16-byte aligned for the vector paths and neighbouring rows fall into different banks), else dim + 1.
 __host__ __device__ __forceinline__ int key_ld(int dim) { return (dim & 3) ? dim + 1 : dim + 4; }
 
+__device__ __forceinline__ float taken(const RetStep& s, size_t row, int col) {
+  const float x = s.proj[row * s.stride + col];
+  return s.silu ? x / (1.0f + expf(-x)) : x;
+}
+
 // k[j][d] (scaled), v[j][c] for the block's columns
 __device__ __forceinline__ void load_kv(const RetStep& s, int row0, int n, int head, int v0, float* ks, float* vs, int tid) {
   const int D = s.dim, KD = key_ld(D);
   for (int idx = tid; idx < SEG * D; idx += THREADS) {
     const int j = idx / D, d = idx - j * D;
-    ks[j * KD + d] = j < n ? s.proj[(size_t)(row0 + j) * s.stride + s.k_col + head * D + d] * s.k_scale : 0.0f;
+    ks[j * KD + d] = j < n ? taken(s, row0 + j, s.k_col + head * D + d) * s.k_scale : 0.0f;
   }
   for (int idx = tid; idx < SEG * VT; idx += THREADS) {
     const int j = idx / VT, c = idx - j * VT;
-    vs[idx] = (j < n && v0 + c < s.vdim) ? s.proj[(size_t)(row0 + j) * s.stride + s.v_col + head * s.vdim + v0 + c] : 0.0f;
+    vs[idx] = (j < n && v0 + c < s.vdim) ? taken(s, row0 + j, s.v_col + head * s.vdim + v0 + c) : 0.0f;
   }
 }
 
@@ -172,7 +179,7 @@ retention_outputs_kernel(RetStep s, const float* __restrict__ seg_start, float* 
   load_kv(s, row0, n, head, v0, ks, vs, tid);
   for (int idx = tid; idx < SEG * D; idx += THREADS) {
     const int j = idx / D, d = idx - j * D;
-    qs[idx] = j < n ? s.proj[(size_t)(row0 + j) * s.stride + s.q_col + head * D + d] : 0.0f;
+    qs[idx] = j < n ? taken(s, row0 + j, s.q_col + head * D + d) : 0.0f;
   }
   float* slot_tile = s.state + ((size_t)s.entry_slot[e] * s.heads + head) * D * V;
   const float* start = seg_start ? seg_start + ((size_t)seg * s.heads + head) * D * V : slot_tile;
@@ -298,6 +305,49 @@ retention_finish_kernel(const float* __restrict__ o, const float* __restrict__ g
   }
 }
 
+// Single tokens, one per entry: a block a (head, entry, 32 value columns), eight threads a column, NI state rows a thread
+// in registers between the slot's read and its write.
+template <int NI>
+__global__ void __launch_bounds__(256)
+retention_step_kernel(RetStep s, float* __restrict__ out) {
+  __shared__ float ks[8 * NI], qs[8 * NI], red[8][33];
+  pdl_enter();
+  const int head = blockIdx.x, e = blockIdx.y, tid = threadIdx.x, lane = tid & 31, grp = tid >> 5;
+  const int D = s.dim, V = s.vdim, c = blockIdx.z * 32 + lane;
+  const bool on = c < V;
+  const size_t row = s.entry_q_start[e];
+  float* st = s.state + ((size_t)s.entry_slot[e] * s.heads + head) * D * V + (on ? c : 0);
+  float S[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int d = grp + 8 * i;
+    S[i] = (on && d < D) ? st[(size_t)d * V] : 0.0f;
+  }
+  for (int d = tid; d < 8 * NI; d += 256) {
+    ks[d] = d < D ? taken(s, row, s.k_col + head * D + d) * s.k_scale : 0.0f;
+    qs[d] = d < D ? taken(s, row, s.q_col + head * D + d) : 0.0f;
+  }
+  const float v = on ? taken(s, row, s.v_col + head * V + c) : 0.0f;
+  const float g = s.decay[head];
+  __syncthreads();
+  float o = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int d = grp + 8 * i;
+    S[i] = fmaf(g, S[i], ks[d] * v);
+    o = fmaf(qs[d], S[i], o);
+    if (on && d < D) st[(size_t)d * V] = S[i];
+  }
+  red[grp][lane] = o;
+  __syncthreads();
+  if (grp == 0 && on) {
+    o = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) o += red[w][lane];
+    out[(row * s.heads + head) * V + c] = o;
+  }
+}
+
 size_t outputs_smem(int D) {
   return ((size_t)SEG * key_ld(D) + SEG * VT + SEG + 4 + (size_t)SEG * D + (size_t)D * VT + SEG * (SEG + 1)) * sizeof(float);
 }
@@ -305,17 +355,26 @@ size_t outputs_smem(int D) {
 
 IFX_API int ifx_retention_segment() { return SEG; }
 
-// proj: float32 [N][stride] with q, k (rotated) and v at the given columns.  multi = some entry has more than
+// proj: float32 [N][stride] with q, k (rotated) and v at the given columns, through silu first if asked for.  multi = some entry has more than
 // one segment: then seg_b and seg_start ([segments][heads][dim][vdim] float32 each) are used.
 IFX_API int ifx_retention_scan(const float* proj, int stride, int q_col, int k_col, int v_col, int heads, int dim, int vdim,
-                               const float* decay, float k_scale, float* state,
+                               const float* decay, float k_scale, int silu, float* state,
                                const int* seg_entry, const int* seg_t0, int n_segments, const int* entry_first_seg,
                                const int* entry_q_start, const int* entry_q_len, const int* entry_slot, int n_entries,
-                               int multi, float* seg_b, float* seg_start, float* out, cudaStream_t stream) {
-  if (n_segments <= 0) return 0;
+                               int n_rows, int multi, float* seg_b, float* seg_start, float* out, cudaStream_t stream) {
+  if (n_segments <= 0 || n_rows <= 0) return 0;
   if (dim < 1 || dim > 256 || vdim < 1 || heads < 1 || heads > 65535) return IFX_ERR_UNSUPPORTED;
-  RetStep s{proj, stride, q_col, k_col, v_col, heads, dim, vdim, decay, k_scale, seg_entry, seg_t0, entry_q_start,
+  RetStep s{proj, stride, q_col, k_col, v_col, heads, dim, vdim, decay, k_scale, silu, seg_entry, seg_t0, entry_q_start,
             entry_q_len, entry_slot, state};
+  if (n_rows <= n_entries && n_entries <= 65535) {
+    const dim3 grid(heads, n_entries, (vdim + 31) / 32);
+    int rs;
+    if (dim <= 32) rs = launch_pdl(retention_step_kernel<4>, grid, dim3(256), 0, stream, s, out);
+    else if (dim <= 64) rs = launch_pdl(retention_step_kernel<8>, grid, dim3(256), 0, stream, s, out);
+    else if (dim <= 128) rs = launch_pdl(retention_step_kernel<16>, grid, dim3(256), 0, stream, s, out);
+    else rs = launch_pdl(retention_step_kernel<32>, grid, dim3(256), 0, stream, s, out);
+    return rs ? rs : IFX_LAUNCH_CHECK();
+  }
   const int vtiles = (vdim + VT - 1) / VT;
   const size_t smem_c = outputs_smem(dim);
   static bool attr_done = false;

@@ -2,7 +2,9 @@
 //
 //   causal convolution   y_t[c] = act(b[c] + sum_{j < taps} w[c][j] * u_{t - taps + 1 + j}[c]),  u = 0 ahead of a
 //                        sequence's first token; the last taps-1 inputs of every sequence live in its state slot
-//                        ("tail") and are brought up to date by a second kernel after all rows have been read
+//                        ("tail") and are brought up to date by a second kernel after all rows have been read (by the
+//                        same one in a step of single tokens); leading channels may be heads that are made unit
+//                        vectors straight away, y / sqrt(sum(y^2) + eps), the first of them times a factor
 //   scan                 per head h (its B and C from group h / (heads / groups)):
 //                          dt_t = softplus(raw_t[h] + dt_bias[h])          (no clamp)
 //                          S_t  = exp(-exp(A_log[h]) dt_t) S_{t-1} + dt_t B_t x_t^T        S: [state x vdim]
@@ -66,6 +68,53 @@ causal_conv_tail_kernel(ConvArgs p) {
     v[s] = m < keep ? tail[(size_t)m * p.channels + c] : p.in[(size_t)(r0 + m - keep) * p.in_stride + p.col0 + c];
   }
   for (int s = 0; s < keep; ++s) tail[(size_t)s * p.channels + c] = v[s];
+}
+
+// The same for a row whose first unit_heads * unit_dim channels are heads to be made unit vectors: a warp a (row, head) and
+// a warp for every REST other channels.  With `single` every entry brings one token: then the lane that owns a channel
+// is its tail's only reader and moves the tail on itself.
+struct UnitHeads { int heads, dim, scaled; float scale, eps; };
+constexpr int UNIT_MAX = 512;            // channels of a head at most
+constexpr int REST = 128;
+
+__global__ void __launch_bounds__(256)
+causal_conv_heads_kernel(ConvArgs p, UnitHeads unit, int single) {
+  pdl_enter();
+  const int row = blockIdx.x, lane = threadIdx.x & 31;
+  const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const bool head = item < unit.heads;
+  const int c0 = head ? item * unit.dim : unit.heads * unit.dim + (item - unit.heads) * REST;
+  const int size = head ? unit.dim : min(REST, p.channels - c0);
+  if (size <= 0) return;                                 // warps never wait for one another
+  const int e = p.row_entry[row];
+  const int i = row - p.entry_q_start[e];
+  const int keep = p.taps - 1;
+  float* tail = p.tail ? p.tail + (size_t)p.entry_slot[e] * keep * p.channels : nullptr;
+  float y[UNIT_MAX / 32], ss = 0.0f;
+#pragma unroll
+  for (int b = 0; b < UNIT_MAX / 32; ++b) {
+    const int k = lane + 32 * b;
+    y[b] = 0.0f;
+    if (k >= size) continue;
+    const int c = c0 + k;
+    const float* w = p.w + (size_t)c * p.taps;
+    float v = p.bias ? p.bias[c] : 0.0f;
+    for (int j = 0; j < p.taps; ++j) {
+      const int m = i - keep + j;
+      const float u = m >= 0 ? p.in[(size_t)(row - (i - m)) * p.in_stride + p.col0 + c] : tail[(size_t)(keep + m) * p.channels + c];
+      if (single && j > 0) tail[(size_t)(j - 1) * p.channels + c] = u;
+      v = fmaf(w[j], u, v);
+    }
+    if (p.act == 1) v = v / (1.0f + expf(-v));
+    y[b] = v;
+    ss = fmaf(v, v, ss);
+  }
+  float f = 1.0f;
+  if (head) f = (item < unit.scaled ? unit.scale : 1.0f) / sqrtf(warp_sum(ss) + unit.eps);
+  float* dst = p.out + (size_t)row * p.out_stride + c0;
+#pragma unroll
+  for (int b = 0; b < UNIT_MAX / 32; ++b)
+    if (lane + 32 * b < size) dst[lane + 32 * b] = y[b] * f;
 }
 
 struct SsmArgs {
@@ -222,6 +271,28 @@ IFX_API int ifx_causal_conv(const float* in, long long in_stride, int col0, cons
              channels, act};
   int rc = launch_pdl(causal_conv_kernel, dim3(n_rows, (channels + 255) / 256), dim3(256), 0, stream, p);
   if (!rc && taps > 1)
+    rc = launch_pdl(causal_conv_tail_kernel, dim3(n_entries, (channels + 255) / 256), dim3(256), 0, stream, p);
+  return rc ? rc : IFX_LAUNCH_CHECK();
+}
+
+// The same; the first unit_heads * unit_dim channels are heads that become unit vectors (eps inside the root), the first
+// scaled_heads of them times scale.
+IFX_API int ifx_causal_conv_heads(const float* in, long long in_stride, int col0, const float* w, const float* bias, int taps,
+                                  float* tail, const int* row_entry, const int* entry_q_start, const int* entry_q_len,
+                                  const int* entry_slot, int n_rows, int n_entries, float* out, long long out_stride,
+                                  int channels, int act, int unit_heads, int unit_dim, int scaled_heads, float scale, float eps,
+                                  cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (taps < 1 || taps > MAX_TAPS || channels < 1 || (taps > 1 && !tail) || act < 0 || act > 1) return IFX_ERR_UNSUPPORTED;
+  if (unit_heads < 0 || unit_dim < 1 || unit_dim > UNIT_MAX || unit_heads * unit_dim > channels) return IFX_ERR_UNSUPPORTED;
+  ConvArgs p{in, in_stride, col0, w, bias, taps, tail, row_entry, entry_q_start, entry_q_len, entry_slot, out, out_stride,
+             channels, act};
+  const UnitHeads unit{unit_heads, unit_dim, scaled_heads, scale, eps};
+  const int items = unit_heads + (channels - unit_heads * unit_dim + REST - 1) / REST;
+  const int single = n_rows <= n_entries;
+  const int warps = items * n_rows < 148 * 8 ? 2 : 8;
+  int rc = launch_pdl(causal_conv_heads_kernel, dim3(n_rows, (items + warps - 1) / warps), dim3(32 * warps), 0, stream, p, unit, single);
+  if (!rc && taps > 1 && !single)
     rc = launch_pdl(causal_conv_tail_kernel, dim3(n_entries, (channels + 255) / 256), dim3(256), 0, stream, p);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }

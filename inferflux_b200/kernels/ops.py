@@ -154,8 +154,8 @@ def _lib():
         lib.ifx_attn_prefill_bf16_ex.restype = c_int
         lib.ifx_retention_segment.argtypes = []
         lib.ifx_retention_scan.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
-                                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                                           c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
+                                           c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                           c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.ifx_retention_finish.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_ll, c_int, c_int, c_int, c_float,
                                              c_void_p]
         lib.ifx_gelu_tanh.argtypes = [c_void_p, c_int, c_ll, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
@@ -186,7 +186,8 @@ def _lib():
                                                 c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                                 c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p]
         lib.ifx_add_group_rmsnorm.argtypes = [c_void_p, c_void_p, c_int, c_ll, c_float, c_void_p, c_int, c_ll, c_float, c_int,
-                                              c_void_p, c_float, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]
+                                              c_void_p, c_float, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
+                                              c_void_p, c_void_p]
         lib.ifx_glu_clamped.argtypes = [c_void_p, c_int, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float,
                                         c_void_p]
         lib.ifx_gla_scan.argtypes = [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_ll, c_void_p, c_float, c_float, c_void_p,
@@ -194,20 +195,34 @@ def _lib():
                                      c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p]
         lib.ifx_gla_segment.argtypes = []
         lib.ifx_gla_segment.restype = c_int
-        lib.ifx_attn_paged_generic_ex2.argtypes = list(lib.ifx_attn_paged_generic_ex.argtypes[:-1]) + [
-            c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
+        lib.ifx_attn_paged_generic_ex2.argtypes = list(lib.ifx_attn_paged_generic_ex.argtypes[:-2]) + [
+            c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.ifx_attn_latent_paged_ex.argtypes = [c_void_p, c_ll, c_ll, c_void_p, c_ll, c_ll, c_void_p, c_int, c_ll, c_int,
                                                  c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                  c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p]
         lib.ifx_latent_rope_prep.argtypes = [c_void_p, c_ll, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                              c_void_p, c_void_p, c_ll, c_ll, c_void_p, c_int, c_ll, c_int, c_void_p, c_int,
                                              c_void_p]
-        lib.ifx_attn_decode_bf16_ex.argtypes = list(lib.ifx_attn_decode_bf16.argtypes[:-1]) + [c_float, c_int, c_void_p, c_void_p, c_void_p]
+        lib.ifx_attn_decode_bf16_ex.argtypes = list(lib.ifx_attn_decode_bf16.argtypes[:-1]) + [
+            c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
         lib.ifx_attn_decode_bf16_ex.restype = c_int
-        lib.ifx_attn_prefill_bf16_ex2.argtypes = list(lib.ifx_attn_prefill_bf16_ex.argtypes[:-1]) + [c_float, c_int, c_void_p, c_void_p, c_void_p]
+        lib.ifx_attn_prefill_bf16_ex2.argtypes = list(lib.ifx_attn_prefill_bf16_ex.argtypes[:-1]) + [
+            c_int, c_float, c_int, c_void_p, c_void_p, c_void_p]
         lib.ifx_attn_prefill_bf16_ex2.restype = c_int
         lib.ifx_attn_latent_mma_ex.argtypes = list(lib.ifx_attn_latent_mma.argtypes[:-1]) + [c_int, c_int, c_void_p, c_void_p]
         lib.ifx_attn_latent_mma_ex.restype = c_int
+        lib.ifx_head_norm_rope_write.argtypes = [c_void_p, c_int, c_ll, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                                                 c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
+                                                 c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p]
+        lib.ifx_causal_conv_heads.argtypes = list(lib.ifx_causal_conv.argtypes[:-1]) + [c_int, c_int, c_int, c_float, c_float, c_void_p]
+        lib.ifx_gated_delta_segment.argtypes = []
+        lib.ifx_gated_delta_scan.argtypes = [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p,
+                                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+        lib.ifx_softcap.argtypes = [c_void_p, c_ll, c_float, c_void_p]
+        for name in ("ifx_head_norm_rope_write", "ifx_causal_conv_heads", "ifx_gated_delta_segment", "ifx_gated_delta_scan",
+                     "ifx_softcap"):
+            getattr(lib, name).restype = c_int
         for name in ("ifx_add_group_rmsnorm", "ifx_glu_clamped", "ifx_gla_scan", "ifx_attn_paged_generic_ex2",
                      "ifx_attn_latent_paged_ex", "ifx_latent_rope_prep"):
             getattr(lib, name).restype = c_int
@@ -683,12 +698,14 @@ def attn_decode_bf16(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_layer:
                      dec_entries: torch.Tensor, n_dec: int, entry_q_start: torch.Tensor,
                      entry_q_len: torch.Tensor, entry_ctx_start: torch.Tensor, part_o: Optional[torch.Tensor],
                      part_ml: Optional[torch.Tensor], n_heads: int, n_kv: int, head_dim: int, scale: float,
-                     window: int, n_splits: int, q_temp=None, distance_toll=None) -> torch.Tensor:
+                     window: int, n_splits: int, q_temp=None, distance_toll=None, gate: Optional[torch.Tensor] = None,
+                     gate_per_head: bool = False) -> torch.Tensor:
     """Tensor-core attention of single decoded tokens (entries listed in
     dec_entries), the keys split ``n_splits`` ways and merged.  Scratch:
     part_o float32 [n_dec * n_heads * n_splits * head_dim], part_ml float32
-    [n_dec * n_heads * n_splits * 2].  ``q_temp`` and ``distance_toll`` as in
-    :func:`attn_paged_options`."""
+    [n_dec * n_heads * n_splits * 2].  ``window``, ``q_temp``, ``distance_toll``,
+    ``gate`` and ``gate_per_head`` as in :func:`attn_paged_options`."""
+    gp, g_parts, g_pstride, g_stride = _gate_slices(gate, n_heads if gate_per_head else n_heads * head_dim, "attn_decode_bf16")
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
     r1, r2 = distance_toll if distance_toll else (None, None)
     for t in (r1, r2):
@@ -710,7 +727,8 @@ def attn_decode_bf16(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_layer:
                                           _ptr(dec_entries), n_dec, _ptr(entry_q_start), _ptr(entry_q_len),
                                           _ptr(entry_ctx_start), _ptr(part_o), _ptr(part_ml), n_heads, n_kv, head_dim,
                                           float(scale), int(window), int(n_splits), coef, every, _ptr(r1), _ptr(r2),
-                                          _stream()), "attn_decode_bf16")
+                                          gp, g_parts, g_pstride, g_stride, int(bool(gate_per_head)), _stream()),
+           "attn_decode_bf16")
     return out
 
 
@@ -1330,7 +1348,7 @@ def attn_paged_options(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_laye
                        entry_ctx_start: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, scale: float, window: int,
                        v_dim: int, softcap: float = 0.0, keep_first: int = 0, sink: bool = False,
                        gate: Optional[torch.Tensor] = None, single_tokens: bool = False, q_temp=None,
-                       distance_toll=None, sink_value: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       distance_toll=None, sink_value: Optional[torch.Tensor] = None, gate_per_head: bool = False) -> torch.Tensor:
     """With ``single_tokens`` every listed tile is one token (``tile_q0`` = its place in its entry) and the kernel
     for single tokens runs (a block a token and head, its warps sharing the keys out).  Otherwise
     :func:`attn_paged_generic` with values ``v_dim`` wide, a cap on the scores (``softcap * tanh(s / softcap)``,
@@ -1339,7 +1357,9 @@ def attn_paged_options(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_laye
     ``n_heads * v_dim`` columns go through a sigmoid and multiply the result element by element.
     ``q_temp`` = ``(coef, every)``: the query at position p counts ``1 + coef * ln(floor((p + 1) / every) + 1)`` times;
     ``distance_toll`` = ``(r1, r2)``, float32 ``[n_heads]`` each: the score of key j loses ``r1 * ln(1 + r2 * (p - j))``
-    (after the cap); ``sink_value`` float32 ``[n_heads]``: the sink's score per head instead of 0."""
+    (after the cap); ``sink_value`` float32 ``[n_heads]``: the sink's score per head instead of 0; ``gate_per_head``: the
+    gate's first ``n_heads`` columns multiply a head's result as a whole.  ``window``: 0 everything, w > 0 the last w
+    positions, -c < 0 the query's chunk of c positions (chunks counted from position 0)."""
     _need(block_tables.dtype == torch.int32 and block_tables.dim() == 2 and block_tables.stride(1) == 1,
           "attn: block_tables int32 [R, B]")
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
@@ -1347,21 +1367,14 @@ def attn_paged_options(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_laye
     for t in (r1, r2, sink_value):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_heads), "attn: per-head numbers float32 [heads]")
     _need(out.is_contiguous() and out.dtype == q.dtype and k_layer.dtype == q.dtype and out.shape[1] == n_heads * v_dim, "attn: types")
-    gp, g_parts, g_pstride, g_stride = None, 0, 0, 0
-    if gate is not None:
-        _need(gate.dtype == torch.float32 and gate.stride(-1) == 1 and gate.shape[-1] >= n_heads * v_dim, "attn: gate float32 rows")
-        gp = _ptr(gate)
-        if gate.dim() == 3:
-            g_parts, g_pstride, g_stride = gate.shape[0], gate.stride(0), gate.stride(1)
-        else:
-            g_parts, g_pstride, g_stride = 1, 0, gate.stride(0)
+    gp, g_parts, g_pstride, g_stride = _gate_slices(gate, n_heads if gate_per_head else n_heads * v_dim, "attn")
     _check(_lib().ifx_attn_paged_generic_ex2(_ptr(q), q_stride, _ptr(out), out.stride(0), _code(q), _ptr(k_layer),
                                             _ptr(v_layer), page_stride, page_size, _ptr(block_tables),
                                             block_tables.stride(0), _ptr(tile_entry), _ptr(tile_q0), n_tiles,
                                             _ptr(entry_q_start), _ptr(entry_q_len), _ptr(entry_ctx_start),
                                             n_heads, n_kv, head_dim, float(scale), int(window), int(v_dim), float(softcap),
                                             int(keep_first), 1 if sink else 0, gp, g_parts, g_pstride, g_stride,
-                                            1 if single_tokens else 0, coef, every, _ptr(r1), _ptr(r2), _ptr(sink_value),
+                                            int(bool(gate_per_head)), 1 if single_tokens else 0, coef, every, _ptr(r1), _ptr(r2), _ptr(sink_value),
                                             _stream()),
            "attn_paged_options")
     return out
@@ -1381,7 +1394,8 @@ def attn_prefill_options_bf16(q: torch.Tensor, q_stride: int, out: torch.Tensor,
                               tile_q0: torch.Tensor, n_tiles: int, entry_q_start: torch.Tensor, entry_q_len: torch.Tensor,
                               entry_ctx_start: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, scale: float,
                               window: int, softcap: float = 0.0, keep_first: int = 0, sink: bool = False,
-                              gate: Optional[torch.Tensor] = None, q_temp=None, distance_toll=None) -> torch.Tensor:
+                              gate: Optional[torch.Tensor] = None, q_temp=None, distance_toll=None,
+                              gate_per_head: bool = False) -> torch.Tensor:
     """:func:`attn_prefill_bf16` (tensor cores, bfloat16, keys and values both ``head_dim`` = 64 or 128 wide, query
     tiles of 64 tokens) with the options of :func:`attn_paged_options` (all but the sink's own score)."""
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
@@ -1392,13 +1406,14 @@ def attn_prefill_options_bf16(q: torch.Tensor, q_stride: int, out: torch.Tensor,
           "attn_prefill_options_bf16: bfloat16 operands")
     _need(head_dim in FAST_ATTENTION_HEAD_DIMS, f"attn_prefill_options_bf16: head_dim {head_dim} not in {FAST_ATTENTION_HEAD_DIMS}")
     _need(block_tables.dtype == torch.int32 and block_tables.stride(1) == 1, "attn: block_tables int32 [R, B]")
-    gp, g_parts, g_pstride, g_stride = _gate_slices(gate, n_heads * head_dim, "attn_prefill_options_bf16")
+    gp, g_parts, g_pstride, g_stride = _gate_slices(gate, n_heads if gate_per_head else n_heads * head_dim, "attn_prefill_options_bf16")
     _check(_lib().ifx_attn_prefill_bf16_ex2(_ptr(q), q_stride, _ptr(out), out.stride(0), _ptr(k_layer), _ptr(v_layer),
                                            page_stride, page_size, _ptr(block_tables), block_tables.stride(0),
                                            _ptr(tile_entry), _ptr(tile_q0), n_tiles, _ptr(entry_q_start),
                                            _ptr(entry_q_len), _ptr(entry_ctx_start), n_heads, n_kv, head_dim,
                                            float(scale), int(window), float(softcap), int(keep_first), 1 if sink else 0,
-                                           gp, g_parts, g_pstride, g_stride, coef, every, _ptr(r1), _ptr(r2), _stream()),
+                                           gp, g_parts, g_pstride, g_stride, int(bool(gate_per_head)), coef, every, _ptr(r1),
+                                           _ptr(r2), _stream()),
            "attn_prefill_options_bf16")
     return out
 
@@ -1411,9 +1426,9 @@ def retention_segment() -> int:
 def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int, dim: int, vdim: int,
                    decay: torch.Tensor, k_scale: float, state: torch.Tensor, seg_entry: torch.Tensor, seg_t0: torch.Tensor,
                    n_segments: int, entry_first_seg: torch.Tensor, entry_q_start: torch.Tensor, entry_q_len: torch.Tensor,
-                   entry_slot: torch.Tensor, n_entries: int, multi: bool, out: torch.Tensor) -> torch.Tensor:
+                   entry_slot: torch.Tensor, n_entries: int, multi: bool, out: torch.Tensor, silu: bool = False) -> torch.Tensor:
     """``S_t = decay_h S_{t-1} + (k_scale k_t) v_t^T``, ``o_t = S_t^T q_t`` per head over the step's entries, all
-    float32.  ``proj`` float32 ``[N, W]`` holds q, k (already rotated) and v heads from the given columns on;
+    float32; with ``silu`` q, k and v go through it first.  ``proj`` float32 ``[N, W]`` holds q, k (already rotated) and v heads from the given columns on;
     ``state`` float32 ``[slots, heads, dim, vdim]``; ``out`` float32 ``[N, heads * vdim]``."""
     n = proj.shape[0]
     _need(proj.dtype == torch.float32 and proj.dim() == 2 and proj.stride(1) == 1, "retention: float32 projection rows")
@@ -1426,9 +1441,9 @@ def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads
         seg_b = torch.empty((n_segments, heads, dim, vdim), dtype=torch.float32, device=proj.device)
         seg_start = torch.empty_like(seg_b)
     _check(_lib().ifx_retention_scan(_ptr(proj), proj.stride(0), q_col, k_col, v_col, heads, dim, vdim, _ptr(decay),
-                                     float(k_scale), _ptr(state), _ptr(seg_entry), _ptr(seg_t0), n_segments,
+                                     float(k_scale), 1 if silu else 0, _ptr(state), _ptr(seg_entry), _ptr(seg_t0), n_segments,
                                      _ptr(entry_first_seg), _ptr(entry_q_start), _ptr(entry_q_len), _ptr(entry_slot),
-                                     n_entries, 1 if multi else 0, _ptr(seg_b), _ptr(seg_start), _ptr(out), _stream()),
+                                     n_entries, n, 1 if multi else 0, _ptr(seg_b), _ptr(seg_start), _ptr(out), _stream()),
            "retention_scan")
     if multi:
         global launch_count
@@ -1709,8 +1724,10 @@ def qkv_norm_rope_write(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Opti
 
 
 def add_group_rmsnorm(residual: torch.Tensor, a, weight: torch.Tensor, eps: float, groups: int, out: Optional[torch.Tensor],
-                      rows: Optional[torch.Tensor] = None, a_scale: float = 1.0, b=None, b_scale: float = 1.0) -> Optional[torch.Tensor]:
-    """``residual`` (float32 ``[N, H]``) ``+= a_scale * a + b_scale * b``; ``out`` = the sum with each of ``groups``
+                      rows: Optional[torch.Tensor] = None, a_scale: float = 1.0, b=None, b_scale: float = 1.0,
+                      x: Optional[torch.Tensor] = None, vec: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """``residual`` (float32 ``[N, H]``) ``+= a_scale * a + b_scale * b + x + vec`` (``x`` float32 ``[N, H]``, ``vec``
+    float32 ``[H]``); ``out`` = the sum with each of ``groups``
     equal consecutive parts of a row divided by its own root mean square (eps inside the root), times ``weight``.
     ``a`` and ``b`` are None, ``[N, H]`` or slices ``[P, N, H]`` (float32 or bfloat16, both of one type).  With
     ``rows`` (int32) only those rows are normed into ``out [R, H]`` and the residual is left untouched."""
@@ -1732,9 +1749,12 @@ def add_group_rmsnorm(residual: torch.Tensor, a, weight: torch.Tensor, eps: floa
     dd = _code(a if a is not None else b) if (a is not None or b is not None) else F32
     if out is not None:
         _need(out.is_contiguous() and tuple(out.shape) == (n_rows, hidden), "add_group_rmsnorm: out [rows, H]")
+    _need(x is None or (x.dtype == torch.float32 and x.is_contiguous() and tuple(x.shape) == (n, hidden)), "add_group_rmsnorm: x float32 [N, H]")
+    _need(vec is None or (vec.dtype == torch.float32 and vec.is_contiguous() and vec.numel() == hidden), "add_group_rmsnorm: vec float32 [H]")
     _check(_lib().ifx_add_group_rmsnorm(_ptr(residual), pa, na, sa, float(a_scale), pb, nb, sb, float(b_scale), dd, _ptr(weight),
                                         float(eps), int(groups), _ptr(out), _code(out) if out is not None else F32, _ptr(rows),
-                                        n_rows, hidden, 0 if rows is not None else 1, _stream()), "add_group_rmsnorm")
+                                        n_rows, hidden, 0 if rows is not None else 1, _ptr(x), _ptr(vec), _stream()),
+           "add_group_rmsnorm")
     return out
 
 
@@ -1789,3 +1809,103 @@ def gla_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, z: torch.Te
 def gla_segment() -> int:
     """Tokens per segment of the gated linear attention scan."""
     return int(_lib().ifx_gla_segment())
+
+
+# ------------------------------------------------- head-wise norms of q and k, unit heads behind a convolution, gated delta rule
+def head_norm_rope_write(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: torch.Tensor, wk: torch.Tensor, eps: float,
+                         cos: torch.Tensor, sin: torch.Tensor, layout: int, n_heads: int, n_kv: int, dim: int, vdim: int,
+                         q_out: torch.Tensor, slot_map: torch.Tensor, k_layer: torch.Tensor, v_layer: torch.Tensor,
+                         page_stride: int, page_size: int) -> None:
+    """The first ``(n_heads + n_kv) * dim + n_kv * vdim`` columns of the float32 projection ``proj [N, W]`` (or slices
+    ``[P, N, W]``) are q, k and v heads side by side; ``bias`` (float32, a number per column) is added.  Every query
+    (key) head is divided by its own root mean square (eps inside the root), multiplied by ``wq`` (``wk``), float32
+    ``[dim]``, and rotated by ``cos``/``sin`` ``[N, r/2]``.  q goes to ``q_out``, k and v into the paged cache at
+    ``slot_map``."""
+    n = q_out.shape[0]
+    channels = (n_heads + n_kv) * dim + n_kv * vdim
+    width = proj.shape[-1]
+    _need(proj.dtype == torch.float32 and proj.is_contiguous() and width >= channels, "head_norm_rope: float32 projection")
+    parts, pstride = (proj.shape[0], n * width) if proj.dim() == 3 else (1, 0)
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() >= channels), "head_norm_rope: bias float32")
+    _need(all(w.dtype == torch.float32 and w.is_contiguous() and w.numel() == dim for w in (wq, wk)), "head_norm_rope: weights float32 [dim]")
+    _need(cos.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous() and cos.shape == sin.shape
+          and cos.shape[0] == n, "head_norm_rope: cos/sin float32 [N, r/2]")
+    _need(q_out.is_contiguous() and tuple(q_out.shape) == (n, n_heads * dim) and k_layer.dtype == q_out.dtype,
+          "head_norm_rope: q_out [N, heads * dim] of the cache's type")
+    _check(_lib().ifx_head_norm_rope_write(_ptr(proj), parts, pstride, width, _ptr(bias), _ptr(wq), _ptr(wk), float(eps),
+                                           _ptr(cos), _ptr(sin), cos.shape[1], layout, n_heads, n_kv, dim, vdim, _ptr(q_out),
+                                           _code(q_out), _ptr(slot_map), _ptr(k_layer), _ptr(v_layer), page_stride, page_size, n,
+                                           _stream()), "head_norm_rope_write")
+
+
+def causal_conv_heads(x: torch.Tensor, col0: int, channels: int, w: torch.Tensor, bias: Optional[torch.Tensor],
+                      tail: Optional[torch.Tensor], row_entry: torch.Tensor, entry_q_start: torch.Tensor,
+                      entry_q_len: torch.Tensor, entry_slot: torch.Tensor, n_entries: int, out: torch.Tensor, unit_heads: int,
+                      unit_dim: int, scaled_heads: int, scale: float, eps: float, silu: bool = True) -> torch.Tensor:
+    """:func:`causal_conv` whose first ``unit_heads * unit_dim`` channels are heads that become unit vectors behind the
+    activation, ``y / sqrt(sum(y^2) + eps)``, the first ``scaled_heads`` of them times ``scale``."""
+    n, taps = x.shape[0], w.shape[1]
+    _need(x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1 and col0 + channels <= x.shape[1],
+          "causal_conv_heads: float32 rows")
+    _need(w.dtype == torch.float32 and w.is_contiguous() and w.shape[0] == channels, "causal_conv_heads: w float32 [channels, taps]")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == channels), "causal_conv_heads: bias float32 [channels]")
+    _need(out.dtype == torch.float32 and out.stride(1) == 1 and tuple(out.shape) == (n, channels), "causal_conv_heads: out")
+    if taps > 1:
+        _need(tail is not None and tail.dtype == torch.float32 and tail.is_contiguous()
+              and tuple(tail.shape[1:]) == (taps - 1, channels), "causal_conv_heads: tail float32 [slots, taps - 1, channels]")
+    _check(_lib().ifx_causal_conv_heads(_ptr(x), x.stride(0), col0, _ptr(w), _ptr(bias), taps, _ptr(tail) if taps > 1 else None,
+                                        _ptr(row_entry), _ptr(entry_q_start), _ptr(entry_q_len), _ptr(entry_slot), n, n_entries,
+                                        _ptr(out), out.stride(0), channels, 1 if silu else 0, unit_heads, unit_dim, scaled_heads,
+                                        float(scale), float(eps), _stream()), "causal_conv_heads")
+    if taps > 1 and n > n_entries:
+        global launch_count
+        launch_count += 1
+    return out
+
+
+def gated_delta_segment() -> int:
+    """Tokens per segment of :func:`gated_delta_scan`."""
+    return int(_lib().ifx_gated_delta_segment())
+
+
+def gated_delta_scan(qkv: torch.Tensor, q_col: int, k_col: int, v_col: int, raw: torch.Tensor, a_col: int, b_col: int,
+                     a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, entry_q_start: torch.Tensor,
+                     entry_q_len: torch.Tensor, entry_slot: torch.Tensor, n_entries: int, out: torch.Tensor, heads: int,
+                     kv_heads: int, dim: int, vdim: int, seg_entry: torch.Tensor, seg_t0: torch.Tensor,
+                     entry_first_seg: torch.Tensor, n_segments: int) -> torch.Tensor:
+    """The gated delta rule, float32.  Per head (query and key of head ``h // (heads / kv_heads)``): ``g = exp(-exp(a_log)
+    softplus(a + dt_bias))``, ``beta = sigmoid(b)``, ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
+    ``o = S^T q``.  ``qkv`` float32 rows hold the prepared q and k (``kv_heads * dim``) and v (``heads * vdim``) from the
+    given columns; ``raw`` float32 rows hold a and b (``heads`` each); ``state [slots, heads, dim, vdim]``; ``out``
+    float32 ``[N, heads * vdim]``.  The step's entries are cut into segments of :func:`gated_delta_segment` tokens
+    (``n_segments`` 0: every entry brings one token)."""
+    n, dev = qkv.shape[0], qkv.device
+    _need(qkv.dtype == torch.float32 and qkv.stride(1) == 1 and raw.dtype == torch.float32 and raw.stride(1) == 1
+          and raw.shape[0] == n, "gated_delta_scan: float32 rows")
+    _need(all(v.dtype == torch.float32 and v.numel() == heads and v.is_contiguous() for v in (a_log, dt_bias)),
+          "gated_delta_scan: a_log, dt_bias float32 [heads]")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim),
+          "gated_delta_scan: state float32 [slots, heads, dim, vdim]")
+    _need(out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, heads * vdim), "gated_delta_scan: out")
+    _need(n_segments > 0 or n == n_entries, "gated_delta_scan: a step with portions lists its segments")
+    w_rows = u_rows = cum = seg_start = None
+    if n_segments:
+        f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
+        w_rows, u_rows, cum = f32(n, heads * dim), f32(n, heads * vdim), f32(n, heads)
+        seg_start = f32(n_segments, heads, dim, vdim)
+    _check(_lib().ifx_gated_delta_scan(_ptr(qkv), qkv.stride(0), q_col, k_col, v_col, _ptr(raw), raw.stride(0), a_col, b_col,
+                                       _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(entry_q_start), _ptr(entry_q_len),
+                                       _ptr(entry_slot), n_entries, _ptr(seg_entry), _ptr(seg_t0), _ptr(entry_first_seg),
+                                       n_segments, _ptr(w_rows), _ptr(u_rows), _ptr(cum), _ptr(seg_start), _ptr(out), heads,
+                                       kv_heads, dim, vdim, _stream()), "gated_delta_scan")
+    if n_segments:
+        global launch_count
+        launch_count += 2
+    return out
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``x <- cap * tanh(x / cap)`` in place, float32."""
+    _need(x.dtype == torch.float32 and x.is_contiguous() and cap > 0, "softcap: float32, a positive cap")
+    _check(_lib().ifx_softcap(_ptr(x), x.numel(), float(cap), _stream()), "softcap")
+    return x

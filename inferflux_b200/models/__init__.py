@@ -4,3 +4,4 @@ from . import kunonex  # noqa: F401
 from . import pemorax  # noqa: F401
 from . import tekosun  # noqa: F401
 from . import malazen  # noqa: F401
+from . import zetivik  # noqa: F401

@@ -17,7 +17,7 @@ from .window_attention import WindowAttention
 from .retention import Retention
 from .side_by_side import SideBySide
 from .state_space import Mamba2
-from .delta_rule import GeneralDelta
+from .delta_rule import GatedDelta, GeneralDelta
 from .gated_linear_attention import GatedLinearAttention
 
 __all__ = ["Part", "KVNeed", "StateNeed", "RunInfo", "Linear", "RMSNorm", "RotaryHalf",

@@ -32,18 +32,20 @@ class KVNeed:
     """What a mixer keeps per token in pages: one or more streams (keys and
     values for attention; a single latent vector for a mixer that caches
     one), and for how long: ``window`` None = every token is kept, w = only
-    the last w.  Runs whose mixers ask for equal needs share a cache group."""
+    the last w; ``chunk`` c = only those of the newest token's stretch of c
+    positions.  Runs whose mixers ask for equal needs share a cache group."""
 
     streams: Tuple[CacheStream, ...]
     window: Optional[int] = None
     keep_first: int = 0         # with a window: this many first tokens stay visible (and cached) for good
+    chunk: Optional[int] = None # tokens see their own chunk of so many positions only (counted from the sequence's start)
 
     @classmethod
     def keys_and_values(cls, n_kv_heads: int, head_dim: int, window: Optional[int] = None,
-                        value_dim: Optional[int] = None, keep_first: int = 0) -> "KVNeed":
+                        value_dim: Optional[int] = None, keep_first: int = 0, chunk: Optional[int] = None) -> "KVNeed":
         """``n_kv_heads * head_dim`` keys and as many values per token (values ``value_dim`` wide if given)."""
         return cls((CacheStream("k", n_kv_heads, head_dim), CacheStream("v", n_kv_heads, value_dim or head_dim)),
-                   window, keep_first if window else 0)
+                   window, keep_first if window else 0, chunk)
 
     @property
     def elements_per_token(self) -> int:
@@ -85,6 +87,16 @@ class ScaledSum:
 
     def __init__(self, terms):
         self.terms = list(terms)                # [(sums, factor), ...]: two of them
+
+
+class JoinedSum:
+    """A pending result that is joined by rows of its own and one vector for all rows: ``value + rows + vector``, with
+    ``value`` a tensor, :class:`PartialSums`, :class:`ScaledSum` or None, ``rows`` float32 ``[N, H]`` or None and
+    ``vector`` float32 ``[H]`` or None.  What a junction adds to the stream goes on like this, so that the next norm
+    adds everything in one pass."""
+
+    def __init__(self, value, rows: Optional[torch.Tensor], vector: Optional[torch.Tensor]):
+        self.value, self.rows, self.vector = value, rows, vector
 
 
 class NormedDelta:

@@ -142,7 +142,9 @@ class ParallelBlock:
 
 class JunctionBlock:
     """An arrangement that is no layer: the pending delta goes into the stream,
-    then its one part (family ``junction``) rewrites the stream in place."""
+    then its one part (family ``junction``) rewrites the stream in place.  A part
+    that has ``pending(delta, ctx, run)`` only adds to the stream: what it makes
+    of the pending delta goes on to the next norm instead."""
 
     family = "arrangement"
     roles = {"junction": "junction"}
@@ -153,6 +155,8 @@ class JunctionBlock:
         self.junction = parts["junction"]
 
     def forward(self, residual: torch.Tensor, delta, ctx, run: RunInfo):
+        if hasattr(self.junction, "pending"):
+            return self.junction.pending(delta, ctx, run)
         if isinstance(delta, ScaledSum):
             for value, factor in delta.terms:
                 t = value.tensor.sum(0) if isinstance(value, PartialSums) else value

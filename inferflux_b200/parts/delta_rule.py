@@ -13,10 +13,26 @@ and by sigmoid(W_g h), and projected.  r, k, v, the raw removal rates, the gate 
 one stacked product whose sums stay float32; the decay, the removal rate, the unit key, the state and the norm are
 float32 in either engine type.  The inner size of the decay's two-step projection is the stored tensors' own.  The
 state lives in the request's state slot.
+
+``gated_delta``: the gated delta rule.  Per head, with unit query and key (``kv_heads`` of them, shared by
+``heads / kv_heads`` value heads each) and one decay and one rate per head and token,
+
+    (q, k, v) = silu(conv(W_q h, W_k h, W_v h))                      a causal convolution over time on every channel
+    q = q / sqrt(sum(q^2) + 1e-6) * dim^(-1/2),   k = k / sqrt(sum(k^2) + 1e-6)
+    g_t = exp(-exp(A_log) softplus(W_a h_t + dt_bias)),   beta_t = sigmoid(W_b h_t)
+    S <- g_t S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T     S: [dim x vdim], float32, zero at the start
+    o_t = S^T q_t
+
+every head's o is divided by its root mean square, multiplied by a weight ``vdim`` long that the heads share and by
+silu(W_g h), and projected.  All input projections are one stacked product whose sums stay float32, and so does
+everything up to the output projection's input.  The state and the last ``taps - 1`` inputs of the convolutions live in
+the request's state slot, so a prompt may be cut anywhere; a portion is cut into segments whose part that does not
+depend on the state is worked out side by side.
 """
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 from typing import Any, Dict, List
 
 import torch
@@ -26,6 +42,7 @@ from ..kernels import ops
 from ..weights.loader import MATRIX, VECTOR, WeightSpec
 from .base import Part, RunInfo, StateNeed
 from .linear import Linear
+from .state_space import describe_row_entries
 
 DECAY_SCALE = math.exp(-0.5)
 KEY_EPS = 1e-6
@@ -107,3 +124,123 @@ class GeneralDelta(Part):
 
 
 register_part("mixer", "general_delta", GeneralDelta)
+
+
+@dataclass
+class GatedDeltaStep:
+    """The entry of every row, and the step cut into segments for the scan kernels: int32 device tensors; ``n_segments``
+    0 = every entry brings one token."""
+
+    row_entry: torch.Tensor
+    seg_entry: torch.Tensor
+    seg_t0: torch.Tensor
+    entry_first_seg: torch.Tensor
+    n_segments: int
+
+
+class GatedDelta(Part):
+    """params: ``hidden``, ``heads``, ``kv_heads`` (default ``heads``), ``dim``, ``vdim``, ``conv`` (taps), ``eps`` (of the
+    per-head norm), ``q_scale`` (default ``dim^-1/2``), ``key_eps`` (default 1e-6), ``name`` (tensors
+    ``<prefix>.<name>.{q,k,v,a,b,g,o,A_log,dt_bias,norm}`` and ``.{q,k,v}.conv`` ``[channels, taps]``; ``b`` is the rate's
+    projection).  State: ``gated_delta`` float32 ``[heads, dim, vdim]``, ``gated_delta_tail`` float32 ``[taps - 1,
+    channels of q, k and v]``."""
+
+    family = "mixer"
+    describe_key = "gated_delta_segments"
+
+    def __init__(self, params, prefix, dtype, device):
+        super().__init__(params, prefix, dtype, device)
+        p = params
+        self.hidden, self.heads = int(p["hidden"]), int(p["heads"])
+        self.kv_heads = int(p.get("kv_heads") or p["heads"])
+        self.dim, self.vdim, self.taps = int(p["dim"]), int(p["vdim"]), int(p["conv"])
+        self.eps, self.key_eps = float(p["eps"]), float(p.get("key_eps", KEY_EPS))
+        self.q_scale = float(p["q_scale"]) if p.get("q_scale") is not None else float(self.dim) ** -0.5
+        if self.heads % self.kv_heads:
+            raise ValueError(f"gated_delta: heads {self.heads} is not a multiple of kv_heads {self.kv_heads}")
+        if not 1 <= self.dim <= 256:
+            raise ValueError("gated_delta: dim must be within 1..256")
+        if not 1 <= self.taps <= 16:
+            raise ValueError("gated_delta: conv must be within 1..16 taps")
+        self.channels = self._channels(p)
+        self.stacked: Linear = None         # [q; k; v; g; a; b]
+        self.o: Linear = None
+
+    @classmethod
+    def _channels(cls, p) -> int:
+        nk = int(p.get("kv_heads") or p["heads"])
+        return 2 * nk * int(p["dim"]) + int(p["heads"]) * int(p["vdim"])
+
+    @classmethod
+    def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
+        h, nh, d, vd, taps = (int(params[k]) for k in ("hidden", "heads", "dim", "vdim", "conv"))
+        nk = int(params.get("kv_heads") or nh)
+        n = lambda leaf: cls.full_name(prefix, params, leaf)
+        rows = {"q": nk * d, "k": nk * d, "v": nh * vd}
+        return ([WeightSpec(n(x), (r, h), MATRIX) for x, r in rows.items()]
+                + [WeightSpec(n(f"{x}.conv"), (r, taps), VECTOR, std=0.5) for x, r in rows.items()]
+                + [WeightSpec(n("g"), (nh * vd, h), MATRIX), WeightSpec(n("a"), (nh, h), MATRIX), WeightSpec(n("b"), (nh, h), MATRIX),
+                   WeightSpec(n("A_log"), (nh,), VECTOR, std=0.5), WeightSpec(n("dt_bias"), (nh,), VECTOR, std=0.5),
+                   WeightSpec(n("norm"), (vd,), VECTOR, init="one_plus_normal"), WeightSpec(n("o"), (h, nh * vd), MATRIX)])
+
+    @classmethod
+    def state_needs(cls, params: Dict[str, Any]) -> List[StateNeed]:
+        needs = [StateNeed("gated_delta", (int(params["heads"]), int(params["dim"]), int(params["vdim"])), torch.float32)]
+        if int(params["conv"]) > 1:
+            needs.append(StateNeed("gated_delta_tail", (int(params["conv"]) - 1, cls._channels(params)), torch.float32))
+        return needs
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        n = lambda leaf: self.full_name(self.prefix, self.params, leaf)
+        f32 = lambda leaf: tensors.pop(n(leaf)).to(torch.float32).contiguous()
+        mats = [tensors.pop(n(x)) for x in ("q", "k", "v", "g", "a", "b")]
+        if len({m.dtype for m in mats}) > 1:
+            mats = [m.float() for m in mats]
+        self.stacked = Linear(torch.cat(mats, dim=0))
+        del mats
+        self.conv_w = torch.cat([f32(f"{x}.conv") for x in ("q", "k", "v")]).contiguous()
+        self.a_log, self.dt_bias = f32("A_log"), f32("dt_bias")
+        self.norm_w = f32("norm").repeat(self.heads).contiguous()
+        self.o = Linear(tensors.pop(n("o")))
+
+    def describe_step(self, layout, put) -> GatedDeltaStep:
+        rows = describe_row_entries(layout, put)
+        lens = [int(v) for v in layout.q_len[:layout.n_entries]]
+        if all(v == 1 for v in lens):
+            return GatedDeltaStep(rows, put([]), put([]), put([]), 0)
+        seg = ops.gated_delta_segment() if torch.device(self.device).type == "cuda" else 32
+        seg_entry, seg_t0, first = [], [], []
+        for i, v in enumerate(lens):
+            first.append(len(seg_entry))
+            for t0 in range(0, v, seg):
+                seg_entry.append(i), seg_t0.append(t0)
+        return GatedDeltaStep(rows, put(seg_entry), put(seg_t0), put(first), len(seg_entry))
+
+    @property
+    def inner_width(self) -> int:
+        return self.heads * self.vdim
+
+    def inner(self, x: torch.Tensor, ctx, run: RunInfo, position=None, out: torch.Tensor = None) -> torch.Tensor:
+        """The normed, gated heads ``[N, heads * vdim]`` that the output projection takes."""
+        n, dev = x.shape[0], x.device
+        kd, hv, c = self.kv_heads * self.dim, self.heads * self.vdim, self.channels
+        step: GatedDeltaStep = ctx.extras[self.describe_key]
+        proj = self.stacked.forward(x, out_dtype=torch.float32)               # [q | k | v | g | a | b]
+        qkv = torch.empty((n, c), dtype=torch.float32, device=dev)
+        ops.causal_conv_heads(proj, 0, c, self.conv_w, None, run.states["gated_delta_tail"] if self.taps > 1 else None,
+                              step.row_entry, ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, qkv,
+                              2 * self.kv_heads, self.dim, self.kv_heads, self.q_scale, self.key_eps)
+        o = torch.empty((n, hv), dtype=torch.float32, device=dev)
+        ops.gated_delta_scan(qkv, 0, kd, 2 * kd, proj, c + hv, c + hv + self.heads, self.a_log, self.dt_bias,
+                             run.states["gated_delta"], ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, o,
+                             self.heads, self.kv_heads, self.dim, self.vdim, step.seg_entry, step.seg_t0, step.entry_first_seg,
+                             step.n_segments)
+        if out is None:
+            out = torch.empty((n, hv), dtype=x.dtype, device=dev)
+        return ops.head_norm_gate(o, proj[:, c:c + hv], self.norm_w, out, self.heads, self.vdim, self.eps, ops.GATE_SILU)
+
+    def forward(self, x: torch.Tensor, ctx, run: RunInfo, position):
+        return self.o.forward(self.inner(x, ctx, run), allow_partials=True, f32_sums=True, out_dtype=torch.float32)
+
+
+register_part("mixer", "gated_delta", GatedDelta)

@@ -91,7 +91,8 @@ class LinearHead(Part):
     """params: ``vocab``, ``hidden``, ``name``, ``tied_to`` (None, or the full
     name of the embedding table to use instead of a weight of its own),
     ``weight_name`` (the weight's full name where it is not ``<name>.weight``),
-    ``scale`` (a factor on the float32 logits, default 1)."""
+    ``scale`` (a factor on the float32 logits, default 1), ``softcap`` (None, or c: the logits become
+    ``c * tanh(logits / c)``)."""
 
     family = "lm_head"
 
@@ -99,6 +100,7 @@ class LinearHead(Part):
         super().__init__(params, prefix, dtype, device)
         self.vocab, self.hidden = int(params["vocab"]), int(params["hidden"])
         self.scale = float(params.get("scale", 1.0) or 1.0)
+        self.softcap = float(params.get("softcap") or 0.0)
         self.linear: Linear = None
 
     @classmethod
@@ -120,7 +122,9 @@ class LinearHead(Part):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         """x [W, hidden] -> float32 logits [W, vocab]."""
         logits = self.linear.forward(x, out_dtype=torch.float32)
-        return logits if self.scale == 1.0 else logits.mul_(self.scale)
+        if self.scale != 1.0:
+            logits.mul_(self.scale)
+        return ops.softcap(logits, self.softcap) if self.softcap else logits
 
 
 register_part("embedding", "token_embedding", TokenEmbedding)

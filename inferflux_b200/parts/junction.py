@@ -10,6 +10,10 @@ the stream as the embedding left it.  The half of the product that reads x0
 is the same in every pass and is made once per step; the sum is float32.
 
 ``add_embedding``: ``x <- x + x0``, nothing else.
+
+``loop_step``: ``x <- x + x0 + step[t]``, without ``x0`` ahead of the first
+pass.  It rewrites nothing itself: it hands what it adds on with the pending
+sum, and the norm that comes next adds it all.
 """
 from __future__ import annotations
 
@@ -20,7 +24,7 @@ import torch
 from ..config.registry import register_part
 from ..kernels import ops
 from ..weights.loader import MATRIX, VECTOR, WeightSpec
-from .base import Part, RunInfo
+from .base import JoinedSum, Part, RunInfo
 from .linear import Linear
 
 
@@ -72,5 +76,30 @@ class AddEmbedding(Part):
         ops.add_into(residual, ctx.embedding_output, 1)
 
 
+class LoopStep(Part):
+    """What joins the stream ahead of pass ``t`` (the run's parameter ``pass``) over a stretch of layers: the vector
+    ``step[t]`` and, from the second pass on, the stream as the embedding left it.  params: ``hidden``, ``passes``,
+    ``step_name`` (the full name of the tensor ``[passes, hidden]``)."""
+
+    family = "junction"
+
+    def __init__(self, params, prefix, dtype, device):
+        super().__init__(params, prefix, dtype, device)
+        self.hidden, self.passes = int(params["hidden"]), int(params["passes"])
+        self.step: torch.Tensor = None
+
+    @classmethod
+    def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
+        return [WeightSpec(params["step_name"], (int(params["passes"]), int(params["hidden"])), VECTOR, std=0.3)]
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.step = tensors.pop(self.params["step_name"]).to(torch.float32).contiguous()
+
+    def pending(self, delta, ctx, run: RunInfo) -> JoinedSum:
+        t = int(run.params["pass"])
+        return JoinedSum(delta, ctx.embedding_output if t > 0 else None, self.step[t])
+
+
 register_part("junction", "loop_entry", LoopEntry)
+register_part("junction", "loop_step", LoopStep)
 register_part("junction", "add_embedding", AddEmbedding)

@@ -15,12 +15,13 @@ import torch
 from ..config.registry import register_part
 from ..kernels import ops
 from ..weights.loader import VECTOR, WeightSpec
-from .base import BranchMean, NormedDelta, Part, PartialSums, ScaledSum
+from .base import BranchMean, JoinedSum, NormedDelta, Part, PartialSums, ScaledSum
 
 
 class RMSNorm(Part):
     """params: ``hidden``, ``eps``, and the weight's name: ``name`` (weight is ``<prefix>.<name>.weight``) or
-    ``weight_name`` (the leaf itself, ``<prefix>.<weight_name>``).
+    ``weight_name`` (the leaf itself, ``<prefix>.<weight_name>``); ``weight_offset`` (default 0) joins the stored weight
+    at load, in float32 (1 for a weight that is stored around zero).
 
     ``delta`` may also be a :class:`NormedDelta` (a sublayer's result that is normed before it joins the
     stream, itself possibly the mean of two normed branches): both norms and the sum are one kernel."""
@@ -41,10 +42,14 @@ class RMSNorm(Part):
 
     @classmethod
     def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
+        if params.get("weight_offset"):
+            return [WeightSpec(cls._weight_name(prefix, params), (int(params["hidden"]),), VECTOR, std=0.1)]
         return [WeightSpec(cls._weight_name(prefix, params), (int(params["hidden"]),), VECTOR, init="one_plus_normal")]
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.weight = tensors[self._weight_name(self.prefix, self.params)].to(torch.float32).contiguous()
+        if self.params.get("weight_offset"):
+            self.weight = self.weight + float(self.params["weight_offset"])
 
     def forward(self, residual: torch.Tensor, delta, out: Optional[torch.Tensor] = None,
                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -129,8 +134,8 @@ class LayerNorm(Part):
 class GroupRMSNorm(RMSNorm):
     """RMS norm over ``groups`` equal consecutive parts of the row, each divided by its own root mean square, the whole
     multiplied by one weight of the row's length; fused with the sum into the stream like :class:`RMSNorm`.
-    ``delta`` may also be a :class:`ScaledSum` of two branches: the weighted sum, the sum into the stream and the norm
-    are one kernel.  params: those of ``rmsnorm`` and ``groups`` (default 1, which is the plain norm)."""
+    ``delta`` may also be a :class:`ScaledSum` of two branches, or a :class:`JoinedSum`: the weighted sum, what joins it,
+    the sum into the stream and the norm are one kernel.  params: those of ``rmsnorm`` and ``groups`` (default 1, which is the plain norm)."""
 
     family = "norm"
 
@@ -147,16 +152,19 @@ class GroupRMSNorm(RMSNorm):
             out = torch.empty((n_rows, self.hidden), dtype=self.dtype, device=residual.device)
         if isinstance(delta, NormedDelta) or isinstance(delta, BranchMean):
             raise TypeError("group_rmsnorm takes a tensor, partial sums or a weighted sum of two branches")
+        x = vec = None
+        if isinstance(delta, JoinedSum):
+            delta, x, vec = delta.value, delta.rows, delta.vector
         terms = delta.terms if isinstance(delta, ScaledSum) else ([(delta, 1.0)] if delta is not None else [])
         if len(terms) > 2:
             raise ValueError("a weighted sum is built for two branches")
         flat = [((v.tensor if isinstance(v, PartialSums) else v), float(f)) for v, f in terms] + [(None, 1.0)] * (2 - len(terms))
         (a, fa), (b, fb) = flat
-        if rows is not None and (a is not None or b is not None):
+        if rows is not None and any(t is not None for t in (a, b, x, vec)):
             # picked rows leave the stream untouched: the pending sum goes in first
-            ops.add_group_rmsnorm(residual, a, self.weight, self.eps, self.groups, None, None, fa, b, fb)
-            a = b = None
-        return ops.add_group_rmsnorm(residual, a, self.weight, self.eps, self.groups, out, rows, fa, b, fb)
+            ops.add_group_rmsnorm(residual, a, self.weight, self.eps, self.groups, None, None, fa, b, fb, x, vec)
+            a = b = x = vec = None
+        return ops.add_group_rmsnorm(residual, a, self.weight, self.eps, self.groups, out, rows, fa, b, fb, x, vec)
 
 
 register_part("norm", "rmsnorm", RMSNorm)

@@ -5,7 +5,8 @@
 
 with q and k rotated by the layer's position table (first ``rot_dims`` dimensions, pairs in ``half``s or
 ``interleaved``), k then scaled by ``dim^-1/2``; each head's o is brought to unit root mean square (no weight),
-the heads side by side are multiplied by silu(g) and projected.  q, k, v and g are one stacked projection whose
+the heads side by side are multiplied by silu(g) and projected.  Other designs' forms are parameters: q, k and v through
+silu, another factor on k, all heads of a token normed together with a weight over them, sigmoid(g).  q, k, v and g are one stacked projection whose
 sums stay float32; rotation, state, scores and the norm are float32 in either engine type.  The state lives in
 the request's state slot; portions are cut into segments that run side by side (the recurrence is linear in S).
 """
@@ -18,7 +19,7 @@ import torch
 
 from ..config.registry import register_part
 from ..kernels import ops
-from ..weights.loader import MATRIX, WeightSpec
+from ..weights.loader import MATRIX, VECTOR, WeightSpec
 from .base import Part, RunInfo, StateNeed
 from .linear import Linear
 
@@ -36,7 +37,10 @@ class RetentionStep:
 
 class Retention(Part):
     """params: ``hidden``, ``heads``, ``dim``, ``vdim``, ``decay`` (one number per head), ``rot_dims``,
-    ``rot_layout``, ``eps`` (of the per-head norm), ``name`` (tensors ``<prefix>.<name>.{q,k,v,g,o}``).
+    ``rot_layout``, ``activation`` (None or ``silu``: of q, k and v; without rotation), ``k_scale`` (None = ``dim^-1/2``),
+    ``norm`` (``heads``: each by itself, no weight; ``row``: all heads of a token together, times the weight
+    ``<prefix>.<name>.norm`` ``[heads * vdim]``), ``gate`` (``silu`` or ``sigmoid``), ``eps`` (of the norm), ``name`` (tensors
+    ``<prefix>.<name>.{q,k,v,g,o}``).
     State: ``retention`` float32 ``[heads, dim, vdim]``.
     Position: a pair ``(cos, sin)`` of float32 ``[N, rot_dims / 2]`` tensors."""
 
@@ -58,6 +62,15 @@ class Retention(Part):
             raise ValueError(f"rot_dims {self.rot_dims} must be even and at most dim {self.dim}")
         if not 1 <= self.dim <= 256:
             raise ValueError("retention: dim must be within 1..256")
+        self.silu = {None: False, "silu": True}.get(p.get("activation"))
+        if self.silu is None or (self.silu and self.rot_dims):
+            raise ValueError("retention: activation is None or 'silu', and 'silu' is built without rotation")
+        self.k_scale = float(p["k_scale"]) if p.get("k_scale") is not None else float(self.dim) ** -0.5
+        self.norm = p.get("norm") or "heads"
+        self.gate = {"silu": ops.GATE_SILU, "sigmoid": ops.GATE_SIGMOID}.get(p.get("gate") or "silu")
+        if self.norm not in ("heads", "row") or self.gate is None:
+            raise ValueError("retention: norm is 'heads' or 'row', gate 'silu' or 'sigmoid'")
+        self.norm_w: torch.Tensor = None
         self.decay = torch.tensor(decay, dtype=torch.float32, device=device)
         self.qkvg: Linear = None
         self.o: Linear = None
@@ -66,9 +79,12 @@ class Retention(Part):
     def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
         h, nh, d, vd = (int(params[k]) for k in ("hidden", "heads", "dim", "vdim"))
         n = lambda leaf: cls.full_name(prefix, params, leaf)
-        return [WeightSpec(n("q"), (nh * d, h), MATRIX), WeightSpec(n("k"), (nh * d, h), MATRIX),
-                WeightSpec(n("v"), (nh * vd, h), MATRIX), WeightSpec(n("g"), (nh * vd, h), MATRIX),
-                WeightSpec(n("o"), (h, nh * vd), MATRIX)]
+        specs = [WeightSpec(n("q"), (nh * d, h), MATRIX), WeightSpec(n("k"), (nh * d, h), MATRIX),
+                 WeightSpec(n("v"), (nh * vd, h), MATRIX), WeightSpec(n("g"), (nh * vd, h), MATRIX),
+                 WeightSpec(n("o"), (h, nh * vd), MATRIX)]
+        if params.get("norm") == "row":
+            specs.append(WeightSpec(n("norm"), (nh * vd,), VECTOR, init="one_plus_normal"))
+        return specs
 
     @classmethod
     def state_needs(cls, params: Dict[str, Any]) -> List[StateNeed]:
@@ -81,6 +97,8 @@ class Retention(Part):
             mats = [m.float() for m in mats]
         self.qkvg = Linear(torch.cat(mats, dim=0))
         del mats
+        if self.norm == "row":
+            self.norm_w = tensors.pop(n("norm")).to(torch.float32).contiguous()
         self.o = Linear(tensors.pop(n("o")))
 
     def describe_step(self, layout, put) -> RetentionStep:
@@ -108,11 +126,14 @@ class Retention(Part):
                                 "the layer's position encoding gave something else")
             ops.rotate_heads(proj, 0, 2 * self.heads, self.dim, position[0], position[1], self.layout)   # q and k heads
         o = torch.empty((n, hv), dtype=torch.float32, device=x.device)
-        ops.retention_scan(proj, 0, hd, 2 * hd, self.heads, self.dim, self.vdim, self.decay, float(self.dim) ** -0.5,
+        ops.retention_scan(proj, 0, hd, 2 * hd, self.heads, self.dim, self.vdim, self.decay, self.k_scale,
                            run.states["retention"], step.seg_entry, step.seg_t0, step.n_segments, step.entry_first_seg,
-                           ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, step.multi, o)
+                           ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, step.multi, o, silu=self.silu)
         if out is None:
             out = torch.empty((n, hv), dtype=x.dtype, device=x.device)
+        if self.norm == "row" or self.gate != ops.GATE_SILU:
+            heads, width = (1, hv) if self.norm == "row" else (self.heads, self.vdim)
+            return ops.head_norm_gate(o, proj[:, 2 * hd + hv:], self.norm_w, out, heads, width, self.eps, self.gate)
         return ops.retention_finish(o, proj[:, 2 * hd + hv:], out, self.heads, self.vdim, self.eps)
 
     def forward(self, x: torch.Tensor, ctx, run: RunInfo, position):

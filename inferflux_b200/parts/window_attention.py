@@ -4,9 +4,10 @@ decoder designs, each a parameter:
   q, k, v (and a gate g) = one stacked projection of the normed input, float32 sums
   ``conv`` taps          a short causal convolution over time on every channel of q, k and v, straight after
                          the projection: y_t = sum_j w[:, j] u_(t - taps + 1 + j), with u = 0 ahead of the first token
-  ``qk_norm``            all of a token's query columns (heads side by side) are divided by their common root
-                         mean square and multiplied by a weight of that size; the key columns likewise; ahead
-                         of the rotation
+  ``qk_norm``            ``rows``: all of a token's query columns (heads side by side) are divided by their common
+                         root mean square and multiplied by a weight of that size; the key columns likewise.
+                         ``heads``: every query and key head by its own root mean square, with one weight ``dim``
+                         long for all query heads and one for all key heads.  Ahead of the rotation
   ``v_norm``             every value head is divided by its own root mean square (no weight); cached so
   ``v_mix``              ``first``: this layer's (normed) values are kept for the step's later layers;
                          ``blend``: v <- (1 - lambda) v + lambda v_first with the kept values of the same token
@@ -16,10 +17,13 @@ decoder designs, each a parameter:
   scores                 s = (q . k) * scale, then ``softcap`` * tanh(s / softcap) if given
   visibility             key j for the query at p: j <= p and (p - j < window or j < keep_first); no window
                          = all earlier keys.  Kept tokens keep their own positions.
+  ``chunk``              instead of a window: key j for the query at p if floor(j / chunk) = floor(p / chunk), j <= p
   ``sink``               one more term of score 0 and no value in the denominator:
                          p_j = exp(s_j) / (1 + sum exp(s_j))
-  ``gate``               the heads' results times sigmoid(g), element by element, ahead of the output projection
-  ``bias``               q, k, v and the output projection have a bias each, added in the projection
+  ``gate``               ``elements``: the heads' results times sigmoid(g), element by element, ahead of the output
+                         projection; ``heads``: one number a head
+  ``bias``               ``all``: q, k, v and the output projection have a bias each, added in the projection;
+                         ``qkv``: the first three have
   ``q_temp``             {coef, every}: the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
   ``distance_toll``      the score of key j for the query at p loses r1_h * ln(1 + r2_h * (p - j)), with two stored
                          numbers per head (after the cap, if there is one)
@@ -100,8 +104,9 @@ def describe_query_tiles(layout, put) -> QueryTiles:
 class WindowAttention(Part):
     """params: ``hidden``, ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``conv`` (taps, 0 = none), ``rot_dims``,
     ``rot_layout`` (``interleaved`` or ``half``), ``scale`` (None = ``dim^-1/2``), ``softcap`` (None = none),
-    ``window`` (None = all keys), ``keep_first``, ``sink``, ``gate``, ``qk_norm``, ``v_norm``, ``v_mix`` (None,
-    ``first`` or ``blend``), ``eps`` (of these norms), ``bias``, ``q_temp``, ``distance_toll``, ``name``.  Tensors
+    ``window`` (None = all keys), ``keep_first``, ``chunk`` (None = none), ``sink``, ``gate`` (None, ``elements`` = True,
+    ``heads``), ``qk_norm`` (None, ``rows`` = True, ``heads``), ``v_norm``, ``v_mix`` (None, ``first`` or ``blend``), ``eps``
+    (of these norms), ``bias`` (None, ``all`` = True, ``qkv``), ``q_temp``, ``distance_toll``, ``name``.  Tensors
     ``<prefix>.<name>.{q,k,v,g,o}``, ``<prefix>.<name>.{q,k,v,o}.b``, ``<prefix>.<name>.{r1,r2}`` ``[heads]``,
     ``<prefix>.<name>.{q,k,v}.conv`` ``[channels, taps]``, ``<prefix>.<name>.{q,k}.norm`` and ``<prefix>.<name>.vmix``
     (one number; stored but unused in the ``first`` layer).
@@ -126,10 +131,15 @@ class WindowAttention(Part):
         self.softcap = float(p.get("softcap") or 0.0)
         self.window = int(p.get("window") or 0)
         self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
-        self.sink, self.gate = bool(p.get("sink")), bool(p.get("gate"))
-        self.qk_norm, self.v_norm, self.v_mix = bool(p.get("qk_norm")), bool(p.get("v_norm")), p.get("v_mix") or None
+        self.chunk = int(p.get("chunk") or 0)
+        if self.window and self.chunk:
+            raise ValueError("window_attention: a window or chunks, not both")
+        self.reach = -self.chunk if self.chunk else self.window       # how the kernels take either
+        self.sink, self.gate = bool(p.get("sink")), self._option(p, "gate", "elements", ("elements", "heads"))
+        self.qk_norm = self._option(p, "qk_norm", "rows", ("rows", "heads"))
+        self.v_norm, self.v_mix = bool(p.get("v_norm")), p.get("v_mix") or None
         self.eps = float(p.get("eps") or 0.0)
-        self.bias = bool(p.get("bias"))
+        self.bias = self._option(p, "bias", "all", ("all", "qkv"))
         qt = p.get("q_temp") or None
         self.q_temp = (float(qt["coef"]), int(qt["every"])) if qt else None
         if self.q_temp and self.q_temp[1] < 1:
@@ -138,7 +148,9 @@ class WindowAttention(Part):
         self.toll = None
         if self.v_mix not in (None, "first", "blend"):
             raise ValueError(f"v_mix {self.v_mix!r} is not one of None, 'first', 'blend'")
-        self.normed = self.qk_norm or self.v_norm or self.v_mix is not None
+        self.normed = self.qk_norm is not None or self.v_norm or self.v_mix is not None
+        if self.qk_norm == "heads" and (self.v_norm or self.v_mix):
+            raise ValueError("window_attention: norms of single heads and norms or a blend of the values are not built together")
         if self.normed and self.taps:
             raise ValueError("window_attention: the short convolution and the norms of q, k, v are not built together")
         if self.normed and self.eps <= 0.0:
@@ -156,6 +168,15 @@ class WindowAttention(Part):
         self.q_norm_w = self.k_norm_w = self.mix_lambda = None
         self.o: Linear = None
 
+    @staticmethod
+    def _option(p, key: str, of_true: str, known) -> Optional[str]:
+        """A parameter that is off, on (the first form there was) or one of several forms by name."""
+        v = p.get(key)
+        v = of_true if v is True else (v or None)
+        if v is not None and v not in known:
+            raise ValueError(f"window_attention: {key} {v!r} is not one of {known}")
+        return v
+
     @classmethod
     def _channels(cls, p) -> int:
         return (int(p["heads"]) + int(p["kv_heads"])) * int(p["dim"]) + int(p["kv_heads"]) * int(p["vdim"])
@@ -170,15 +191,19 @@ class WindowAttention(Part):
         if taps >= 1:                       # one tap is a weight per channel and no reach back in time
             specs += [WeightSpec(n(f"{x}.conv"), (r, taps), VECTOR, std=0.5) for x, r in rows.items()]
         if params.get("gate"):
-            specs.append(WeightSpec(n("g"), (nh * vd, h), MATRIX))
-        if params.get("qk_norm"):
+            specs.append(WeightSpec(n("g"), (nh if params["gate"] == "heads" else nh * vd, h), MATRIX))
+        if params.get("qk_norm") == "heads":
+            specs += [WeightSpec(n(f"{x}.norm"), (d,), VECTOR, init="one_plus_normal") for x in ("q", "k")]
+        elif params.get("qk_norm"):
             specs += [WeightSpec(n("q.norm"), (nh * d,), VECTOR, init="one_plus_normal"),
                       WeightSpec(n("k.norm"), (nkv * d,), VECTOR, init="one_plus_normal")]
         if params.get("v_mix"):
             specs.append(WeightSpec(n("vmix"), (), VECTOR, std=0.3))
         specs.append(WeightSpec(n("o"), (h, nh * vd), MATRIX))
         if params.get("bias"):
-            specs += [WeightSpec(n(f"{x}.b"), (r,), VECTOR) for x, r in rows.items()] + [WeightSpec(n("o.b"), (h,), VECTOR)]
+            specs += [WeightSpec(n(f"{x}.b"), (r,), VECTOR) for x, r in rows.items()]
+            if params["bias"] != "qkv":
+                specs.append(WeightSpec(n("o.b"), (h,), VECTOR))
         if params.get("distance_toll"):
             specs += [WeightSpec(n("r1"), (nh,), VECTOR, init="abs_normal", std=0.5),
                       WeightSpec(n("r2"), (nh,), VECTOR, init="abs_normal", std=0.5)]
@@ -188,7 +213,8 @@ class WindowAttention(Part):
     def kv_need(cls, params: Dict[str, Any]) -> Optional[KVNeed]:
         window = int(params.get("window") or 0) or None
         return KVNeed.keys_and_values(int(params["kv_heads"]), int(params["dim"]), window,
-                                      value_dim=int(params["vdim"]), keep_first=int(params.get("keep_first") or 0))
+                                      value_dim=int(params["vdim"]), keep_first=int(params.get("keep_first") or 0),
+                                      chunk=int(params.get("chunk") or 0) or None)
 
     @classmethod
     def state_needs(cls, params: Dict[str, Any]) -> List[StateNeed]:
@@ -204,8 +230,10 @@ class WindowAttention(Part):
         bias = None
         if self.bias:
             bias = torch.cat([tensors.pop(n(f"{x}.b")).float() for x in ("q", "k", "v")]
-                             + ([torch.zeros(mats[3].shape[0], device=mats[3].device)] if self.gate else []))
-        self.qkvg = Linear(torch.cat(mats, dim=0), bias)
+                             + ([torch.zeros(mats[3].shape[0], device=mats[3].device)] if self.gate else [])).contiguous()
+        # where heads are normed one by one, the kernel that norms them adds the biases
+        self.head_bias = bias if self.qk_norm == "heads" else None
+        self.qkvg = Linear(torch.cat(mats, dim=0), None if self.qk_norm == "heads" else bias)
         del mats
         if self.distance_toll:
             self.toll = tuple(tensors.pop(n(x)).to(torch.float32).contiguous() for x in ("r1", "r2"))
@@ -216,7 +244,7 @@ class WindowAttention(Part):
             self.k_norm_w = tensors.pop(n("k.norm")).to(torch.float32).contiguous()
         if self.v_mix:
             self.mix_lambda = tensors.pop(n("vmix")).to(torch.float32).reshape(1).contiguous()
-        self.o = Linear(tensors.pop(n("o")), tensors.pop(n("o.b")) if self.bias else None)
+        self.o = Linear(tensors.pop(n("o")), tensors.pop(n("o.b")) if self.bias == "all" else None)
 
     def describe_step(self, layout, put) -> QueryTiles:
         return describe_query_tiles(layout, put)
@@ -241,7 +269,11 @@ class WindowAttention(Part):
         k_layer, v_layer = views["k"], views["v"]
         proj = self.qkvg.forward(x, out_dtype=torch.float32)            # float32 sums: they go on into the convolution and the rotation
         q = torch.empty((n, self.heads * self.dim), dtype=x.dtype, device=x.device)
-        if self.normed:
+        if self.qk_norm == "heads":
+            ops.head_norm_rope_write(proj, self.head_bias, self.q_norm_w, self.k_norm_w, self.eps, cos, sin, self.layout, self.heads,
+                                     self.kv_heads, self.dim, self.vdim, q, ctx.slot_maps[g], k_layer, v_layer, page_stride,
+                                     ctx.page_size)
+        elif self.normed:
             mode, v_first = ops.MIX_NONE, None
             if self.v_mix == "first":
                 mode = ops.MIX_STORE
@@ -263,16 +295,16 @@ class WindowAttention(Part):
             out = torch.empty((n, self.heads * self.vdim), dtype=x.dtype, device=x.device)
         gate = proj[:, self._channels(self.params):] if self.gate else None
         common = (ctx.entry_q_start, ctx.entry_q_len, ctx.entry_ctx_start, self.heads, self.kv_heads, self.dim, self.scale,
-                  self.window)
+                  self.reach)
         rest = (self.vdim, self.softcap, self.keep_first, self.sink, gate)
-        more = dict(q_temp=self.q_temp, distance_toll=self.toll)
+        more = dict(q_temp=self.q_temp, distance_toll=self.toll, gate_per_head=self.gate == "heads")
         pages = (k_layer, v_layer, page_stride, ctx.page_size, ctx.block_tables[g])
         fast = (self.TENSOR_CORES and x.dtype == torch.bfloat16 and self.dim == self.vdim and out.is_contiguous()
                 and self.dim in ops.FAST_ATTENTION_HEAD_DIMS)
         singles = (step.single_entry, step.single_q0, step.n_single)
-        if fast and step.n_dec and not (self.softcap or self.keep_first or self.sink or self.gate):
+        if fast and step.n_dec and not (self.softcap or self.keep_first or self.sink):
             # entries of one token: the split tensor-core kernel, which reads a key once for all the heads that share it
-            max_keys = min(ctx.max_ctx_len, self.window) if self.window else ctx.max_ctx_len
+            max_keys = min(ctx.max_ctx_len, abs(self.reach)) if self.reach else ctx.max_ctx_len
             n_splits = ops.attn_decode_splits(step.n_dec, self.heads, self.kv_heads, self.dim, max_keys)
             part_o = part_ml = None
             if n_splits > 1:
@@ -280,7 +312,7 @@ class WindowAttention(Part):
                 part_ml = torch.empty(step.n_dec * self.heads * n_splits * 2, dtype=torch.float32, device=x.device)
             ops.attn_decode_bf16(q, q.stride(0), out, *pages, step.dec_entry, step.n_dec, ctx.entry_q_start, ctx.entry_q_len,
                                  ctx.entry_ctx_start, part_o, part_ml, self.heads, self.kv_heads, self.dim, self.scale,
-                                 self.window, n_splits, **more)
+                                 self.reach, n_splits, gate=gate, **more)
             singles = (step.short_entry, step.short_q0, step.n_short)
         if singles[2]:          # decoded tokens and the shortest portions: a block a token and head
             ops.attn_paged_options(q, q.stride(0), out, *pages, *singles, *common, *rest, single_tokens=True, **more)
