@@ -446,3 +446,102 @@ def make_malazen_folder(cfg: dict, seed: int, folder: Optional[str] = None, **kw
         json.dump(cfg, f)
     write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
     return folder
+
+
+def _zt_left(heads, dim, kv_heads=None, vdim=None, scale=None, chunk=None, rot=None):
+    m = dict(heads=heads, dim=dim)
+    for k, v in (("kv_heads", kv_heads), ("vdim", vdim), ("scale", scale), ("rot", rot)):
+        if v is not None:
+            m[k] = v
+    if chunk is not None:
+        m["mask"] = dict(size=chunk)
+    return m
+
+
+def _zt_right(heads, dim, conv, kv_heads=None, vdim=None):
+    m = dict(heads=heads, dim=dim, conv=conv)
+    for k, v in (("kv_heads", kv_heads), ("vdim", vdim)):
+        if v is not None:
+            m[k] = v
+    return m
+
+
+def _zt_parallel(left, right, mlp, left_scale=None, right_scale=None):
+    mixer = dict(left=left, right=right)
+    if left_scale is not None:
+        mixer.update(left_scale=left_scale, right_scale=right_scale)
+    return dict(type="parallel", mixer=mixer, mlp=mlp)
+
+
+def _zt_lightning(dim, decay, vdim=None, mlp=None):
+    m = dict(heads=len(decay), dim=dim, decay=list(decay))
+    if vdim is not None:
+        m["vdim"] = vdim
+    return dict(type="lightning", mixer=m, mlp=mlp)
+
+
+# Tiny Zetivik configurations that differ in every size, option and order of layers.  A: key, value and state sizes all
+# different, key/value heads shared in both branches, chunks of 20, a partly rotated head, a loop from layer 0 that runs
+# three times, layers without feed-forward, capped logits.
+ZT_A = dict(architecture="Zetivik", width=64, vocab=300, norm=dict(eps=1e-5), logit_softcap=9.0, layers=[
+    _zt_parallel(_zt_left(4, 16, kv_heads=2, vdim=24, scale=0.3, chunk=20, rot=dict(dims=12, base=1000.0)),
+                 _zt_right(4, 12, 4, kv_heads=2, vdim=20), _ML_FF(96, 2.0), 0.8, 1.3),
+    _zt_lightning(12, (0.999, 0.5, 0.9), vdim=20),
+    _zt_parallel(_zt_left(2, 32, kv_heads=1, scale=0.2, chunk=33, rot=dict(dims=32, base=500.0)),
+                 _zt_right(1, 16, 3, vdim=8), None, 1.5, 0.5)], loop=dict(start=0, stop=2, times=3))
+# B: sizes that are no multiple of 4 or 8 anywhere, chunks shorter than a page and none, no rotation in one layer, one tap
+# and two, as many key/value heads as heads, factors left out, a lightning layer with a feed-forward first, no loop, no cap
+ZT_B = dict(architecture="Zetivik", width=50, vocab=77, norm=dict(eps=3e-6), layers=[
+    _zt_lightning(6, (1.0, 0.7, 0.0, 0.95, 0.3), vdim=10, mlp=_ML_FF(35, 0.7)),
+    _zt_parallel(_zt_left(3, 10, vdim=6, chunk=7), _zt_right(2, 6, 1, vdim=10), _ML_FF(45, 3.0)),
+    _zt_parallel(_zt_left(5, 6, kv_heads=1, vdim=10, scale=0.5, rot=dict(dims=2, base=50.0)), _zt_right(6, 10, 2, kv_heads=3, vdim=6),
+                 _ML_FF(18, 1.2), 1.0, 2.0)])
+# C: heads of 64 (the size tensor-core kernels take), chunks longer than several pages, five taps, states of 64 x 64, a
+# loop over the last layer, a lightning layer between
+ZT_C = dict(architecture="Zetivik", width=128, vocab=200, norm=dict(eps=1e-6), logit_softcap=30.0, layers=[
+    _zt_parallel(_zt_left(4, 64, kv_heads=2, scale=0.125, chunk=70, rot=dict(dims=64, base=200000.0)), _zt_right(2, 64, 5), _ML_FF(160, 1.5), 1.1, 0.7),
+    _zt_lightning(64, (0.99, 0.8), mlp=_ML_FF(96, 2.5)),
+    _zt_parallel(_zt_left(2, 64, scale=0.1, chunk=48, rot=dict(dims=8, base=1e4)), _zt_right(4, 32, 4, kv_heads=2, vdim=48), _ML_FF(64, 1.0))],
+    loop=dict(start=2, stop=3, times=2))
+ZT = {"A": ZT_A, "B": ZT_B, "C": ZT_C}
+
+
+def zetivik_tensors(cfg: dict, seed: int, sharpen: float = 4.0):
+    """Random tensors (bfloat16 matrices) for a Zetivik configuration.  ``sharpen`` multiplies the normed heads' weights,
+    so that the softmax is peaked on single keys wherever they lie in the chunk (a lost key would hide below the
+    bfloat16 tolerance otherwise); the projections are enlarged so that every branch carries weight in the sums, and
+    the decays' sizes are set so that a state lost many tokens back would show."""
+    from inferflux_b200.config import load_config
+    from inferflux_b200.config.registry import build_spec
+    from inferflux_b200.engine.model import Model
+    from inferflux_b200.weights.random_init import random_tensors
+    config = load_config(json.loads(json.dumps(cfg)))
+    specs = Model(build_spec(config), torch.float32, "cpu").weight_specs()
+    tensors = random_tensors(specs, seed, torch.bfloat16, None, "cpu")
+    for name in tensors:
+        f, add = 1.0, 0.0
+        if name.endswith((".q.norm", ".k.norm")):
+            f = sharpen ** 0.5
+        elif name.endswith((".q", ".k", ".v", ".g", ".o", ".up", ".down", ".gate", ".right.a", ".right.b")):
+            f = 5.0
+        elif name.endswith((".q.b", ".k.b", ".v.b")):
+            f = 10.0
+        elif name.endswith(".A_log"):
+            add = -2.0
+        elif name.endswith(".conv"):
+            add = 0.3
+        elif name == "embed":
+            f = 20.0
+        if f != 1.0 or add:
+            tensors[name] = (tensors[name].float() * f + add).to(tensors[name].dtype)
+    return config, tensors
+
+
+def make_zetivik_folder(cfg: dict, seed: int, folder: Optional[str] = None, **kw) -> str:
+    from inferflux_b200.weights.safetensors_io import write_safetensors
+    folder = folder or tempfile.mkdtemp(prefix="ifx_zt_")
+    config, tensors = zetivik_tensors(cfg, seed, **kw)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
+    return folder
