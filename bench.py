@@ -240,11 +240,32 @@ def malazen_config(size: str, layers: int):
                 layers=[pair if i % 2 == 0 else latent for i in range(layers)])
 
 
+def zetivik_config(size: str, layers: int):
+    """A Zetivik config.json at the widths of one of the family sizes above: layers in turn a pair of mixers side by side
+    (attention with the family's heads and kv heads of 128 in chunks of 8,192, beside the gated delta rule with half as many
+    value heads of 128 x 128, two to a query and key head, four taps) and lightning attention (the family's heads of
+    128 x 128); every layer with a clamped gated feed-forward of the family's width; capped logits; no loop."""
+    _, hidden, heads, kv_heads, inter, vocab, _ = SIZES[size]
+    ff = dict(kind="dense", ff=inter, limit=7.0)
+    left = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=8192), rot=dict(dims=128, base=500000.0))
+    right = dict(heads=heads // 2, kv_heads=heads // 4, dim=128, vdim=128, conv=4)
+    pair = dict(type="parallel", mixer=dict(left=left, right=right, left_scale=1.0, right_scale=1.0), mlp=ff)
+    lightning = dict(type="lightning", mlp=ff, mixer=dict(heads=heads, dim=128, vdim=128,
+                                                          decay=[1.0 - 0.2 * 0.5 ** (8.0 * i / heads) for i in range(heads)]))
+    return dict(architecture="Zetivik", width=hidden, vocab=vocab, norm=dict(eps=1e-6), logit_softcap=30.0,
+                layers=[pair if i % 2 == 0 else lightning for i in range(layers)])
+
+
+#: --arch: the design's config.json at a size, and the design it is timed beside (the closest one that was there)
+DESIGNS = {"kunonex": (kunonex_config, "qwen2"), "pemorax": (pemorax_config, "qwen2"), "tekosun": (tekosun_config, "pemorax"),
+           "malazen": (malazen_config, "pemorax"), "zetivik": (zetivik_config, "malazen")}
+
+
 def architecture_workload(args) -> int:
-    """--arch kunonex / pemorax / tekosun / malazen: prefill (one 2,048-token prompt) and decode (batch 8 at the given context)
-    of a model of that design beside a model of the same width, layer count and vocabulary (Qwen2 with the same
-    feed-forward width; for tekosun and malazen the closest design, Pemorax), both with random bfloat16 weights, device-timed
-    with CUDA events after warm-up.  One JSON line."""
+    """--arch: prefill (one 2,048-token prompt) and decode (batch 8 at the given context) of a model of that design beside
+    a model of the same width, layer count and vocabulary (the closest design that was there before it, or Qwen2 with the
+    same feed-forward width), both with random bfloat16 weights, device-timed with CUDA events after warm-up.  One JSON
+    line."""
     import torch
     from inferflux_b200 import Engine, SamplingParams, StepEntry
     layers = args.layers or 8
@@ -252,9 +273,8 @@ def architecture_workload(args) -> int:
     warmup = max(3, args.warmup)
     greedy = SamplingParams(temperature=0.0, max_tokens=1 << 30, ignore_eos=True)
     arch = args.arch
-    design = {"kunonex": kunonex_config, "pemorax": pemorax_config, "tekosun": tekosun_config, "malazen": malazen_config}[arch]
-    beside = "pemorax" if arch in ("tekosun", "malazen") else "qwen2"
-    beside_cfg = pemorax_config(args.size, layers) if beside == "pemorax" else dict(family_config(args.size), num_hidden_layers=layers)
+    design, beside = DESIGNS[arch]
+    beside_cfg = dict(family_config(args.size), num_hidden_layers=layers) if beside == "qwen2" else DESIGNS[beside][0](args.size, layers)
     out = {"metric": f"prefill and decode tokens/s, {arch.capitalize()} beside {beside.capitalize()} at the {args.size.upper()} widths", "impl": "ours",
            "n_gpus": 1, "dtype": "bf16", "data": "synthetic: seeded random weights, uniform random token ids",
            "steps": args.steps, "warmup": warmup,
@@ -327,12 +347,12 @@ def main() -> int:
     ap.add_argument("--mixed", type=int, default=0, metavar="N",
                     help="instead of the decode step: N requests with prompts of 128 to 2,048 tokens and 256 output "
                          "tokens each through Engine.generate (chunked prompts beside decoding requests)")
-    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "kunonex", "pemorax", "tekosun", "malazen"],
-                    help="kunonex, pemorax, tekosun or malazen: instead of the default workload, a model of that design beside a "
-                         "model of equal size (Qwen2; for tekosun and malazen, Pemorax) (--size, --layers, default 8), prefill and decode")
+    ap.add_argument("--arch", default="qwen2", choices=["qwen2", *DESIGNS],
+                    help="another design than qwen2: instead of the default workload, a model of that design beside a model of "
+                         "equal size of the closest design before it (--size, --layers, default 8), prefill and decode")
     args = ap.parse_args()
 
-    if args.arch in ("kunonex", "pemorax", "tekosun", "malazen") and args.impl == "ours":
+    if args.arch in DESIGNS and args.impl == "ours":
         return architecture_workload(args)
     if args.impl == "reference":
         return reference_arm()

@@ -111,6 +111,65 @@ struct HeadNormArgs {
 
 constexpr int HN_WARPS = 8;
 
+// Heads of exactly 128 whose rotated pairs lie in halves of a multiple of 4 dimensions: a lane holds four neighbours in
+// registers and gets their partners from the lane rot_half / 4 further or back.
+template <typename T>
+__global__ void __launch_bounds__(HN_WARPS * 32)
+head_norm_rope128_kernel(HeadNormArgs p) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int per_token = p.n_heads + 2 * p.n_kv;
+  const long long item = (long long)blockIdx.x * HN_WARPS + warp;
+  if (item >= (long long)p.n_tokens * per_token) return;         // warps never wait for one another
+  const int t = (int)(item / per_token), h = (int)(item - (long long)t * per_token);
+  const bool is_q = h < p.n_heads, is_v = h >= p.n_heads + p.n_kv;
+  const int col = h * 128 + 4 * lane;
+  float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  for (int s = 0; s < p.parts; ++s) {
+    const float4 x = *reinterpret_cast<const float4*>(p.proj + (size_t)s * p.part_stride + (size_t)t * p.width + col);
+    v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
+  }
+  if (p.bias) {
+    const float4 b = *reinterpret_cast<const float4*>(p.bias + col);
+    v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+  }
+  if (!is_v) {                                                   // warp-uniform
+    const float ss = warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))));
+    const float inv = 1.0f / sqrtf(ss / 128.0f + p.eps);
+    const float4 w = *reinterpret_cast<const float4*>((is_q ? p.wq : p.wk) + 4 * lane);
+    v.x = v.x * inv * w.x; v.y = v.y * inv * w.y; v.z = v.z * inv * w.z; v.w = v.w * inv * w.w;
+    const int step = p.rot_half >> 2;                            // lanes between the two of a pair
+    const bool turns = lane < 2 * step, lower = lane < step;
+    const int other = turns ? (lower ? lane + step : lane - step) : lane;
+    const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, other), __shfl_sync(0xffffffffu, v.y, other),
+                                 __shfl_sync(0xffffffffu, v.z, other), __shfl_sync(0xffffffffu, v.w, other));
+    if (turns) {
+      const size_t at = (size_t)t * p.rot_half + 4 * (lower ? lane : lane - step);
+      const float4 cs = *reinterpret_cast<const float4*>(p.cos_t + at);
+      float4 sn = *reinterpret_cast<const float4*>(p.sin_t + at);
+      if (lower) sn = make_float4(-sn.x, -sn.y, -sn.z, -sn.w);
+      v.x = v.x * cs.x + o.x * sn.x; v.y = v.y * cs.y + o.y * sn.y;
+      v.z = v.z * cs.z + o.z * sn.z; v.w = v.w * cs.w + o.w * sn.w;
+    }
+  }
+  T* dst;
+  if (is_q) {
+    dst = (T*)p.q_out + ((size_t)t * p.n_heads + h) * 128;
+  } else {
+    const int where = p.slot_map ? p.slot_map[t] : -1;
+    if (where < 0) return;
+    const int g = is_v ? h - p.n_heads - p.n_kv : h - p.n_heads;
+    dst = (T*)(is_v ? p.v_cache : p.k_cache) + (size_t)(where >> p.page_shift) * p.page_stride +
+          ((size_t)g * p.page_size + (where & (p.page_size - 1))) * 128;
+  }
+  if (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(dst + 4 * lane) = v;
+  } else {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(dst + 4 * lane) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(HN_WARPS * 32)
 head_norm_rope_kernel(HeadNormArgs p) {
@@ -178,6 +237,13 @@ IFX_API int ifx_head_norm_rope_write(const float* proj, int parts, long long par
                  n_tokens, q_out, slot_map, k_cache, v_cache, page_stride, page_size, 0};
   while ((1 << p.page_shift) < page_size) ++p.page_shift;
   const long long items = (long long)n_tokens * (n_heads + 2 * n_kv);
+  if (dim == 128 && vdim == 128 && layout == 0 && !(rot_half & 3) && !((width | part_stride | page_stride) & 3) &&
+      !(((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)wq | (uintptr_t)wk | (uintptr_t)cos_t | (uintptr_t)sin_t | (uintptr_t)q_out |
+         (uintptr_t)k_cache | (uintptr_t)v_cache) & 15)) {
+    const int r = launch_pdl(dtype == IFX_BF16 ? head_norm_rope128_kernel<bf16> : head_norm_rope128_kernel<float>,
+                             dim3((unsigned)((items + HN_WARPS - 1) / HN_WARPS)), dim3(HN_WARPS * 32), 0, stream, p);
+    return r ? r : IFX_LAUNCH_CHECK();
+  }
   const size_t smem = (size_t)HN_WARPS * (dim > vdim ? dim : vdim) * sizeof(float);
   const int rc = launch_pdl(dtype == IFX_BF16 ? head_norm_rope_kernel<bf16> : head_norm_rope_kernel<float>,
                             dim3((unsigned)((items + HN_WARPS - 1) / HN_WARPS)), dim3(HN_WARPS * 32), smem, stream, p);

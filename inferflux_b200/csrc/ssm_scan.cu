@@ -117,6 +117,68 @@ causal_conv_heads_kernel(ConvArgs p, UnitHeads unit, int single) {
     if (lane + 32 * b < size) dst[lane + 32 * b] = y[b] * f;
 }
 
+// The same for steps with portions, up to four taps and channels in fours: a lane takes four neighbouring channels of
+// ROWS rows one after the other, with the weights and the last TAPS - 1 inputs in registers, so an input is read once.
+constexpr int ROWS = 8;
+
+template <int TAPS>
+__global__ void __launch_bounds__(256)
+causal_conv_heads_rows_kernel(ConvArgs p, UnitHeads unit, int n_rows) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31;
+  const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const bool head = item < unit.heads;
+  const int c0 = head ? item * unit.dim : unit.heads * unit.dim + (item - unit.heads) * REST;
+  const int size = head ? unit.dim : min(REST, p.channels - c0);
+  if (size <= 0) return;                                 // warps never wait for one another
+  const bool on = 4 * lane < size;
+  const int c = on ? c0 + 4 * lane : c0;                 // lanes behind the item's end compute along and store nothing
+  constexpr int KEEP = TAPS - 1;
+  float4 w[TAPS];
+  {
+    float raw[4 * TAPS];                                 // four channels' taps lie side by side
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) *reinterpret_cast<float4*>(raw + 4 * i) = *reinterpret_cast<const float4*>(p.w + (size_t)c * TAPS + 4 * i);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = make_float4(raw[j], raw[TAPS + j], raw[2 * TAPS + j], raw[3 * TAPS + j]);
+  }
+  const float4 bias = p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  const float factor = item < unit.scaled ? unit.scale : 1.0f;
+  float4 u[TAPS];                                        // u[j]: the input TAPS - 1 - j tokens back
+  const int first = blockIdx.x * ROWS, last = min(first + ROWS, n_rows);
+  for (int row = first; row < last; ++row) {
+    const int e = p.row_entry[row], i = row - p.entry_q_start[e];
+    if (row == first || i == 0) {                        // the inputs before this row, from the step or from the slot
+      const float* tail = p.tail + (size_t)p.entry_slot[e] * KEEP * p.channels;
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) {
+        const int m = i - KEEP + j;
+        u[j + 1] = *reinterpret_cast<const float4*>(m >= 0 ? p.in + (size_t)(row - (i - m)) * p.in_stride + p.col0 + c
+                                                           : tail + (size_t)(KEEP + m) * p.channels + c);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) u[j] = u[j + 1];
+    u[KEEP] = *reinterpret_cast<const float4*>(p.in + (size_t)row * p.in_stride + p.col0 + c);
+    float4 y = bias;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      y.x = fmaf(w[j].x, u[j].x, y.x); y.y = fmaf(w[j].y, u[j].y, y.y);
+      y.z = fmaf(w[j].z, u[j].z, y.z); y.w = fmaf(w[j].w, u[j].w, y.w);
+    }
+    if (p.act == 1) {
+      y.x = y.x / (1.0f + expf(-y.x)); y.y = y.y / (1.0f + expf(-y.y));
+      y.z = y.z / (1.0f + expf(-y.z)); y.w = y.w / (1.0f + expf(-y.w));
+    }
+    if (head) {
+      const float ss = on ? fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w))) : 0.0f;
+      const float f = factor / sqrtf(warp_sum(ss) + unit.eps);
+      y.x *= f; y.y *= f; y.z *= f; y.w *= f;
+    }
+    if (on) *reinterpret_cast<float4*>(p.out + (size_t)row * p.out_stride + c) = y;
+  }
+}
+
 struct SsmArgs {
   const float* xbc; long long xbc_stride; int x_col, b_col, c_col;     // convolved x, B, C rows
   const float* dt; long long dt_stride;                                // raw dt, [row][head]
@@ -291,7 +353,17 @@ IFX_API int ifx_causal_conv_heads(const float* in, long long in_stride, int col0
   const int items = unit_heads + (channels - unit_heads * unit_dim + REST - 1) / REST;
   const int single = n_rows <= n_entries;
   const int warps = items * n_rows < 148 * 8 ? 2 : 8;
-  int rc = launch_pdl(causal_conv_heads_kernel, dim3(n_rows, (items + warps - 1) / warps), dim3(32 * warps), 0, stream, p, unit, single);
+  const bool rows = !single && taps >= 2 && taps <= 4 && unit_dim <= 128 && !((unit_dim | channels | col0) & 3) &&
+                    !((in_stride | out_stride) & 3) &&
+                    !(((uintptr_t)in | (uintptr_t)w | (uintptr_t)bias | (uintptr_t)tail | (uintptr_t)out) & 15);
+  int rc;
+  if (rows) {
+    const dim3 grid((n_rows + ROWS - 1) / ROWS, (items + 7) / 8);
+    rc = taps == 4 ? launch_pdl(causal_conv_heads_rows_kernel<4>, grid, dim3(256), 0, stream, p, unit, n_rows)
+       : taps == 3 ? launch_pdl(causal_conv_heads_rows_kernel<3>, grid, dim3(256), 0, stream, p, unit, n_rows)
+                   : launch_pdl(causal_conv_heads_rows_kernel<2>, grid, dim3(256), 0, stream, p, unit, n_rows);
+  } else
+    rc = launch_pdl(causal_conv_heads_kernel, dim3(n_rows, (items + warps - 1) / warps), dim3(32 * warps), 0, stream, p, unit, single);
   if (!rc && taps > 1 && !single)
     rc = launch_pdl(causal_conv_tail_kernel, dim3(n_entries, (channels + 255) / 256), dim3(256), 0, stream, p);
   return rc ? rc : IFX_LAUNCH_CHECK();

@@ -155,7 +155,7 @@ def _lib():
         lib.ifx_retention_segment.argtypes = []
         lib.ifx_retention_scan.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
                                            c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                                           c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
+                                           c_int, c_int, c_void_p, c_void_p, c_void_p]
         lib.ifx_retention_finish.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_ll, c_int, c_int, c_int, c_float,
                                              c_void_p]
         lib.ifx_gelu_tanh.argtypes = [c_void_p, c_int, c_ll, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
@@ -1424,30 +1424,29 @@ def retention_segment() -> int:
 
 
 def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int, dim: int, vdim: int,
-                   decay: torch.Tensor, k_scale: float, state: torch.Tensor, seg_entry: torch.Tensor, seg_t0: torch.Tensor,
+                   powers: torch.Tensor, k_scale: float, state: torch.Tensor, seg_entry: torch.Tensor, seg_t0: torch.Tensor,
                    n_segments: int, entry_first_seg: torch.Tensor, entry_q_start: torch.Tensor, entry_q_len: torch.Tensor,
-                   entry_slot: torch.Tensor, n_entries: int, multi: bool, out: torch.Tensor, silu: bool = False) -> torch.Tensor:
+                   entry_slot: torch.Tensor, n_entries: int, out: torch.Tensor, silu: bool = False) -> torch.Tensor:
     """``S_t = decay_h S_{t-1} + (k_scale k_t) v_t^T``, ``o_t = S_t^T q_t`` per head over the step's entries, all
-    float32; with ``silu`` q, k and v go through it first.  ``proj`` float32 ``[N, W]`` holds q, k (already rotated) and v heads from the given columns on;
+    float32; with ``silu`` q, k and v go through it first (``proj`` itself does, in a step with portions).
+    ``powers`` float32 ``[heads, segment + 1]``: ``decay_h`` to the 0th, 1st, .. power.  ``proj`` float32 ``[N, W]`` holds q, k (already rotated) and v heads from the given columns on;
     ``state`` float32 ``[slots, heads, dim, vdim]``; ``out`` float32 ``[N, heads * vdim]``."""
     n = proj.shape[0]
     _need(proj.dtype == torch.float32 and proj.dim() == 2 and proj.stride(1) == 1, "retention: float32 projection rows")
     _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim),
           "retention: state float32 [slots, heads, dim, vdim]")
-    _need(decay.dtype == torch.float32 and decay.numel() == heads, "retention: decay float32 [heads]")
+    _need(powers.dtype == torch.float32 and powers.is_contiguous() and tuple(powers.shape) == (heads, retention_segment() + 1),
+          "retention: powers float32 [heads, segment + 1]")
     _need(out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, heads * vdim), "retention: out float32")
-    seg_b = seg_start = None
-    if multi:
-        seg_b = torch.empty((n_segments, heads, dim, vdim), dtype=torch.float32, device=proj.device)
-        seg_start = torch.empty_like(seg_b)
-    _check(_lib().ifx_retention_scan(_ptr(proj), proj.stride(0), q_col, k_col, v_col, heads, dim, vdim, _ptr(decay),
+    portions = n > n_entries
+    seg_start = torch.empty((n_segments, heads, dim, vdim), dtype=torch.float32, device=proj.device) if portions else None
+    _check(_lib().ifx_retention_scan(_ptr(proj), proj.stride(0), q_col, k_col, v_col, heads, dim, vdim, _ptr(powers),
                                      float(k_scale), 1 if silu else 0, _ptr(state), _ptr(seg_entry), _ptr(seg_t0), n_segments,
                                      _ptr(entry_first_seg), _ptr(entry_q_start), _ptr(entry_q_len), _ptr(entry_slot),
-                                     n_entries, n, 1 if multi else 0, _ptr(seg_b), _ptr(seg_start), _ptr(out), _stream()),
-           "retention_scan")
-    if multi:
+                                     n_entries, n, _ptr(seg_start), _ptr(out), _stream()), "retention_scan")
+    if portions:
         global launch_count
-        launch_count += 2
+        launch_count += 2 if silu else 1
     return out
 
 

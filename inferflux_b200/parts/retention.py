@@ -32,7 +32,6 @@ class RetentionStep:
     seg_t0: torch.Tensor
     entry_first_seg: torch.Tensor
     n_segments: int
-    multi: bool                               # some entry has more than one segment
 
 
 class Retention(Part):
@@ -71,7 +70,10 @@ class Retention(Part):
         if self.norm not in ("heads", "row") or self.gate is None:
             raise ValueError("retention: norm is 'heads' or 'row', gate 'silu' or 'sigmoid'")
         self.norm_w: torch.Tensor = None
-        self.decay = torch.tensor(decay, dtype=torch.float32, device=device)
+        # the decays' powers over a segment, worked out in float64
+        seg = ops.retention_segment() if torch.device(device).type == "cuda" else 32
+        self.powers = (torch.tensor(decay, dtype=torch.float64)[:, None]
+                       ** torch.arange(seg + 1, dtype=torch.float64)).to(torch.float32).to(device)
         self.qkvg: Linear = None
         self.o: Linear = None
 
@@ -108,7 +110,7 @@ class Retention(Part):
             first.append(len(seg_entry))
             for t0 in range(0, int(layout.q_len[i]), seg):
                 seg_entry.append(i), seg_t0.append(t0)
-        return RetentionStep(put(seg_entry), put(seg_t0), put(first), len(seg_entry), len(seg_entry) > layout.n_entries)
+        return RetentionStep(put(seg_entry), put(seg_t0), put(first), len(seg_entry))
 
     @property
     def inner_width(self) -> int:
@@ -126,9 +128,9 @@ class Retention(Part):
                                 "the layer's position encoding gave something else")
             ops.rotate_heads(proj, 0, 2 * self.heads, self.dim, position[0], position[1], self.layout)   # q and k heads
         o = torch.empty((n, hv), dtype=torch.float32, device=x.device)
-        ops.retention_scan(proj, 0, hd, 2 * hd, self.heads, self.dim, self.vdim, self.decay, self.k_scale,
+        ops.retention_scan(proj, 0, hd, 2 * hd, self.heads, self.dim, self.vdim, self.powers, self.k_scale,
                            run.states["retention"], step.seg_entry, step.seg_t0, step.n_segments, step.entry_first_seg,
-                           ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, step.multi, o, silu=self.silu)
+                           ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, o, silu=self.silu)
         if out is None:
             out = torch.empty((n, hv), dtype=x.dtype, device=x.device)
         if self.norm == "row" or self.gate != ops.GATE_SILU:

@@ -394,6 +394,21 @@ def _logits_in_steps(runner, rid, toks, sizes):
     return torch.cat(outs)
 
 
+def _steady_prompt(cfg, w, n, seed):
+    """The first prompt from ``seed`` on whose logits one float32 rounding of the weights does not move by more than
+    5e-6: a retention head whose query all but misses its keys is blown up by the unit norm behind it, and on such a
+    prompt two exact ways of adding up in float32 can lie 1e-5 apart."""
+    while True:
+        toks = random_tokens(cfg["vocab"], n, seed)
+        want = plain.forward(cfg, w, toks)
+        gen = torch.Generator().manual_seed(seed)
+        moved = [plain.forward(cfg, {k: v * (1 + 6e-8 * torch.randn(v.shape, generator=gen).double()) for k, v in w.items()}, toks)
+                 for _ in range(2)]
+        if max(_rel(m, want) for m in moved) < 5e-6:
+            return toks
+        seed += 1
+
+
 @gpu
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", ["A", "B", "C"])
@@ -402,7 +417,7 @@ def test_model_whole_one_by_one_and_in_portions(dtype, name):
     for the whole prompt."""
     cfg = _for_dtype(PX[name], dtype)
     model, runner, w = _runner_for(cfg, dtype, ord(name), tokens=1024, sharpen=SHARPEN[dtype])
-    toks = random_tokens(cfg["vocab"], 150, 31)
+    toks = _steady_prompt(cfg, w, 150, 31) if dtype == torch.float32 else random_tokens(cfg["vocab"], 150, 31)
     want = plain.forward(cfg, w, toks)
     whole = _logits_in_steps(runner, "w", toks, [150])
     assert _model_ok(whole, want, dtype)

@@ -439,7 +439,7 @@ def test_gated_delta_alone(dtype, name, layer):
 
 
 @gpu
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim,taps", [(2, 1, 128, 128, 4), (1, 1, 256, 40, 2), (3, 3, 7, 130, 16), (6, 2, 100, 33, 3), (2, 2, 1, 1, 4)])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,taps", [(2, 1, 128, 128, 4), (1, 1, 256, 40, 2), (3, 3, 7, 130, 16), (6, 2, 100, 33, 3), (2, 2, 1, 1, 4), (4, 2, 64, 64, 2)])
 def test_gated_delta_shapes(heads, kv_heads, dim, vdim, taps):
     """Heads from one number to the largest the kernels take, value sizes across their blocks' columns."""
     cfg = dict(ZT["A"], width=48, loop=None, layers=[dict(type="parallel", mlp=None, mixer=dict(
