@@ -117,14 +117,14 @@ causal_conv_heads_kernel(ConvArgs p, UnitHeads unit, int single) {
     if (lane + 32 * b < size) dst[lane + 32 * b] = y[b] * f;
 }
 
-// The same for up to four taps and channels in fours: a lane takes four neighbouring channels of `rows_each` rows one after
-// the other (ROWS in a step with portions, one in a step of single tokens), with the weights and the last TAPS - 1 inputs in
+// The same for up to four taps and channels in fours: a lane takes four neighbouring channels of EACH rows one after the
+// other (ROWS in a step with portions, one in a step of single tokens), with the weights and the last TAPS - 1 inputs in
 // registers, so an input is read once.
 constexpr int ROWS = 8;
 
-template <int TAPS>
+template <int TAPS, int EACH>
 __global__ void __launch_bounds__(256)
-causal_conv_heads_rows_kernel(ConvArgs p, UnitHeads unit, int n_rows, int rows_each, int single) {
+causal_conv_heads_rows_kernel(ConvArgs p, UnitHeads unit, int n_rows) {
   pdl_enter();
   const int lane = threadIdx.x & 31;
   const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -146,7 +146,7 @@ causal_conv_heads_rows_kernel(ConvArgs p, UnitHeads unit, int n_rows, int rows_e
   const float4 bias = p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   const float factor = item < unit.scaled ? unit.scale : 1.0f;
   float4 u[TAPS];                                        // u[j]: the input TAPS - 1 - j tokens back
-  const int first = blockIdx.x * rows_each, last = min(first + rows_each, n_rows);
+  const int first = blockIdx.x * EACH, last = min(first + EACH, n_rows);
   for (int row = first; row < last; ++row) {
     const int e = p.row_entry[row], i = row - p.entry_q_start[e];
     if (row == first || i == 0) {                        // the inputs before this row, from the step or from the slot
@@ -176,9 +176,8 @@ causal_conv_heads_rows_kernel(ConvArgs p, UnitHeads unit, int n_rows, int rows_e
       const float f = factor / sqrtf(warp_sum(ss) + unit.eps);
       y.x *= f; y.y *= f; y.z *= f; y.w *= f;
     }
-    if (!on) continue;
-    *reinterpret_cast<float4*>(p.out + (size_t)row * p.out_stride + c) = y;
-    if (single) {
+    if (on) *reinterpret_cast<float4*>(p.out + (size_t)row * p.out_stride + c) = y;
+    if (EACH == 1 && on) {                               // single tokens: the tail moves on here
       float* tail = p.tail + (size_t)p.entry_slot[e] * KEEP * p.channels;
 #pragma unroll
       for (int j = 0; j < KEEP; ++j) *reinterpret_cast<float4*>(tail + (size_t)j * p.channels + c) = u[j + 1];
@@ -365,11 +364,14 @@ IFX_API int ifx_causal_conv_heads(const float* in, long long in_stride, int col0
                     !(((uintptr_t)in | (uintptr_t)w | (uintptr_t)bias | (uintptr_t)tail | (uintptr_t)out) & 15);
   int rc;
   if (rows) {
-    const int each = single ? 1 : ROWS;
-    const dim3 grid((n_rows + each - 1) / each, (items + warps - 1) / warps), block(32 * warps);
-    rc = taps == 4 ? launch_pdl(causal_conv_heads_rows_kernel<4>, grid, block, 0, stream, p, unit, n_rows, each, single)
-       : taps == 3 ? launch_pdl(causal_conv_heads_rows_kernel<3>, grid, block, 0, stream, p, unit, n_rows, each, single)
-                   : launch_pdl(causal_conv_heads_rows_kernel<2>, grid, block, 0, stream, p, unit, n_rows, each, single);
+    const dim3 one(n_rows, (items + warps - 1) / warps), many((n_rows + ROWS - 1) / ROWS, (items + 7) / 8);
+#define IFX_CONV_ROWS(T)                                                                                                          \
+  rc = single ? launch_pdl(causal_conv_heads_rows_kernel<T, 1>, one, dim3(32 * warps), 0, stream, p, unit, n_rows)               \
+              : launch_pdl(causal_conv_heads_rows_kernel<T, ROWS>, many, dim3(256), 0, stream, p, unit, n_rows)
+    if (taps == 4) IFX_CONV_ROWS(4);
+    else if (taps == 3) IFX_CONV_ROWS(3);
+    else IFX_CONV_ROWS(2);
+#undef IFX_CONV_ROWS
   } else
     rc = launch_pdl(causal_conv_heads_kernel, dim3(n_rows, (items + warps - 1) / warps), dim3(32 * warps), 0, stream, p, unit, single);
   if (!rc && taps > 1 && !single)
