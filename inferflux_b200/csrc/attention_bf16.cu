@@ -413,10 +413,13 @@ attn_prefill_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* _
   } else if (opt.gate.p) {
 #pragma unroll
     for (int d = 0; d < DT; ++d) {
-      const int col = d * 8 + t4 * 2;
+      const int col = head * HD + d * 8 + t4 * 2;
       float ga[2] = {0.0f, 0.0f}, gb[2] = {0.0f, 0.0f};
-      if (ra < rows) { ga[0] = opt.gate.sums(tok0 + ra, head, HD, col); ga[1] = opt.gate.sums(tok0 + ra, head, HD, col + 1); }
-      if (rb < rows) { gb[0] = opt.gate.sums(tok0 + rb, head, HD, col); gb[1] = opt.gate.sums(tok0 + rb, head, HD, col + 1); }
+      for (int sl = 0; sl < opt.gate.parts; ++sl) {               // the four numbers of a slice are asked for together
+        const float* gp = opt.gate.p + (size_t)sl * opt.gate.part_stride + col;
+        if (ra < rows) { ga[0] += gp[(size_t)(tok0 + ra) * opt.gate.stride]; ga[1] += gp[(size_t)(tok0 + ra) * opt.gate.stride + 1]; }
+        if (rb < rows) { gb[0] += gp[(size_t)(tok0 + rb) * opt.gate.stride]; gb[1] += gp[(size_t)(tok0 + rb) * opt.gate.stride + 1]; }
+      }
       o[d][0] *= 1.0f / (1.0f + __expf(-ga[0])); o[d][1] *= 1.0f / (1.0f + __expf(-ga[1]));
       o[d][2] *= 1.0f / (1.0f + __expf(-gb[0])); o[d][3] *= 1.0f / (1.0f + __expf(-gb[1]));
     }
