@@ -490,6 +490,28 @@ class PemoraxConfig(ModelConfig):
                 "norm": {"eps": self.norm_eps}, "layers": layers}
 
 
+def _rotation(m: Dict[str, Any], where: str, dim: int) -> Dict[str, Any]:
+    """``rot`` of a mixer with heads of ``dim``: how many dimensions rotate (none without the key), the base, and the
+    frequencies' scaling by wavelength bands or None."""
+    out = {"dims": 0, "base": 10000.0, "scaling": None}
+    rot = _sub(m, "rot", where, optional=True)
+    if rot is None or not rot.get("dims"):
+        return out
+    dims = _require_int(rot, "dims")
+    if dims % 2 or dims > dim:
+        raise ConfigError(f"{where}: rot.dims {dims} must be even and at most dim {dim}")
+    base = _require_number(rot, "base", where + " rot")
+    if base <= 1.0:
+        raise ConfigError(f"{where}: rot.base must be above 1")
+    out.update(dims=dims, base=base)
+    sc = _sub(rot, "scaling", where + " rot", optional=True)
+    if sc is not None:
+        s = out["scaling"] = {k: _require_number(sc, k, where + " rot.scaling") for k in ("factor", "low", "high", "original")}
+        if min(s.values()) <= 0 or s["high"] == s["low"]:
+            raise ConfigError(f"{where}: the numbers of rot.scaling must be positive, high and low different")
+    return out
+
+
 @dataclass(frozen=True)
 class TekosunLayer:
     """One layer of a Tekosun model as config.json gives it: ``type`` (which mixer), the mixer's sizes and
@@ -554,7 +576,7 @@ class TekosunConfig(ModelConfig):
         heads, dim = _require_int(m, "heads"), _require_int(m, "dim")
         out = {"heads": heads, "kv_heads": cls._opt_int(m, "kv_heads", heads), "dim": dim, "vdim": cls._opt_int(m, "vdim", dim),
                "scale": _require_number(m, "scale", where) if m.get("scale") is not None else float(dim) ** -0.5,
-               "v_mix": bool(m.get("v_mix") or False), "window": None, "rot": {"dims": 0, "base": 10000.0, "scaling": None}}
+               "v_mix": bool(m.get("v_mix") or False), "window": None}
         if heads % out["kv_heads"]:
             raise ConfigError(f"{where}: heads {heads} is not a multiple of kv_heads {out['kv_heads']}")
         if dim > 256 or out["vdim"] > 256:
@@ -562,21 +584,7 @@ class TekosunConfig(ModelConfig):
         mask = _sub(m, "mask", where, optional=True)
         if mask is not None and mask.get("size") is not None:
             out["window"] = _require_int(mask, "size")
-        rot = _sub(m, "rot", where, optional=True)
-        if rot is not None and rot.get("dims"):
-            dims = _require_int(rot, "dims")
-            if dims % 2 or dims > dim:
-                raise ConfigError(f"{where}: rot.dims {dims} must be even and at most dim {dim}")
-            base = _require_number(rot, "base", where + " rot")
-            if base <= 1.0:
-                raise ConfigError(f"{where}: rot.base must be above 1")
-            out["rot"] = {"dims": dims, "base": base, "scaling": None}
-            sc = _sub(rot, "scaling", where + " rot", optional=True)
-            if sc is not None:
-                out["rot"]["scaling"] = {k: _require_number(sc, k, where + " rot.scaling") for k in ("factor", "low", "high", "original")}
-                s = out["rot"]["scaling"]
-                if min(s.values()) <= 0 or s["high"] == s["low"]:
-                    raise ConfigError(f"{where}: the numbers of rot.scaling must be positive, high and low different")
+        out["rot"] = _rotation(m, where, dim)
         return out
 
     @classmethod
@@ -974,6 +982,157 @@ class ZetivikConfig(ModelConfig):
                "layers": layers}
         if self.logit_softcap is not None:
             out["logit_softcap"] = self.logit_softcap
+        if self.loop_times:
+            out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return out
+
+
+@dataclass(frozen=True)
+class KibilixLayer:
+    """One layer of a Kibilix model as config.json gives it: ``type`` (which mixer), the mixer's sizes and constants
+    (checked, defaults filled in) and its feed-forward (``None`` = none; ``kind`` ``dense`` with ``ff``, or ``moe`` with the
+    experts' ``ff`` and ``limit`` and the router's ``experts``, ``identity`` and ``top``)."""
+
+    type: str = ""
+    mixer: Dict[str, Any] = field(default_factory=dict)
+    mlp: Optional[Dict[str, Any]] = None
+
+
+@dataclass(frozen=True)
+class KibilixConfig(ModelConfig):
+    """``Kibilix``: a decoder whose layers are listed one by one in config.json (``layers``: ``type``, the mixer's sizes
+    under ``mixer``, the feed-forward under ``mlp`` or null).  The residual stream is ``streams`` copies wide: a sublayer
+    reads a weighted sum of the copies and its result, times ``residual_mult``, joins them as they are mixed anew.  The
+    embedding is a token's row plus, with ``embedding.bigram``, a hashed row of the token and the one before it.
+    Mixers: ``attention`` (grouped queries inside chunks of ``mask.size`` positions, capped scores, rotate-half positions
+    with an optional scaling by wavelength bands) and ``channel_delta`` (the gated delta rule with one decay per head and
+    key channel).  Feed-forwards: ``dense`` (squared relu) and ``moe`` (gated experts with clamped inputs, chosen by
+    softmax scores plus a correction, some of the router's outputs standing for the identity).  A stretch of layers
+    (``loop``: ``start``, ``stop``, ``times``) may run several times in a row on the same weights."""
+
+    width: int = 0
+    vocab: int = 0
+    norm_eps: float = 1e-6
+    streams: int = 1
+    residual_mult: float = 1.0
+    bigram: Optional[Dict[str, int]] = None          # buckets, mul_prev, mul_cur
+    layers: List[KibilixLayer] = field(default_factory=list)
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0              # 0 = the model has no loop
+
+    ARCHITECTURE = "Kibilix"
+    MODEL_TYPE = "kibilix"
+    MIXERS = ("attention", "channel_delta")
+    MAX_STREAMS = 16
+
+    @classmethod
+    def _attention(cls, m: Dict[str, Any], where: str) -> Dict[str, Any]:
+        out = ZetivikConfig._heads(m, where)
+        if out["vdim"] > 256:
+            raise ConfigError(f"{where}: vdim {out['vdim']} is not supported (at most 256)")
+        out["scale"] = _require_number(m, "scale", where) if m.get("scale") is not None else float(out["dim"]) ** -0.5
+        out["softcap"] = _require_number(m, "softcap", where) if m.get("softcap") is not None else None
+        if out["softcap"] is not None and out["softcap"] <= 0:
+            raise ConfigError(f"{where}: softcap must be positive")
+        mask = _sub(m, "mask", where, optional=True)
+        out["chunk"] = _require_int(mask, "size") if mask is not None and mask.get("size") is not None else None
+        out["rot"] = _rotation(m, where, out["dim"])
+        return out
+
+    @classmethod
+    def _channel_delta(cls, m: Dict[str, Any], where: str) -> Dict[str, Any]:
+        return ZetivikConfig._right(m, where)
+
+    @staticmethod
+    def _mlp(mlp: Dict[str, Any], where: str) -> Dict[str, Any]:
+        kind = mlp.get("kind")
+        if kind == "dense":
+            return {"kind": "dense", "ff": _require_int(mlp, "ff")}
+        if kind != "moe":
+            raise ConfigError(f"{where}: kind {kind!r} is not one of ['dense', 'moe']")
+        expert, router = _sub(mlp, "expert", where), _sub(mlp, "router", where)
+        out = {"kind": "moe", "ff": _require_int(expert, "ff"), "limit": _require_number(expert, "limit", where + " expert"),
+               "experts": _require_int(router, "experts"), "top": _require_int(router, "top"),
+               "identity": _require_int(router, "identity", 0) if router.get("identity") is not None else 0}
+        if out["limit"] <= 0:
+            raise ConfigError(f"{where}: expert.limit must be positive")
+        if out["top"] > out["experts"] + out["identity"]:
+            raise ConfigError(f"{where}: router.top {out['top']} exceeds the router's {out['experts'] + out['identity']} outputs")
+        if out["top"] > 64:
+            raise ConfigError(f"{where}: router.top {out['top']} is not supported (at most 64)")
+        return out
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "KibilixConfig":
+        width, vocab = _require_int(d, "width"), _require_int(d, "vocab")
+        eps = _require_number(_sub(d, "norm", "config.json"), "eps", "config.json norm")
+        if eps <= 0:
+            raise ConfigError(f"norm eps must be positive, got {eps}")
+        streams = _require_int(d, "streams") if d.get("streams") is not None else 1
+        if streams > cls.MAX_STREAMS:
+            raise ConfigError(f"config.json: {streams} streams are not supported (at most {cls.MAX_STREAMS})")
+        b = _sub(_sub(d, "embedding", "config.json", optional=True) or {}, "bigram", "config.json embedding", optional=True)
+        bigram = None
+        if b is not None:
+            bigram = {"buckets": _require_int(b, "buckets"), "mul_prev": _require_int(b, "mul_prev", 0), "mul_cur": _require_int(b, "mul_cur", 0)}
+            if (bigram["mul_prev"] + bigram["mul_cur"]) * vocab >= 1 << 63:
+                raise ConfigError("config.json: the bigram's multipliers times the vocabulary exceed 64 bits")
+        raw = d.get("layers")
+        if not isinstance(raw, list) or not raw:
+            raise ConfigError("config.json: 'layers' must be a non-empty list")
+        layers = []
+        for i, entry in enumerate(raw):
+            where = f"config.json layers[{i}]"
+            if not isinstance(entry, dict):
+                raise ConfigError(f"{where}: must be an object")
+            kind = entry.get("type")
+            if kind not in cls.MIXERS:
+                raise ConfigError(f"{where}: type {kind!r} is not one of {list(cls.MIXERS)}")
+            mixer = getattr(cls, "_" + kind)(_sub(entry, "mixer", where), where + " mixer")
+            mlp = _sub(entry, "mlp", where, optional=True)
+            layers.append(KibilixLayer(type=kind, mixer=mixer, mlp=cls._mlp(mlp, where + " mlp") if mlp is not None else None))
+        start = stop = times = 0
+        loop = _sub(d, "loop", "config.json", optional=True)
+        if loop is not None:
+            start, stop = _require_int(loop, "start", 0), _require_int(loop, "stop", 0)
+            times = _require_int(loop, "times", 1)
+            if not 0 <= start < stop <= len(layers):
+                raise ConfigError(f"config.json: loop {start}..{stop} does not lie within the {len(layers)} layers")
+        arch = d.get("architecture") or (d.get("architectures") or [cls.ARCHITECTURE])[0]
+        return cls(architectures=[str(arch)], model_type=str(d.get("model_type", "") or cls.MODEL_TYPE), width=width,
+                   vocab=vocab, norm_eps=eps, streams=streams, residual_mult=_opt_number(d, "residual_mult", 1.0), bigram=bigram,
+                   layers=layers, loop_start=start, loop_stop=stop, loop_times=times)
+
+    @property
+    def vocab_size(self) -> int:
+        return self.vocab
+
+    @property
+    def eos_token_id(self) -> Optional[int]:
+        return None
+
+    def to_dict(self) -> Dict[str, Any]:
+        """The config.json this configuration was read from (its own keys)."""
+        layers = []
+        for l in self.layers:
+            m, mlp = {k: v for k, v in l.mixer.items() if v is not None}, None
+            if l.type == "attention":
+                chunk, rot = m.pop("chunk", None), m.pop("rot")
+                if chunk:
+                    m["mask"] = {"size": chunk}
+                if rot["dims"]:
+                    m["rot"] = {k: v for k, v in rot.items() if v is not None}
+            if l.mlp and l.mlp["kind"] == "dense":
+                mlp = dict(l.mlp)
+            elif l.mlp:
+                mlp = {"kind": "moe", "expert": {k: l.mlp[k] for k in ("ff", "limit")},
+                       "router": {k: l.mlp[k] for k in ("experts", "identity", "top")}}
+            layers.append({"type": l.type, "mixer": m, "mlp": mlp})
+        out = {"architecture": self.architecture, "width": self.width, "vocab": self.vocab, "norm": {"eps": self.norm_eps},
+               "streams": self.streams, "residual_mult": self.residual_mult, "layers": layers}
+        if self.bigram:
+            out["embedding"] = {"bigram": dict(self.bigram)}
         if self.loop_times:
             out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
         return out

@@ -463,9 +463,10 @@ struct QkvPrep {
 
 // What shapes a decoded token's scores beyond the scale (all off for plain attention): a query temperature (the
 // query at position p counts 1 + coef * ln(floor((p + 1) / every) + 1) times; every = 0: none) and a toll on
-// distance (the score of key j loses r1[head] * ln(1 + r2[head] * (p - j)); null: none).
+// distance (the score of key j loses r1[head] * ln(1 + r2[head] * (p - j)); null: none); softcap > 0: scores become
+// softcap * tanh(s / softcap), ahead of the toll.
 struct ScoreShape {
-  float q_temp_coef; int q_temp_every; const float* dist_r1; const float* dist_r2;
+  float q_temp_coef; int q_temp_every; const float* dist_r1; const float* dist_r2; float softcap;
   HeadGate gate;            // the heads' results times the sigmoid of sums beside them
 };
 
@@ -596,9 +597,10 @@ attn_decode_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __
         qb[k][1] = g < nrows ? pq[k * 8 + 4 + t4] : 0u;
       }
     }
-    // shaped scores (a temperature, a toll) are brought to their final form before the softmax; their exponents
+    // shaped scores (a temperature, a cap, a toll) are brought to their final form before the softmax; their exponents
     // need no further scale
-    const bool shaped = shape.q_temp_every > 0 || shape.dist_r1 != nullptr;
+    const bool shaped = shape.q_temp_every > 0 || shape.dist_r1 != nullptr || shape.softcap > 0.0f;
+    const float cap = shape.softcap, cap_inv = cap > 0.0f ? 1.0f / cap : 0.0f;
     const float sl2 = shaped ? LOG2E : scale * LOG2E;
     float row_scale = scale, toll1[2] = {0.0f, 0.0f}, toll2[2] = {0.0f, 0.0f};
     if (shape.q_temp_every > 0) row_scale *= 1.0f + shape.q_temp_coef * logf((float)(len / shape.q_temp_every + 1));
@@ -652,7 +654,9 @@ attn_decode_bf16_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int dist = max(len - 1 - (key0 + g + (c >> 1) * 8), 0);
-          s[c] = s[c] * row_scale - toll1[c & 1] * __logf(fmaf(toll2[c & 1], (float)dist, 1.0f));
+          s[c] *= row_scale;
+          if (cap > 0.0f) s[c] = cap * tanh_exp(s[c] * cap_inv);
+          if (shape.dist_r1) s[c] -= toll1[c & 1] * __logf(fmaf(toll2[c & 1], (float)dist, 1.0f));
         }
       }
       const bool in0 = key0 + g >= kb && key0 + g < ke, in1 = key0 + g + 8 >= kb && key0 + g + 8 < ke;
@@ -1308,19 +1312,20 @@ IFX_API int ifx_attn_prefill_bf16(const void* q, long long q_stride, void* out, 
 
 // Scratch: part_o float32 [n_dec * n_heads * n_splits * head_dim], part_ml float32
 // [n_dec * n_heads * n_splits * 2] (unused when n_splits == 1).
-// q_temp_every > 0: a query temperature; dist_r1 / dist_r2 ([n_heads] float32 or null): a toll on distance; gate: float32
+// softcap > 0: capped scores; q_temp_every > 0: a query temperature; dist_r1 / dist_r2 ([n_heads] float32 or null): a toll
+// on distance; gate: float32
 // slices [gate_parts][N][gate_stride] or null, a column per element or (gate_per_head) per head; window < 0: chunks.
 IFX_API int ifx_attn_decode_bf16_ex(const void* q, long long q_stride, void* out, long long out_stride,
                                     void* k_layer, void* v_layer, long long page_stride, int page_size,
                                     const int* block_tables, int bt_stride, const int* dec_entries, int n_dec,
                                     const int* entry_q_start, const int* entry_q_len, const int* entry_ctx_start,
                                     float* part_o, float* part_ml, int n_heads, int n_kv, int head_dim, float scale,
-                                    int window, int n_splits, float q_temp_coef, int q_temp_every, const float* dist_r1,
+                                    int window, int n_splits, float softcap, float q_temp_coef, int q_temp_every, const float* dist_r1,
                                     const float* dist_r2, const float* gate, int gate_parts, long long gate_part_stride,
                                     int gate_stride, int gate_per_head, cudaStream_t stream) {
   if (n_dec <= 0) return 0;
-  if (q_temp_every < 0 || (dist_r1 != nullptr) != (dist_r2 != nullptr)) return IFX_ERR_UNSUPPORTED;
-  const ScoreShape shape{q_temp_coef, q_temp_every, dist_r1, dist_r2,
+  if (softcap < 0.0f || q_temp_every < 0 || (dist_r1 != nullptr) != (dist_r2 != nullptr)) return IFX_ERR_UNSUPPORTED;
+  const ScoreShape shape{q_temp_coef, q_temp_every, dist_r1, dist_r2, softcap,
                          HeadGate{gate, gate_parts, gate_part_stride, gate_stride, gate_per_head}};
   if (n_kv < 1 || n_heads % n_kv || n_splits < 1 || n_splits > 65535) return IFX_ERR_UNSUPPORTED;
   if (page_size <= 0 || (page_size & (page_size - 1))) return IFX_ERR_UNSUPPORTED;
@@ -1344,7 +1349,7 @@ IFX_API int ifx_attn_decode_bf16(const void* q, long long q_stride, void* out, l
                                  int window, int n_splits, cudaStream_t stream) {
   return ifx_attn_decode_bf16_ex(q, q_stride, out, out_stride, k_layer, v_layer, page_stride, page_size, block_tables, bt_stride,
                                  dec_entries, n_dec, entry_q_start, entry_q_len, entry_ctx_start, part_o, part_ml, n_heads, n_kv,
-                                 head_dim, scale, window, n_splits, 0.0f, 0, nullptr, nullptr, nullptr, 0, 0, 0, 0, stream);
+                                 head_dim, scale, window, n_splits, 0.0f, 0.0f, 0, nullptr, nullptr, nullptr, 0, 0, 0, 0, stream);
 }
 
 // The same for a step of single tokens only, with the work of ifx_qkv_rope_kv_write folded in: qkv is the

@@ -85,6 +85,14 @@ struct PagedKV {
   int page_shift;          // log2(page_size)
 };
 
+// A gated activation whose two inputs are clamped before they meet: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g * sigmoid(alpha * g) * (u + shift).
+struct GluShape { float limit, alpha, shift; };
+__device__ __forceinline__ float clamped_glu(float gate, float up, const GluShape& c) {
+  const float g = fminf(gate, c.limit), u = fminf(fmaxf(up, -c.limit), c.limit);
+  return g / (1.0f + expf(-c.alpha * g)) * (u + c.shift);
+}
+
 // How far back attention reaches is one int: 0 = to the sequence's start, w > 0 = the last w positions (the token's
 // own among them), -c < 0 = to the start of the token's chunk of c positions, chunks counted from position 0.
 // The first position that the query at position p sees; it never falls as p grows.

@@ -488,14 +488,15 @@ IFX_API int ifx_gelu_tanh(const float* z, int parts, long long part_stride, void
 
 // ---- one-argument activations over float32 sums, rounded once into the engine's type ----------------
 // out[m][c] = act(sum over slices of z[m][c]);  z rows z_stride elements apart (a block of columns of a wider
-// projection), slices part_stride apart.  act: 0 gelu (tanh form), 1 tanh, 2 relu(z)^2, 3 silu, 4 sigmoid.
+// projection), slices part_stride apart.  act: 0 gelu (tanh form), 1 tanh, 2 relu(z)^2, 3 silu, 4 sigmoid, 5 z itself.
 __device__ __forceinline__ float apply_activation(float v, int act) {
   switch (act) {
     case 0: return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
     case 1: return tanhf(v);
     case 2: { const float r = fmaxf(v, 0.0f); return r * r; }
     case 3: return v / (1.0f + expf(-v));
-    default: return 1.0f / (1.0f + expf(-v));
+    case 4: return 1.0f / (1.0f + expf(-v));
+    default: return v;
   }
 }
 
@@ -548,7 +549,7 @@ IFX_API int ifx_activation(const float* z, long long z_stride, int parts, long l
                            long long out_stride, int m, int cols, int act, cudaStream_t stream) {
   const long long total = (long long)m * cols;
   if (total <= 0) return 0;
-  if (act < 0 || act > 4) return IFX_ERR_UNSUPPORTED;
+  if (act < 0 || act > 5) return IFX_ERR_UNSUPPORTED;
   int rc;
   if (!(cols & 3) && !((z_stride | part_stride | out_stride) & 3) && !((uintptr_t)z & 15) && !((uintptr_t)out & 15) &&
       (out_dtype == IFX_F32 || out_dtype == IFX_BF16)) {

@@ -2,7 +2,8 @@
 //
 //   z = the router's float32 logits of a token;  chosen = the `top` largest (lowest index first among equals);
 //   weight_k = exp(z_k) / sum over the chosen exp(z)                                           (route)
-//   the (token, choice) pairs are sorted by expert into tiles of TILE rows, each tile one expert's (group)
+//   the (token, choice) pairs are sorted by expert into tiles of TILE rows, each tile one expert's (group); a choice
+//   beyond the experts is one of the identity: it has no product, and its result is the token's row itself
 //   act = silu(x Wg_e^T) * (x Wu_e^T)   per tile, rows gathered from the tokens                 (expert_product)
 //   y   = act Wd_e^T                    per tile, float32
 //   out[token] = sum_k weight_k y[pair]  in the order of the choices                            (combine)
@@ -15,23 +16,36 @@
 
 namespace {
 constexpr int MAX_TOP = 64;
-// what a tile product does with its sums: nothing; W_e = [gate rows; up rows] and out = silu(gate) * up; out = relu(sum)^2
-constexpr int MODE_PLAIN = 0, MODE_SWIGLU = 1, MODE_RELU2 = 2;
+// what a tile product does with its sums: nothing; W_e = [gate rows; up rows] and out = silu(gate) * up; out = relu(sum)^2;
+// W_e as for the second and out = g * sigmoid(alpha * g) * (u + shift), g = min(gate, limit), u = clamp(up, -limit, limit)
+constexpr int MODE_PLAIN = 0, MODE_SWIGLU = 1, MODE_RELU2 = 2, MODE_CLAMPED = 3;
+
+template <int MODE> __device__ __forceinline__ float glu(float g, float u, const GluShape& c) {
+  if (MODE == MODE_CLAMPED) return clamped_glu(g, u, c);
+  return g / (1.0f + expf(-g)) * u;
+}
 
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const float* __restrict__ logits, int n_tokens, int experts, int top, int over_all, float scale,
-                 int* __restrict__ chosen, float* __restrict__ weights) {
+                 const float* __restrict__ correction, int* __restrict__ chosen, float* __restrict__ weights) {
   pdl_enter();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= n_tokens) return;
   const float* z = logits + (size_t)t * experts;
   int ids[MAX_TOP]; float vals[MAX_TOP];
+  float most = -INFINITY, all = 0.0f;
+  if (over_all) {                        // the scores' softmax over every expert
+    for (int e = lane; e < experts; e += 32) most = fmaxf(most, z[e]);
+    most = warp_max(most);
+    for (int e = lane; e < experts; e += 32) all += expf(z[e] - most);
+    all = warp_sum(all);
+  }
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY; int arg = 0x7fffffff;
     for (int e = lane; e < experts; e += 32) {
       bool taken = false;
       for (int u = 0; u < k; ++u) taken |= ids[u] == e;
-      const float v = z[e];
+      const float v = correction ? expf(z[e] - most) / all + correction[e] : z[e];
       if (!taken && (v > best || (v == best && e < arg))) { best = v; arg = e; }
     }
     for (int o = 16; o > 0; o >>= 1) {
@@ -42,15 +56,15 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int experts, in
     ids[k] = arg; vals[k] = best;
   }
   if (over_all) {
-    // scores are the softmax over every expert; a chosen one's weight is its score over the chosen scores' sum
-    float all = 0.0f;
-    for (int e = lane; e < experts; e += 32) all += expf(z[e] - vals[0]);
-    all = warp_sum(all);
+    // a chosen one's weight is its score (without the correction of the choice) over the chosen scores' sum
     float sum = 0.0f;
-    for (int k = 0; k < top; ++k) sum += expf(vals[k] - vals[0]) / all;
+    for (int k = 0; k < top; ++k) {
+      vals[k] = expf(z[ids[k]] - most) / all;
+      sum += vals[k];
+    }
     for (int k = lane; k < top; k += 32) {
       chosen[(size_t)t * top + k] = ids[k];
-      weights[(size_t)t * top + k] = expf(vals[k] - vals[0]) / all / (sum + 1e-20f) * scale;
+      weights[(size_t)t * top + k] = vals[k] / (sum + 1e-20f) * scale;
     }
     return;
   }
@@ -64,7 +78,7 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int experts, in
 
 // One block: counts per expert, tiles per expert, a place for every pair.
 //   tile_expert[max_tiles]: the expert of each tile or -1;  sorted_pair[max_tiles * tile]: the pair at each sorted
-//   row or -1;  pair_row[pairs]: the sorted row of each pair.
+//   row or -1;  pair_row[pairs]: the sorted row of each pair, -1 for one that chose no expert (a choice >= experts).
 __global__ void __launch_bounds__(1024)
 moe_group_kernel(const int* __restrict__ chosen, int pairs, int experts, int tile, int max_tiles,
                  int* __restrict__ tile_expert, int* __restrict__ sorted_pair, int* __restrict__ pair_row) {
@@ -77,7 +91,8 @@ moe_group_kernel(const int* __restrict__ chosen, int pairs, int experts, int til
   for (int i = threadIdx.x; i < max_tiles * tile; i += blockDim.x) sorted_pair[i] = -1;
   for (int i = threadIdx.x; i < max_tiles; i += blockDim.x) tile_expert[i] = -1;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&count[chosen[i]], 1);
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) 
+    if (chosen[i] < experts) atomicAdd(&count[chosen[i]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int t = 0;
@@ -91,6 +106,7 @@ moe_group_kernel(const int* __restrict__ chosen, int pairs, int experts, int til
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     const int e = chosen[i];
+    if (e >= experts) { pair_row[i] = -1; continue; }
     const int r = first[e] + atomicAdd(&cursor[e], 1);
     sorted_pair[r] = i;
     pair_row[i] = r;
@@ -104,8 +120,8 @@ template <typename TA, typename TW, typename TO, int TM, int MODE>
 __global__ void __launch_bounds__(256)
 moe_product_kernel(const TA* __restrict__ A, long long lda, int gather_div /* 0: rows are sorted rows; else token = pair / gather_div */,
                    const TW* __restrict__ W, const int* __restrict__ tile_expert, const int* __restrict__ sorted_pair,
-                   TO* __restrict__ C, long long ldc, int n_out, int K) {
-  constexpr bool SWIGLU = MODE == MODE_SWIGLU;
+                   TO* __restrict__ C, long long ldc, int n_out, int K, GluShape shape) {
+  constexpr bool SWIGLU = MODE == MODE_SWIGLU || MODE == MODE_CLAMPED;
   constexpr int BM = 16 * TM, BN = 64, BK = 16;
   constexpr int TN = SWIGLU ? 2 : 4;                // per thread: TM x TN outputs (SWIGLU: of gate and of up each)
   pdl_enter();
@@ -172,8 +188,7 @@ moe_product_kernel(const TA* __restrict__ A, long long lda, int gather_div /* 0:
       const int n = n0 + tx * TN + j;
       if (n >= n_out) continue;
       if (SWIGLU) {
-        const float g = acc[i][j], u = acc[i][2 + j];
-        crow[n] = Num<TO>::from_f(g / (1.0f + expf(-g)) * u);
+        crow[n] = Num<TO>::from_f(glu<MODE>(acc[i][j], acc[i][2 + j], shape));
       } else if (MODE == MODE_RELU2) {
         const float r = fmaxf(acc[i][j], 0.0f);
         crow[n] = Num<TO>::from_f(r * r);
@@ -198,8 +213,8 @@ template <typename TO, int MODE>
 __global__ void __launch_bounds__(128)
 moe_product_mma_kernel(const bf16* __restrict__ A, long long lda, int gather_div, const bf16* __restrict__ W,
                        const int* __restrict__ tile_expert, const int* __restrict__ sorted_pair, TO* __restrict__ C,
-                       long long ldc, int n_out, int K) {
-  constexpr bool SWIGLU = MODE == MODE_SWIGLU;
+                       long long ldc, int n_out, int K, GluShape shape) {
+  constexpr bool SWIGLU = MODE == MODE_SWIGLU || MODE == MODE_CLAMPED;
   constexpr int BM = 16, BN = 64, BK = 64, LD = BK + 8;
   pdl_enter();
   __shared__ __align__(16) bf16 As[BM][LD];
@@ -262,8 +277,7 @@ moe_product_mma_kernel(const bf16* __restrict__ A, long long lda, int gather_div
     for (int j = 0; j < 2; ++j) {
       if (SWIGLU) {
         const int n = n0 + 8 * warp + 2 * t + j;
-        const float gt = acc0[2 * h + j], up = acc1[2 * h + j];
-        if (n < n_out) crow[n] = Num<TO>::from_f(gt / (1.0f + expf(-gt)) * up);
+        if (n < n_out) crow[n] = Num<TO>::from_f(glu<MODE>(acc0[2 * h + j], acc1[2 * h + j], shape));
       } else {
         const int na = n0 + 16 * warp + 2 * t + j, nb = na + 8;
         float va = acc0[2 * h + j], vb = acc1[2 * h + j];
@@ -275,49 +289,103 @@ moe_product_mma_kernel(const bf16* __restrict__ A, long long lda, int gather_div
   }
 }
 
+// x: the rows that went in (what a choice of the identity gives), read only where a pair has no sorted row.
+template <typename T>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pair_row, const float* __restrict__ weights,
-                   float* __restrict__ out, int hidden, int top) {
+                   const T* __restrict__ x, float* __restrict__ out, int hidden, int top) {
   pdl_enter();
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float acc = 0.0f;
-    for (int k = 0; k < top; ++k)
-      acc = fmaf(weights[(size_t)t * top + k], y[(size_t)pair_row[(size_t)t * top + k] * hidden + i], acc);
+    for (int k = 0; k < top; ++k) {
+      const int r = pair_row[(size_t)t * top + k];
+      const float v = r >= 0 ? y[(size_t)r * hidden + i] : Num<T>::to_f(x[(size_t)t * hidden + i]);
+      acc = fmaf(weights[(size_t)t * top + k], v, acc);
+    }
     out[(size_t)t * hidden + i] = acc;
   }
 }
 
-// act: MODE_SWIGLU (w_up = [gate rows; up rows] of every expert) or MODE_RELU2 (w_up = up rows alone)
+// Four neighbouring columns a thread, the choices' rows asked for together (rows on 16-byte boundaries).
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ y, const int* __restrict__ pair_row, const float* __restrict__ weights,
+                       const T* __restrict__ x, float* __restrict__ out, int hidden, int top) {
+  pdl_enter();
+  constexpr int AHEAD = 4;
+  const int t = blockIdx.x;
+  const int* rows = pair_row + (size_t)t * top;
+  const float* w = weights + (size_t)t * top;
+  for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
+    float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int k0 = 0; k0 < top; k0 += AHEAD) {
+      float4 v[AHEAD];
+      float f[AHEAD];
+#pragma unroll
+      for (int k = 0; k < AHEAD; ++k) {
+        v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        f[k] = 0.0f;
+        if (k0 + k >= top) continue;
+        const int r = rows[k0 + k];
+        f[k] = w[k0 + k];
+        if (r >= 0) {
+          v[k] = *reinterpret_cast<const float4*>(y + (size_t)r * hidden + i);
+        } else {
+          const T* xr = x + (size_t)t * hidden + i;
+          v[k] = make_float4(Num<T>::to_f(xr[0]), Num<T>::to_f(xr[1]), Num<T>::to_f(xr[2]), Num<T>::to_f(xr[3]));
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < AHEAD; ++k) {
+        acc.x = fmaf(f[k], v[k].x, acc.x); acc.y = fmaf(f[k], v[k].y, acc.y);
+        acc.z = fmaf(f[k], v[k].z, acc.z); acc.w = fmaf(f[k], v[k].w, acc.w);
+      }
+    }
+    *reinterpret_cast<float4*>(out + (size_t)t * hidden + i) = acc;
+  }
+}
+
+template <typename T>
+int launch_combine(const float* y, const int* pair_row, const float* weights, const void* x, float* out, int n_tokens, int hidden,
+                   int top, cudaStream_t stream) {
+  if (!(hidden & 3) && !(((uintptr_t)y | (uintptr_t)out) & 15)) {
+    const int quads = hidden / 4;
+    return launch_pdl(moe_combine_vec_kernel<T>, dim3(n_tokens), dim3(quads >= 256 ? 256 : quads >= 128 ? 128 : 64), 0, stream, y, pair_row,
+                      weights, (const T*)x, out, hidden, top);
+  }
+  return launch_pdl(moe_combine_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, y, pair_row, weights, (const T*)x, out, hidden, top);
+}
+
+// act: MODE_SWIGLU or MODE_CLAMPED (w_up = [gate rows; up rows] of every expert) or MODE_RELU2 (w_up = up rows alone)
 int launch_products_mma(const void* x, const void* w_up, const void* w_down, const int* tile_expert, const int* sorted_pair,
-                        void* act_out, float* y, int max_tiles, int hidden, int ff, int top, int act, cudaStream_t stream) {
-  int rc = act == MODE_SWIGLU
-      ? launch_pdl(moe_product_mma_kernel<bf16, MODE_SWIGLU>, dim3((ff + 31) / 32, max_tiles), dim3(128), 0, stream,
-                   (const bf16*)x, (long long)hidden, top, (const bf16*)w_up, tile_expert, sorted_pair, (bf16*)act_out,
-                   (long long)ff, ff, hidden)
-      : launch_pdl(moe_product_mma_kernel<bf16, MODE_RELU2>, dim3((ff + 63) / 64, max_tiles), dim3(128), 0, stream,
-                   (const bf16*)x, (long long)hidden, top, (const bf16*)w_up, tile_expert, sorted_pair, (bf16*)act_out,
-                   (long long)ff, ff, hidden);
+                        void* act_out, float* y, int max_tiles, int hidden, int ff, int top, int act, GluShape shape,
+                        cudaStream_t stream) {
+  const bool gated = act != MODE_RELU2;
+  auto up = act == MODE_SWIGLU ? moe_product_mma_kernel<bf16, MODE_SWIGLU>
+            : act == MODE_CLAMPED ? moe_product_mma_kernel<bf16, MODE_CLAMPED> : moe_product_mma_kernel<bf16, MODE_RELU2>;
+  int rc = launch_pdl(up, dim3(gated ? (ff + 31) / 32 : (ff + 63) / 64, max_tiles), dim3(128), 0, stream, (const bf16*)x,
+                      (long long)hidden, top, (const bf16*)w_up, tile_expert, sorted_pair, (bf16*)act_out, (long long)ff, ff, hidden,
+                      shape);
   if (rc) return rc;
   return launch_pdl(moe_product_mma_kernel<float, MODE_PLAIN>, dim3((hidden + 63) / 64, max_tiles), dim3(128), 0, stream,
                     (const bf16*)act_out, (long long)ff, 0, (const bf16*)w_down, tile_expert, sorted_pair, y, (long long)hidden,
-                    hidden, ff);
+                    hidden, ff, shape);
 }
 
 template <typename T, int TM>
 int launch_products(const void* x, const void* w_up, const void* w_down, const int* tile_expert, const int* sorted_pair,
-                    void* act_out, float* y, int max_tiles, int hidden, int ff, int top, int act, cudaStream_t stream) {
-  int rc = act == MODE_SWIGLU
-      ? launch_pdl(moe_product_kernel<T, T, T, TM, MODE_SWIGLU>, dim3((ff + 31) / 32, max_tiles), dim3(256), 0, stream,
-                   (const T*)x, (long long)hidden, top, (const T*)w_up, tile_expert, sorted_pair, (T*)act_out,
-                   (long long)ff, ff, hidden)
-      : launch_pdl(moe_product_kernel<T, T, T, TM, MODE_RELU2>, dim3((ff + 63) / 64, max_tiles), dim3(256), 0, stream,
-                   (const T*)x, (long long)hidden, top, (const T*)w_up, tile_expert, sorted_pair, (T*)act_out,
-                   (long long)ff, ff, hidden);
+                    void* act_out, float* y, int max_tiles, int hidden, int ff, int top, int act, GluShape shape,
+                    cudaStream_t stream) {
+  const bool gated = act != MODE_RELU2;
+  auto up = act == MODE_SWIGLU ? moe_product_kernel<T, T, T, TM, MODE_SWIGLU>
+            : act == MODE_CLAMPED ? moe_product_kernel<T, T, T, TM, MODE_CLAMPED> : moe_product_kernel<T, T, T, TM, MODE_RELU2>;
+  int rc = launch_pdl(up, dim3(gated ? (ff + 31) / 32 : (ff + 63) / 64, max_tiles), dim3(256), 0, stream, (const T*)x,
+                      (long long)hidden, top, (const T*)w_up, tile_expert, sorted_pair, (T*)act_out, (long long)ff, ff, hidden, shape);
   if (rc) return rc;
   return launch_pdl(moe_product_kernel<T, T, float, TM, MODE_PLAIN>, dim3((hidden + 63) / 64, max_tiles), dim3(256), 0, stream,
                     (const T*)act_out, (long long)ff, 0, (const T*)w_down, tile_expert, sorted_pair, y, (long long)hidden,
-                    hidden, ff);
+                    hidden, ff, shape);
 }
 }  // namespace
 
@@ -352,21 +420,25 @@ IFX_API int ifx_moe_gather_rows(const void* x, int dtype, const int* sorted_pair
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
-IFX_API int ifx_moe_combine(const float* y, const int* pair_row, const float* weights, float* out, int n_tokens, int hidden,
-                            int top, cudaStream_t stream) {
+// x [N][hidden] of type x_dtype: what went in, for pairs without a row (null if there are none).
+IFX_API int ifx_moe_combine(const float* y, const int* pair_row, const float* weights, const void* x, int x_dtype, float* out,
+                            int n_tokens, int hidden, int top, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  const int rc = launch_pdl(moe_combine_kernel, dim3(n_tokens), dim3(256), 0, stream, y, pair_row, weights, out, hidden, top);
+  const int rc = x_dtype == IFX_BF16 ? launch_combine<bf16>(y, pair_row, weights, x, out, n_tokens, hidden, top, stream)
+                                     : launch_combine<float>(y, pair_row, weights, x, out, n_tokens, hidden, top, stream);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
 // over_all 0: weights are the softmax over the chosen logits alone; 1: the softmax over every expert's logit, the
-// chosen ones' scores divided by their sum (+ 1e-20).  Either is multiplied by scale.
-IFX_API int ifx_moe_route(const float* logits, int n_tokens, int experts, int top, int over_all, float scale, int* chosen,
-                          float* weights, cudaStream_t stream) {
+// chosen ones' scores divided by their sum (+ 1e-20).  Either is multiplied by scale.  correction (float32 [experts] or null;
+// with over_all): the choice goes by score + correction, the weights by the score.
+IFX_API int ifx_moe_route(const float* logits, int n_tokens, int experts, int top, int over_all, float scale,
+                          const float* correction, int* chosen, float* weights, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
+  if (correction && !over_all) return IFX_ERR_UNSUPPORTED;
   if (top < 1 || top > MAX_TOP || top > experts) return IFX_ERR_UNSUPPORTED;
   const int rc = launch_pdl(moe_route_kernel, dim3((n_tokens + 7) / 8), dim3(256), 0, stream, logits, n_tokens, experts, top,
-                            over_all, scale, chosen, weights);
+                            over_all, scale, correction, chosen, weights);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
@@ -374,34 +446,36 @@ IFX_API int ifx_moe_route(const float* logits, int n_tokens, int experts, int to
 IFX_API int ifx_moe_tile_rows(int pairs) { return pairs <= 256 ? 16 : 64; }
 
 // act 1: w_gate_up [experts][2 ff][hidden] and silu(gate) * up; act 2: w_gate_up [experts][ff][hidden] (up rows alone) and
-// relu(up)^2.
+// relu(up)^2; act 3: w_gate_up as for 1 and the clamped gated activation with limit, alpha and shift.  A choice of `experts`
+// or more is one of the identity.
 // x [N][hidden], w_gate_up [experts][2 ff][hidden], w_down [experts][hidden][ff] of one element type `dtype`;
 // act [max_tiles * tile][ff] of that type, y [max_tiles * tile][hidden] float32, out [N][hidden] float32.
 // max_tiles >= pairs / tile + experts, tile = ifx_moe_tile_rows(pairs).
 IFX_API int ifx_moe_experts(const void* x, int dtype, const void* w_gate_up, const void* w_down, const int* chosen,
-                            const float* weights, int n_tokens, int hidden, int ff, int experts, int top, int activation, int tile,
-                            int max_tiles, int* tile_expert, int* sorted_pair, int* pair_row, void* act, float* y,
+                            const float* weights, int n_tokens, int hidden, int ff, int experts, int top, int activation,
+                            float limit, float alpha, float shift, int tile, int max_tiles, int* tile_expert, int* sorted_pair, int* pair_row, void* act, float* y,
                             float* out, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   const int pairs = n_tokens * top;
   if ((tile != 16 && tile != 64) || max_tiles < pairs / tile + experts || experts > 4096) return IFX_ERR_UNSUPPORTED;
-  if (activation != MODE_SWIGLU && activation != MODE_RELU2) return IFX_ERR_UNSUPPORTED;
+  if (activation < MODE_SWIGLU || activation > MODE_CLAMPED) return IFX_ERR_UNSUPPORTED;
+  const GluShape shape{limit, alpha, shift};
   int rc = launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)3 * experts * sizeof(int), stream, chosen, pairs, experts,
                       tile, max_tiles, tile_expert, sorted_pair, pair_row);
   if (rc) return rc;
   if (dtype == IFX_F32)
-    rc = tile == 16 ? launch_products<float, 1>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, stream)
-                    : launch_products<float, 4>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, stream);
+    rc = tile == 16 ? launch_products<float, 1>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, shape, stream)
+                    : launch_products<float, 4>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, shape, stream);
   else if (dtype == IFX_BF16 && tile == 16 && hidden % 8 == 0 && ff % 8 == 0 &&
            (((uintptr_t)x | (uintptr_t)w_gate_up | (uintptr_t)w_down | (uintptr_t)act) & 15) == 0)
-    rc = launch_products_mma(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, stream);
+    rc = launch_products_mma(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, shape, stream);
   else if (dtype == IFX_BF16)
-    rc = tile == 16 ? launch_products<bf16, 1>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, stream)
-                    : launch_products<bf16, 4>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, stream);
+    rc = tile == 16 ? launch_products<bf16, 1>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, shape, stream)
+                    : launch_products<bf16, 4>(x, w_gate_up, w_down, tile_expert, sorted_pair, act, y, max_tiles, hidden, ff, top, activation, shape, stream);
   else
     return IFX_ERR_UNSUPPORTED;
   if (rc) return rc;
-  rc = launch_pdl(moe_combine_kernel, dim3(n_tokens), dim3(256), 0, stream, (const float*)y, (const int*)pair_row, weights, out,
-                  hidden, top);
+  rc = dtype == IFX_BF16 ? launch_combine<bf16>(y, pair_row, weights, x, out, n_tokens, hidden, top, stream)
+                         : launch_combine<float>(y, pair_row, weights, x, out, n_tokens, hidden, top, stream);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }

@@ -18,6 +18,15 @@
 //   3. every segment's outputs from its starting S                    (2 and 3: segment_scan.cuh)
 // The sums c are of numbers below zero, and only differences c_i - c_j with j <= i are raised to e, so nothing overflows.
 //
+// One decay per head and key channel (dec given: g_t is then a diagonal, g_t[d] = exp(-exp(A_log) softplus(dec_t[h][d] +
+// dt_bias[h][d])), and c_i a vector): the same equations with the exponentials inside the dot products,
+//
+//   L_ij = beta_i sum_d k_i[d] e^(c_i[d] - c_j[d]) k_j[d],   W = (I + L)^-1 diag(beta) (e^(c) K)
+//   S_n  = diag(e^(c_n)) S + sum_j (e^(c_n - c_j) k_j) u_j^T,   o_i = (e^(c_i) q_i)^T S + sum_j (q_i e^(c_i - c_j) k_j) u_j
+//
+// The differences are taken pair by pair and channel by channel, so decays of any strength stay finite here too.  The
+// first kernel leaves behind what the other two multiply: e^(c_n - c_j) k_j, e^(c_i) q_i, e^(c_n) and the scores' table.
+//
 // A step of single tokens runs one kernel: a block a (head, entry, 32 value columns), eight threads a column, the
 // column's state in registers between its read from the slot and its write.
 #include "segment_scan.cuh"
@@ -31,7 +40,8 @@ constexpr int LLD = SEG + 4;           // row length of L in shared memory
 struct GdArgs {
   const float* qkv; long long stride; int q_col, k_col, v_col;         // unit q (scaled) and k heads, v heads
   const float* raw; long long raw_stride; int a_col, b_col;            // the two raw projections, [row][heads] each
-  const float* a_log; const float* dt_bias;                            // [heads]
+  const float* dec; long long dec_stride;                              // or: the decays' projection, [row][heads * dim]
+  const float* a_log; const float* dt_bias;                            // [heads]; with dec: dt_bias [heads * dim]
   float* state;                                                        // [slots][heads][dim][vdim]
   const int* entry_q_start; const int* entry_q_len; const int* entry_slot;
   const int* seg_entry; const int* seg_t0; const int* entry_first_seg;
@@ -39,12 +49,15 @@ struct GdArgs {
   float* w_rows;                                                       // [row][heads * dim]
   float* u_rows;                                                       // [row][heads * vdim]
   float* cum;                                                          // [row][heads]
+  float* k_rows; float* q_rows;                                        // with dec: [row][heads * dim] each
+  float* seg_decay;                                                    // with dec: [segments][heads][dim]
+  float* scores;                                                       // with dec: [segments][heads][SEG j][SEG i]
   float* out;                                                          // [row][heads * vdim]
 };
 
+__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float log_decay(const GdArgs& p, int row, int h) {
-  const float x = p.raw[(size_t)row * p.raw_stride + p.a_col + h] + p.dt_bias[h];
-  return -expf(p.a_log[h]) * (fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))));
+  return -expf(p.a_log[h]) * softplus(p.raw[(size_t)row * p.raw_stride + p.a_col + h] + p.dt_bias[h]);
 }
 __device__ __forceinline__ float write_rate(const GdArgs& p, int row, int h) {
   return 1.0f / (1.0f + expf(-p.raw[(size_t)row * p.raw_stride + p.b_col + h]));
@@ -60,6 +73,23 @@ __device__ __forceinline__ void dots_2x2(const float* a, int a_ld, const float* 
     d[0][1] = fmaf(a0.x, b1.x, fmaf(a0.y, b1.y, fmaf(a0.z, b1.z, fmaf(a0.w, b1.w, d[0][1]))));
     d[1][0] = fmaf(a1.x, b0.x, fmaf(a1.y, b0.y, fmaf(a1.z, b0.z, fmaf(a1.w, b0.w, d[1][0]))));
     d[1][1] = fmaf(a1.x, b1.x, fmaf(a1.y, b1.y, fmaf(a1.z, b1.z, fmaf(a1.w, b1.w, d[1][1]))));
+  }
+}
+
+// x <- (I + L)^-1 x for a thread's column of SEG numbers; L zero from the diagonal on, rows LLD apart
+__device__ __forceinline__ void solve_column(const float* L, float (&x)[SEG]) {
+#pragma unroll
+  for (int i = 0; i < SEG; ++i) {
+    float s0 = 0.0f, s1 = 0.0f;
+#pragma unroll
+    for (int j = 0; j < i; j += 4) {       // a group of four may reach past the diagonal
+      const float4 l = *reinterpret_cast<const float4*>(L + i * LLD + j);
+      s0 = fmaf(l.x, x[j], s0);
+      if (j + 1 < i) s1 = fmaf(l.y, x[j + 1], s1);
+      if (j + 2 < i) s0 = fmaf(l.z, x[j + 2], s0);
+      if (j + 3 < i) s1 = fmaf(l.w, x[j + 3], s1);
+    }
+    x[i] -= s0 + s1;
   }
 }
 
@@ -121,19 +151,7 @@ gated_delta_segments_kernel(GdArgs p) {
     }
     float* dst = c < D ? p.w_rows + (size_t)row0 * p.heads * D + h * D + c : p.u_rows + (size_t)row0 * p.heads * V + h * V + (c - D);
     const size_t step = (size_t)p.heads * (c < D ? D : V);
-#pragma unroll
-    for (int i = 0; i < SEG; ++i) {
-      float s0 = 0.0f, s1 = 0.0f;
-#pragma unroll
-      for (int j = 0; j < i; j += 4) {     // L is zero from the diagonal on, so a group of four may reach past it
-        const float4 l = *reinterpret_cast<const float4*>(L + i * LLD + j);
-        s0 = fmaf(l.x, x[j], s0);
-        if (j + 1 < i) s1 = fmaf(l.y, x[j + 1], s1);
-        if (j + 2 < i) s0 = fmaf(l.z, x[j + 2], s0);
-        if (j + 3 < i) s1 = fmaf(l.w, x[j + 3], s1);
-      }
-      x[i] -= s0 + s1;
-    }
+    solve_column(L, x);
 #pragma unroll
     for (int i = 0; i < SEG; ++i)
       if (i < n) dst[(size_t)i * step] = x[i];
@@ -141,10 +159,10 @@ gated_delta_segments_kernel(GdArgs p) {
 }
 
 // Single tokens: NI key rows a thread, g + 8 i of the block's head.
-template <int NI>
+template <int NI, bool CHANNEL>
 __global__ void __launch_bounds__(256)
 gated_delta_step_kernel(GdArgs p) {
-  __shared__ float ks[8 * NI], qs[8 * NI], red[8][33];
+  __shared__ float ks[8 * NI], qs[8 * NI], gs[CHANNEL ? 8 * NI : 1], red[8][33];
   pdl_enter();
   const int h = blockIdx.x, e = blockIdx.y, tid = threadIdx.x, lane = tid & 31, grp = tid >> 5;
   const int c = blockIdx.z * 32 + lane, D = p.dim, V = p.vdim;
@@ -161,14 +179,16 @@ gated_delta_step_kernel(GdArgs p) {
   for (int d = tid; d < 8 * NI; d += 256) {
     ks[d] = d < D ? r[p.k_col + kvh * D + d] : 0.0f;
     qs[d] = d < D ? r[p.q_col + kvh * D + d] : 0.0f;
+    if (CHANNEL)
+      gs[d] = d < D ? expf(-expf(p.a_log[h]) * softplus(p.dec[(size_t)row * p.dec_stride + h * D + d] + p.dt_bias[h * D + d])) : 0.0f;
   }
   const float v = on ? r[p.v_col + h * V + c] : 0.0f;
-  const float g = expf(log_decay(p, row, h)), beta = write_rate(p, row, h);
+  const float g = CHANNEL ? 1.0f : expf(log_decay(p, row, h)), beta = write_rate(p, row, h);
   __syncthreads();
   float dot = 0.0f;
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
-    S[i] *= g;
+    S[i] *= CHANNEL ? gs[grp + 8 * i] : g;
     dot = fmaf(ks[grp + 8 * i], S[i], dot);
   }
   red[grp][lane] = dot;
@@ -196,6 +216,117 @@ gated_delta_step_kernel(GdArgs p) {
   }
 }
 
+// One decay per key channel.  The logarithms' running sums are kept to base two.
+__global__ void __launch_bounds__(THREADS, 2)
+channel_delta_segments_kernel(GdArgs p) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_enter();
+  const int D = p.dim, V = p.vdim, DP = segscan::pad4(D), LD = row_ld(D);
+  float* ks = sm;                          // [SEG][LD]
+  float* qs = ks + SEG * LD;               // [SEG][LD]
+  float* cs = qs + SEG * LD;               // [SEG][LD] running sums of log2 g per channel
+  float* L = cs + SEG * LD;                // [SEG][LLD]
+  float* A = L + SEG * LLD;                // [SEG j][LLD] scores, transposed
+  float* be = A + SEG * LLD;               // [SEG] beta
+  const int seg = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int e = p.seg_entry[seg], t0 = p.seg_t0[seg];
+  const int n = min(SEG, p.entry_q_len[e] - t0), row0 = p.entry_q_start[e] + t0;
+  const int kvh = h / (p.heads / p.kv_heads);
+  segscan::stage_rows(ks, LD, DP, p.qkv + (size_t)row0 * p.stride + p.k_col + kvh * D, p.stride, n, D, p.vec, tid, THREADS);
+  segscan::stage_rows(qs, LD, DP, p.qkv + (size_t)row0 * p.stride + p.q_col + kvh * D, p.stride, n, D, p.vec, tid, THREADS);
+  cp_async_commit();
+  {
+    const float rate = -1.4426950408889634f * expf(p.a_log[h]);
+    const float* dec = p.dec + (size_t)row0 * p.dec_stride + h * D;
+    const float* bias = p.dt_bias + h * D;
+    for (int i = tid >> 5; i < SEG; i += THREADS / 32)
+      for (int d = tid & 31; d < DP; d += 32)
+        cs[i * LD + d] = i < n && d < D ? rate * softplus(dec[(size_t)i * p.dec_stride + d] + bias[d]) : 0.0f;
+  }
+  if (tid < SEG) be[tid] = tid < n ? write_rate(p, row0 + tid, h) : 0.0f;
+  for (int idx = tid; idx < SEG * LLD; idx += THREADS) L[idx] = A[idx] = 0.0f;
+  __syncthreads();
+  for (int d = tid; d < DP; d += THREADS) {
+    float c = 0.0f;
+#pragma unroll
+    for (int i = 0; i < SEG; ++i) {
+      c += cs[i * LD + d];
+      cs[i * LD + d] = c;
+    }
+  }
+  cp_async_wait_all();
+  __syncthreads();
+  {
+    // rows bi and 31 - bi with columns bj and 16 + bj, as far as the column is not behind the row
+    const int bi = tid >> 4, bj = tid & 15, i0 = bi, i1 = SEG - 1 - bi, j0 = bj, j1 = bj + 16;
+    const bool low = j0 <= i0, high = j1 <= i1;
+    float kk[3] = {}, qk[3] = {};          // (i1, j0), (i0, j0), (i1, j1)
+    auto pair = [](float4 k, float4 q, float4 c, float4 kj, float4 cj, float& sk, float& sq) {
+      float t;
+      t = kj.x * exp2f(c.x - cj.x); sk = fmaf(k.x, t, sk); sq = fmaf(q.x, t, sq);
+      t = kj.y * exp2f(c.y - cj.y); sk = fmaf(k.y, t, sk); sq = fmaf(q.y, t, sq);
+      t = kj.z * exp2f(c.z - cj.z); sk = fmaf(k.z, t, sk); sq = fmaf(q.z, t, sq);
+      t = kj.w * exp2f(c.w - cj.w); sk = fmaf(k.w, t, sk); sq = fmaf(q.w, t, sq);
+    };
+#pragma unroll 1
+    for (int d = 0; d < DP; d += 4) {
+      auto at = [&](const float* b, int i) { return *reinterpret_cast<const float4*>(b + i * LD + d); };
+      const float4 k1 = at(ks, i1), q1 = at(qs, i1), c1 = at(cs, i1), kj = at(ks, j0), cj = at(cs, j0);
+      pair(k1, q1, c1, kj, cj, kk[0], qk[0]);
+      if (low) pair(at(ks, i0), at(qs, i0), at(cs, i0), kj, cj, kk[1], qk[1]);
+      if (high) pair(k1, q1, c1, at(ks, j1), at(cs, j1), kk[2], qk[2]);
+    }
+    L[i1 * LLD + j0] = be[i1] * kk[0];     // i1 >= 16 > j0
+    A[j0 * LLD + i1] = qk[0];
+    if (low) {
+      if (j0 < i0) L[i0 * LLD + j0] = be[i0] * kk[1];
+      A[j0 * LLD + i0] = qk[1];
+    }
+    if (high) {
+      if (j1 < i1) L[i1 * LLD + j1] = be[i1] * kk[2];
+      A[j1 * LLD + i1] = qk[2];
+    }
+  }
+  __syncthreads();
+  {
+    float* dst = p.scores + ((size_t)seg * p.heads + h) * SEG * SEG;
+    const int j = tid >> 3, i = 4 * (tid & 7);
+    *reinterpret_cast<float4*>(dst + j * SEG + i) = *reinterpret_cast<const float4*>(A + j * LLD + i);
+  }
+  for (int c = tid; c < D + V; c += THREADS) {
+    float x[SEG];
+    if (c < D) {
+      // this channel's keys and queries with their decays, and what is left of the state at the segment's end
+      const float last = cs[(n - 1) * LD + c];
+      float* kr = p.k_rows + ((size_t)row0 * p.heads + h) * D + c;
+      float* qr = p.q_rows + ((size_t)row0 * p.heads + h) * D + c;
+      p.seg_decay[((size_t)seg * p.heads + h) * D + c] = exp2f(last);
+#pragma unroll
+      for (int i = 0; i < SEG; ++i) {
+        const float ci = cs[i * LD + c], k = ks[i * LD + c], g = exp2f(ci);
+        x[i] = be[i] * g * k;
+        if (i < n) {
+          kr[(size_t)i * p.heads * D] = exp2f(last - ci) * k;
+          qr[(size_t)i * p.heads * D] = g * qs[i * LD + c];
+        }
+      }
+    } else {
+      const float* v = p.qkv + (size_t)row0 * p.stride + p.v_col + h * V + (c - D);
+#pragma unroll
+      for (int i = 0; i < SEG; ++i) x[i] = i < n ? v[(size_t)i * p.stride] : 0.0f;
+#pragma unroll
+      for (int i = 0; i < SEG; ++i) x[i] *= be[i];
+    }
+    float* dst = c < D ? p.w_rows + (size_t)row0 * p.heads * D + h * D + c : p.u_rows + (size_t)row0 * p.heads * V + h * V + (c - D);
+    const size_t step = (size_t)p.heads * (c < D ? D : V);
+    solve_column(L, x);
+#pragma unroll
+    for (int i = 0; i < SEG; ++i)
+      if (i < n) dst[(size_t)i * step] = x[i];
+  }
+}
+
+size_t channel_segments_smem(int D) { return ((size_t)3 * SEG * row_ld(D) + 2 * SEG * LLD + SEG) * sizeof(float); }
 size_t segments_smem(int D) { return ((size_t)SEG * row_ld(D) + SEG * LLD + 3 * SEG) * sizeof(float); }
 }  // namespace
 
@@ -206,33 +337,44 @@ IFX_API int ifx_gated_delta_segment() { return SEG; }
 // state float32 [slots][heads][dim][vdim]; out float32 [N][heads * vdim].  n_segments 0: every entry brings one token.
 // Otherwise w_rows [N][heads * dim], u_rows [N][heads * vdim], cum [N][heads] and seg_start [segments][heads][dim][vdim]
 // (float32) are scratch, and the segments of ifx_gated_delta_segment() tokens are listed entry by entry.
+// dec (or null): float32 rows of heads * dim, the projection of one decay per head and key channel; raw's a_col is not
+// read then, dt_bias is [heads * dim], and k_rows, q_rows [N][heads * dim], seg_decay [segments][heads][dim] and scores
+// [segments][heads][32][32] are scratch in cum's place.
 IFX_API int ifx_gated_delta_scan(const float* qkv, long long stride, int q_col, int k_col, int v_col, const float* raw,
-                                 long long raw_stride, int a_col, int b_col, const float* a_log, const float* dt_bias,
+                                 long long raw_stride, int a_col, int b_col, const float* dec, long long dec_stride,
+                                 const float* a_log, const float* dt_bias,
                                  float* state, const int* entry_q_start, const int* entry_q_len, const int* entry_slot,
                                  int n_entries, const int* seg_entry, const int* seg_t0, const int* entry_first_seg,
-                                 int n_segments, float* w_rows, float* u_rows, float* cum, float* seg_start, float* out,
-                                 int heads, int kv_heads, int dim, int vdim, cudaStream_t stream) {
+                                 int n_segments, float* w_rows, float* u_rows, float* cum, float* k_rows, float* q_rows,
+                                 float* seg_decay, float* scores, float* seg_start, float* out, int heads, int kv_heads, int dim, int vdim, cudaStream_t stream) {
   if (n_entries <= 0) return 0;
   if (heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || dim > segscan::MAX_DIM || vdim < 1 || heads > 65535 || n_entries > 65535)
     return IFX_ERR_UNSUPPORTED;
-  GdArgs p{qkv, stride, q_col, k_col, v_col, raw, raw_stride, a_col, b_col, a_log, dt_bias, state, entry_q_start, entry_q_len,
-           entry_slot, seg_entry, seg_t0, entry_first_seg, heads, kv_heads, dim, vdim, 0, w_rows, u_rows, cum, out};
+  GdArgs p{qkv, stride, q_col, k_col, v_col, raw, raw_stride, a_col, b_col, dec, dec_stride, a_log, dt_bias, state, entry_q_start,
+           entry_q_len, entry_slot, seg_entry, seg_t0, entry_first_seg, heads, kv_heads, dim, vdim, 0, w_rows, u_rows, cum, k_rows,
+           q_rows, seg_decay, scores, out};
   p.vec = !((dim | vdim | q_col | k_col | v_col) & 3) && !(stride & 3) &&
-          !(((uintptr_t)qkv | (uintptr_t)w_rows | (uintptr_t)u_rows | (uintptr_t)seg_start) & 15);
+          !(((uintptr_t)qkv | (uintptr_t)w_rows | (uintptr_t)u_rows | (uintptr_t)seg_start | (uintptr_t)k_rows | (uintptr_t)q_rows) & 15);
   int rc;
   if (n_segments <= 0) {
     const dim3 grid(heads, n_entries, (vdim + 31) / 32);
-    if (dim <= 32) rc = launch_pdl(gated_delta_step_kernel<4>, grid, dim3(256), 0, stream, p);
-    else if (dim <= 64) rc = launch_pdl(gated_delta_step_kernel<8>, grid, dim3(256), 0, stream, p);
-    else if (dim <= 128) rc = launch_pdl(gated_delta_step_kernel<16>, grid, dim3(256), 0, stream, p);
-    else rc = launch_pdl(gated_delta_step_kernel<32>, grid, dim3(256), 0, stream, p);
+    auto kern = dec ? (dim <= 32 ? gated_delta_step_kernel<4, true> : dim <= 64 ? gated_delta_step_kernel<8, true>
+                       : dim <= 128 ? gated_delta_step_kernel<16, true> : gated_delta_step_kernel<32, true>)
+                    : (dim <= 32 ? gated_delta_step_kernel<4, false> : dim <= 64 ? gated_delta_step_kernel<8, false>
+                       : dim <= 128 ? gated_delta_step_kernel<16, false> : gated_delta_step_kernel<32, false>);
+    rc = launch_pdl(kern, grid, dim3(256), 0, stream, p);
     return rc ? rc : IFX_LAUNCH_CHECK();
   }
-  if (!w_rows || !u_rows || !cum || !seg_start) return IFX_ERR_UNSUPPORTED;
-  rc = segscan::allow_smem(gated_delta_segments_kernel, segments_smem(dim));
-  if (rc) return rc;
-  rc = launch_pdl(gated_delta_segments_kernel, dim3(n_segments, heads), dim3(THREADS), segments_smem(dim), stream, p);
-  if (rc) return rc;
+  if (!w_rows || !u_rows || !seg_start) return IFX_ERR_UNSUPPORTED;
+  if (dec ? !k_rows || !q_rows || !seg_decay || !scores || ((uintptr_t)scores & 15) : !cum) return IFX_ERR_UNSUPPORTED;
+  {
+    auto kern = dec ? channel_delta_segments_kernel : gated_delta_segments_kernel;
+    const size_t smem = dec ? channel_segments_smem(dim) : segments_smem(dim);
+    rc = segscan::allow_smem(kern, smem);
+    if (rc) return rc;
+    rc = launch_pdl(kern, dim3(n_segments, heads), dim3(THREADS), smem, stream, p);
+    if (rc) return rc;
+  }
   segscan::Args a{};
   a.q = qkv + q_col; a.k = qkv + k_col; a.qk_stride = stride; a.share = heads / kv_heads; a.k_scale = 1.0f;
   a.v = u_rows; a.v_stride = (long long)heads * vdim;
@@ -241,6 +383,12 @@ IFX_API int ifx_gated_delta_scan(const float* qkv, long long stride, int q_col, 
   a.seg_entry = seg_entry; a.seg_t0 = seg_t0; a.entry_first_seg = entry_first_seg;
   a.seg_start = seg_start; a.out = out; a.heads = heads; a.dim = dim; a.vdim = vdim;
   a.vec = p.vec && !((uintptr_t)out & 15);
+  if (dec) {
+    a.q = q_rows; a.k = k_rows; a.qk_stride = (long long)heads * dim; a.share = 1;
+    a.seg_decay = seg_decay; a.scores = scores;
+    rc = segscan::launch<false, true, true>(a, n_entries, n_segments, stream);
+    return rc ? rc : IFX_LAUNCH_CHECK();
+  }
   rc = segscan::launch<false, true>(a, n_entries, n_segments, stream);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }

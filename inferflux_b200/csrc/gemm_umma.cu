@@ -164,7 +164,7 @@ struct QkvEpilogue {
   int page_size, page_shift, n_heads, n_kv;
 };
 
-// MODE 0: out = A W^T (+ bias) (4: relu(.)^2 of it); 1: SwiGLU of the two halves of W; 2: few rows of A; 3: q, k, v with bias,
+// MODE 0: out = A W^T (+ bias) (4: relu(.)^2 of it); 1: SwiGLU of the two halves of W (5: the clamped gated activation `glu` of them); 2: few rows of A; 3: q, k, v with bias,
 // rotation and cache write (tiles of two heads of 128).  In mode 2 the operands
 // change places, so that the 256 rows of a tile are rows of the weights and its (few) columns the tokens: the
 // kernel is given the weights as map_a (M = their rows) and the activations as map_w (n_out = the tokens, all
@@ -175,11 +175,11 @@ __global__ void __launch_bounds__(P_THREADS, 1)
 gemm_umma_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                       TOut* __restrict__ out, long long ldo, const float* __restrict__ bias, int M, int n_out, int K,
                       int tile_n, int* __restrict__ error_flag, int k_parts, long long part_stride, QkvEpilogue qe,
-                      const int* __restrict__ tile_expert, int expert_rows) {
-  // tile_expert (modes 0 and 1, or null): the rows of A are sorted by expert into groups of 256, tile_expert[i]
+                      const int* __restrict__ tile_expert, int expert_rows, GluShape glu) {
+  // tile_expert (modes 0, 1, 4 and 5, or null): the rows of A are sorted by expert into groups of 256, tile_expert[i]
   // names the expert whose weights row tile i multiplies (its rows of W start at expert * expert_rows) or is
   // negative for a row tile that is not in use, which every role of the kernel skips.
-  constexpr bool SWIGLU = MODE == 1, SKINNY = MODE == 2, QKV = MODE == 3, RELU2 = MODE == 4;
+  constexpr bool SWIGLU = MODE == 1 || MODE == 5, SKINNY = MODE == 2, QKV = MODE == 3, RELU2 = MODE == 4;
   pdl_enter();
   extern __shared__ unsigned char g_smem_raw[];
   __shared__ __align__(8) unsigned long long bars[2 * P_STAGES + 4];    // full[s], empty[s], acc_full[2], acc_empty[2]
@@ -388,7 +388,14 @@ gemm_umma_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
           g_tmem_ld32(taddr + c * 32, gate);
           g_tmem_ld32(taddr + 128 + c * 32, up);
 #pragma unroll
-          for (int i = 0; i < 32; ++i) gate[i] = gate[i] / (1.0f + __expf(-gate[i])) * up[i];
+          for (int i = 0; i < 32; ++i) {
+            if (MODE == 5) {
+              const float g = fminf(gate[i], glu.limit), u = fminf(fmaxf(up[i], -glu.limit), glu.limit);
+              gate[i] = g / (1.0f + __expf(-glu.alpha * g)) * (u + glu.shift);
+            } else {
+              gate[i] = gate[i] / (1.0f + __expf(-gate[i])) * up[i];
+            }
+          }
           const int col = n0 + c * 32;
           if (row < M && col < n_out) store_row32<TOut>(orow + col, gate, min(32, n_out - col), vec && (col % 8 == 0));
         }
@@ -489,7 +496,7 @@ int launch_gemm_pair(const void* A, long long lda, const void* W, const float* b
   const int tiles = ((M + 255) / 256) * ((n_out + out_cols - 1) / out_cols);
   const int pairs = tiles < sms / 2 ? tiles : sms / 2;
   rc = launch_pdl_cluster(kern, dim3(2 * pairs), dim3(P_THREADS), (size_t)P_SMEM, stream, dim3(2, 1, 1), map_a, map_w, (TOut*)out,
-                          ldo, bias, M, n_out, K, tile_n, error_flag, 1, 0ll, QkvEpilogue{}, (const int*)nullptr, 0);
+                          ldo, bias, M, n_out, K, tile_n, error_flag, 1, 0ll, QkvEpilogue{}, (const int*)nullptr, 0, GluShape{});
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
@@ -497,8 +504,8 @@ int launch_gemm_pair(const void* A, long long lda, const void* W, const float* b
 // expert tile_expert[i] (W is [experts][n_out or 2 n_out][K] as one matrix) or is skipped when that is negative.
 template <int MODE, typename TOut>
 int launch_gemm_grouped(const void* A, long long lda, const void* W, void* out, long long ldo, int M, int n_out, int K,
-                        int experts, const int* tile_expert, int* error_flag, cudaStream_t stream) {
-  constexpr bool SWIGLU = MODE == 1;
+                        int experts, const int* tile_expert, GluShape glu, int* error_flag, cudaStream_t stream) {
+  constexpr bool SWIGLU = MODE == 1 || MODE == 5;
   auto kern = gemm_umma_pair_kernel<MODE, TOut>;
   static int sms = 0;
   if (!sms) {
@@ -518,7 +525,7 @@ int launch_gemm_grouped(const void* A, long long lda, const void* W, void* out, 
   const int tiles = ((M + 255) / 256) * ((n_out + out_cols - 1) / out_cols);
   const int pairs = tiles < sms / 2 ? tiles : sms / 2;
   rc = launch_pdl_cluster(kern, dim3(2 * pairs), dim3(P_THREADS), (size_t)P_SMEM, stream, dim3(2, 1, 1), map_a, map_w, (TOut*)out,
-                          ldo, (const float*)nullptr, M, n_out, K, tile_n, error_flag, 1, 0ll, QkvEpilogue{}, tile_expert, expert_rows);
+                          ldo, (const float*)nullptr, M, n_out, K, tile_n, error_flag, 1, 0ll, QkvEpilogue{}, tile_expert, expert_rows, glu);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
@@ -565,7 +572,7 @@ int launch_gemm_qkv(const void* A, long long lda, const void* W, const float* bi
   const int tiles = ((M + 255) / 256) * ((n_out + tile_n - 1) / tile_n);
   const int pairs = tiles < sms / 2 ? tiles : sms / 2;
   rc = launch_pdl_cluster(kern, dim3(2 * pairs), dim3(P_THREADS), (size_t)P_SMEM, stream, dim3(2, 1, 1), map_a, map_w, q_out,
-                          ldo, bias, M, n_out, K, tile_n, error_flag, 1, 0ll, qe, (const int*)nullptr, 0);
+                          ldo, bias, M, n_out, K, tile_n, error_flag, 1, 0ll, qe, (const int*)nullptr, 0, GluShape{});
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
@@ -589,7 +596,7 @@ int launch_gemm_skinny(const void* X, long long ldx, const void* W, float* out, 
   const int tiles = ((n_out + 255) / 256) * k_parts;
   const int pairs = tiles < sms / 2 ? tiles : sms / 2;
   rc = launch_pdl_cluster(kern, dim3(2 * pairs), dim3(P_THREADS), (size_t)P_SMEM, stream, dim3(2, 1, 1), map_w, map_x, out, ldo,
-                          (const float*)nullptr, n_out, tokens, K, tile_n, error_flag, k_parts, part_stride, QkvEpilogue{}, (const int*)nullptr, 0);
+                          (const float*)nullptr, n_out, tokens, K, tile_n, error_flag, k_parts, part_stride, QkvEpilogue{}, (const int*)nullptr, 0, GluShape{});
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 }  // namespace
@@ -633,20 +640,22 @@ IFX_API int ifx_gemm_umma_skinny(const void* X, long long ldx, const void* W, fl
 // tile_expert[row / 256], rows of unused groups (negative) untouched.  act 1: W_e = [gate rows; up rows],
 // out = silu(gate) * up in bfloat16; act 2: out = relu(sum)^2 in bfloat16; act 0: the sums, float32 or bfloat16 by out_dtype.
 IFX_API int ifx_gemm_umma_grouped(const void* A, long long lda, const void* W, void* out, long long ldo, int out_dtype,
-                                  int M, int n_out, int K, int act, int experts, const int* tile_expert,
-                                  int* error_flag, cudaStream_t stream) {
+                                  int M, int n_out, int K, int act, float limit, float alpha, float shift, int experts,
+                                  const int* tile_expert, int* error_flag, cudaStream_t stream) {
   if (M <= 0 || n_out <= 0) return 0;
-  if (K <= 0 || (K % 8) || (lda % 8) || (M % 256) || experts < 1 || !tile_expert || act < 0 || act > 2) return IFX_ERR_UNSUPPORTED;
+  if (K <= 0 || (K % 8) || (lda % 8) || (M % 256) || experts < 1 || !tile_expert || act < 0 || act > 3) return IFX_ERR_UNSUPPORTED;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return IFX_ERR_ALIGNMENT;
+  const GluShape glu{limit, alpha, shift};
   if (act) {
     if (out_dtype != IFX_BF16) return IFX_ERR_UNSUPPORTED;
-    return act == 1 ? launch_gemm_grouped<1, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, error_flag, stream)
-                    : launch_gemm_grouped<4, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, error_flag, stream);
+    return act == 1 ? launch_gemm_grouped<1, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, glu, error_flag, stream)
+         : act == 2 ? launch_gemm_grouped<4, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, glu, error_flag, stream)
+                    : launch_gemm_grouped<5, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, glu, error_flag, stream);
   }
   if (out_dtype == IFX_BF16)
-    return launch_gemm_grouped<0, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, error_flag, stream);
+    return launch_gemm_grouped<0, bf16>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, glu, error_flag, stream);
   if (out_dtype == IFX_F32)
-    return launch_gemm_grouped<0, float>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, error_flag, stream);
+    return launch_gemm_grouped<0, float>(A, lda, W, out, ldo, M, n_out, K, experts, tile_expert, glu, error_flag, stream);
   return IFX_ERR_UNSUPPORTED;
 }
 

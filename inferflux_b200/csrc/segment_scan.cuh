@@ -5,9 +5,12 @@
 //   o_i   = G_i S^T q_i + sum_{j <= i} (G_i / G_j) (q_i . k_j) u_j        tokens of a segment: one kernel over all segments
 //   S_end = G_n S + sum_j (G_n / G_j) k_j u_j^T                           segment after segment: one kernel that carries S
 //
-// Two mixers share the two kernels below.  Where the decay is one number per head (FIXED) its powers come as a table and
+// Three mixers share the two kernels below.  Where the decay is one number per head (FIXED) its powers come as a table and
 // u is the value itself.  Otherwise the decays come as running sums of logarithms from the segment's start, and with
-// SOLVE u = U - W S, with U and W worked out beforehand for all segments at once.
+// SOLVE u = U - W S, with U and W worked out beforehand for all segments at once.  Where there is a decay per key channel
+// (CHANNEL, with SOLVE; G_i is then a diagonal) all that meets it has been worked out beforehand too: the keys come times
+// what is left of them at the segment's end, the queries times G_i, the scores (G_i / G_j) (q_i . k_j) as a table of their
+// own, and G_n row by row.
 //
 // The carry: a block a (head, entry, VC value columns).  256 threads own the state in registers, a thread four
 // neighbouring rows (every 128 of them) of VC / 8 columns; 128 more keep the copies of the next segments' rows into a
@@ -33,6 +36,8 @@ struct Args {
   float k_scale;                                         // keys count so many times
   const float* powers;                                   // FIXED: [heads][SEG + 1] powers of the head's decay
   const float* cum;                                      // else: [row][heads] running sums of ln g from the segment's start
+  const float* seg_decay;                                // CHANNEL: [segments][heads][dim] G_n
+  const float* scores;                                   // CHANNEL: [segments][heads][SEG j][SEG i], zero for j > i
   const float* w_rows; float* u_rows;                    // SOLVE: [row][heads * dim], [row][heads * vdim] (U in, u out)
   float* state;                                          // [slots][heads][dim][vdim]
   const int* entry_q_start; const int* entry_q_len; const int* entry_slot;
@@ -90,24 +95,26 @@ __device__ __forceinline__ void stage_rows(float* dst, int ld, int fill, const f
   }
 }
 
-template <int VC> __host__ __device__ __forceinline__ int carry_buffer(int dim, bool solve) {
-  return SEG * row_ld(dim) + (solve ? SEG * row_ld(dim) : 0) + SEG * VC + SEG;
+// floats of a buffer that hold the decays: running sums, or (CHANNEL) one number per state row
+__host__ __device__ __forceinline__ int decay_floats(int dim, bool channel) { return channel ? row_ld(dim) : SEG; }
+template <int VC> __host__ __device__ __forceinline__ int carry_buffer(int dim, bool solve, bool channel) {
+  return SEG * row_ld(dim) + (solve ? SEG * row_ld(dim) : 0) + SEG * VC + decay_floats(dim, channel);
 }
-template <int VC, int NB> inline size_t carry_smem(int dim, bool solve) {
-  return ((solve ? VC * row_ld(dim) : 0) + SEG * VC + NB * (size_t)carry_buffer<VC>(dim, solve)) * sizeof(float);
+template <int VC, int NB> inline size_t carry_smem(int dim, bool solve, bool channel) {
+  return ((solve ? VC * row_ld(dim) : 0) + SEG * VC + NB * (size_t)carry_buffer<VC>(dim, solve, channel)) * sizeof(float);
 }
 
 // NR: blocks of 128 state rows (1: dim up to 128, 2: up to 256).  NB: segments the ring holds.
-template <bool FIXED, bool SOLVE, int VC, int NR, int NB>
+template <bool FIXED, bool SOLVE, bool CHANNEL, int VC, int NR, int NB>
 __global__ void __launch_bounds__(COMPUTE + HELPERS, 1)
 carry_kernel(Args p) {
   extern __shared__ __align__(16) float sm[];
   pdl_enter();
   constexpr int NC = VC / 8;
-  const int D = p.dim, V = p.vdim, DP = pad4(D), LD = row_ld(D), BUF = carry_buffer<VC>(D, SOLVE);
+  const int D = p.dim, V = p.vdim, DP = pad4(D), LD = row_ld(D), BUF = carry_buffer<VC>(D, SOLVE, CHANNEL), DEC = decay_floats(D, CHANNEL);
   float* us = sm;                         // [SEG][VC]: u, each times what is left of it at the segment's end
   float* St = us + SEG * VC;              // SOLVE: [VC][LD], the state's columns, rows side by side
-  float* bufs = St + (SOLVE ? VC * LD : 0);            // NB of: K [SEG][LD], values [SEG][VC], sums of ln g [SEG], W [SEG][LD]
+  float* bufs = St + (SOLVE ? VC * LD : 0);            // NB of: K [SEG][LD], values [SEG][VC], decays [DEC], W [SEG][LD]
   const int h = blockIdx.x, e = blockIdx.y, v0 = blockIdx.z * VC, tid = threadIdx.x;
   const int len = p.entry_q_len[e], r0 = p.entry_q_start[e];
   const int n_seg = (len + SEG - 1) / SEG, seg0 = p.entry_first_seg[e];
@@ -122,13 +129,20 @@ carry_kernel(Args p) {
       const int t0 = s * SEG, n = min(SEG, len - t0);
       stage_rows(buf, LD, DP, k + (size_t)t0 * p.qk_stride, p.qk_stride, n, D, p.vec, t, HELPERS);
       stage_rows(buf + SEG * LD, VC, VC, v + (size_t)t0 * vs, vs, n, vcols, p.vec, t, HELPERS);
-      if (!FIXED && t < SEG) {
+      if (CHANNEL) {
+        float* c = buf + SEG * LD + SEG * VC;
+        const float* g = p.seg_decay + ((size_t)(seg0 + s) * p.heads + h) * D;
+        for (int d = t; d < LD; d += HELPERS) {
+          if (d < D) cp_async_f32(c + d, g + d);
+          else c[d] = 0.0f;
+        }
+      } else if (!FIXED && t < SEG) {
         float* c = buf + SEG * LD + SEG * VC + t;
         if (t < n) cp_async_f32(c, p.cum + (size_t)(r0 + t0 + t) * p.heads + h);
         else *c = 0.0f;
       }
       if (SOLVE)
-        stage_rows(buf + SEG * LD + SEG * VC + SEG, LD, DP, p.w_rows + ((size_t)(r0 + t0) * p.heads + h) * D, (long long)p.heads * D, n, D,
+        stage_rows(buf + SEG * LD + SEG * VC + DEC, LD, DP, p.w_rows + ((size_t)(r0 + t0) * p.heads + h) * D, (long long)p.heads * D, n, D,
                    p.vec, t, HELPERS);
     };
     // a group of copies a segment, empty past the last one, so that NB - 2 groups behind a segment's may be under way
@@ -187,8 +201,10 @@ carry_kernel(Args p) {
     const float* cs = U + SEG * VC;
     const int n = min(SEG, len - s * SEG);
     __syncthreads();                      // this segment's rows are here and the state is shown
-    float total, left;
-    if (FIXED) {
+    float total = 0.0f, left;
+    if (CHANNEL) {
+      left = 1.0f;
+    } else if (FIXED) {
       total = pw[n];
       left = ur < n ? pw[n - 1 - ur] * p.k_scale : 0.0f;
     } else {
@@ -200,7 +216,7 @@ carry_kernel(Args p) {
 #pragma unroll
     for (int a = 0; a < NC; ++a) u[a] = U[ur * VC + uc + 8 * a];
     if (SOLVE) {
-      const float* W = cs + SEG + 4 * warp * LD + 4 * ks;
+      const float* W = cs + DEC + 4 * warp * LD + 4 * ks;
       const float* X = St + quad * LD + 4 * ks;
       float2 acc[NC][16] = {};            // [row][column], even and odd dimensions apart
 #pragma unroll 2
@@ -274,7 +290,7 @@ carry_kernel(Args p) {
           trade<8>(add[r][a], jq & 2, 4);
           trade<4>(add[r][a], jq & 1, 2);
 #pragma unroll
-          for (int x = 0; x < 4; ++x) S[r][a][x] = fmaf(total, S[r][a][x], add[r][a][x]);
+          for (int x = 0; x < 4; ++x) S[r][a][x] = fmaf(CHANNEL ? cs[k_at[r] + x] : total, S[r][a][x], add[r][a][x]);
         }
     }
     if (SOLVE) show();
@@ -290,8 +306,8 @@ carry_kernel(Args p) {
       }
 }
 
-template <int VT> inline size_t outputs_smem(int dim) {
-  const int dq = pad16(dim), kt = dq * SEG > 4 * SEG * SEG ? dq * SEG : 4 * SEG * SEG;
+template <int VT> inline size_t outputs_smem(int dim, bool channel) {
+  const int dq = pad16(dim), kt = channel ? SEG * SEG : dq * SEG > 4 * SEG * SEG ? dq * SEG : 4 * SEG * SEG;
   return ((size_t)dq * SEG + kt + (size_t)(dq + SEG) * VT + 2 * SEG + 1) * sizeof(float);
 }
 
@@ -309,7 +325,7 @@ __device__ __forceinline__ void stage_transposed(float* dst, const float* src, l
   }
 }
 
-template <bool FIXED, int VT>
+template <bool FIXED, bool CHANNEL, int VT>
 __global__ void __launch_bounds__(COMPUTE, 2)
 outputs_kernel(Args p) {
   extern __shared__ __align__(16) float sm[];
@@ -318,7 +334,7 @@ outputs_kernel(Args p) {
   const int D = p.dim, V = p.vdim, DQ = pad16(D);
   float* Qt = sm;                         // [DQ][SEG]
   float* Kt = Qt + DQ * SEG;              // [DQ][SEG], then the scores: four parts [SEG j][SEG i], then their sum in the first
-  float* B = Kt + max(DQ * SEG, 4 * SEG * SEG);        // [DQ][VT] the starting state, [SEG][VT] u
+  float* B = Kt + (CHANNEL ? SEG * SEG : max(DQ * SEG, 4 * SEG * SEG));        // [DQ][VT] the starting state, [SEG][VT] u
   float* lead = B + (DQ + SEG) * VT;      // [SEG] what is left of the starting state at each token
   float* dec = lead + SEG;                // [SEG + 1] powers or running sums of ln g
   const int seg = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT, tid = threadIdx.x;
@@ -344,11 +360,17 @@ outputs_kernel(Args p) {
       B[idx] = x;
     }
   }
+  if (CHANNEL) {                          // the scores as they are to be multiplied (always 16-byte aligned)
+    const float* a = p.scores + ((size_t)seg * p.heads + h) * SEG * SEG;
+    for (int idx = 4 * tid; idx < SEG * SEG; idx += 4 * COMPUTE) cp_async_f32x4(Kt + idx, a + idx);
+  }
   cp_async_commit();
   const size_t qk = (size_t)row0 * p.qk_stride + (h / p.share) * D;
   stage_transposed(Qt, p.q + qk, p.qk_stride, n, D, DQ, p.vec, tid);
-  stage_transposed(Kt, p.k + qk, p.qk_stride, n, D, DQ, p.vec, tid);
-  if (tid < SEG) {
+  if (!CHANNEL) stage_transposed(Kt, p.k + qk, p.qk_stride, n, D, DQ, p.vec, tid);
+  if (CHANNEL) {
+    if (tid < SEG) lead[tid] = 1.0f;
+  } else if (tid < SEG) {
     if (FIXED) {
       dec[tid] = p.powers[h * (SEG + 1) + tid];
       lead[tid] = p.powers[h * (SEG + 1) + tid + 1];
@@ -359,7 +381,7 @@ outputs_kernel(Args p) {
     }
   }
   __syncthreads();
-  {                                       // the scores, a quarter of the head's dimensions a group of 64 threads
+  if (!CHANNEL) {                         // the scores, a quarter of the head's dimensions a group of 64 threads
     const int part = tid >> 6, ti = 4 * (tid & 7), tj = 4 * ((tid >> 3) & 7);
     float s[4][4] = {};
     const int per = DQ >> 2;
@@ -377,8 +399,8 @@ outputs_kernel(Args p) {
     for (int j = 0; j < 4; ++j)
       *reinterpret_cast<float4*>(Kt + (part * SEG + tj + j) * SEG + ti) = make_float4(s[j][0], s[j][1], s[j][2], s[j][3]);
   }
-  __syncthreads();
-  {                                       // their sum, decayed and masked, in the first part's place (read by this thread alone)
+  if (!CHANNEL) __syncthreads();
+  if (!CHANNEL) {                         // their sum, decayed and masked, in the first part's place (read by this thread alone)
     const int j = tid >> 3, i0 = 4 * (tid & 7);
     float v[4] = {};
 #pragma unroll
@@ -440,28 +462,28 @@ template <typename Kern> inline int allow_smem(Kern kern, size_t bytes) {
   return bytes > 48 * 1024 ? (int)cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) : 0;
 }
 
-template <bool FIXED, bool SOLVE, int VC, int NR, int NB> int launch_carry(const Args& p, int n_entries, cudaStream_t stream) {
-  const size_t smem = carry_smem<VC, NB>(p.dim, SOLVE);
-  const int rc = allow_smem(carry_kernel<FIXED, SOLVE, VC, NR, NB>, smem);
+template <bool FIXED, bool SOLVE, bool CHANNEL, int VC, int NR, int NB> int launch_carry(const Args& p, int n_entries, cudaStream_t stream) {
+  const size_t smem = carry_smem<VC, NB>(p.dim, SOLVE, CHANNEL);
+  const int rc = allow_smem(carry_kernel<FIXED, SOLVE, CHANNEL, VC, NR, NB>, smem);
   if (rc) return rc;
-  return launch_pdl(carry_kernel<FIXED, SOLVE, VC, NR, NB>, dim3(p.heads, n_entries, (p.vdim + VC - 1) / VC), dim3(COMPUTE + HELPERS), smem, stream, p);
+  return launch_pdl(carry_kernel<FIXED, SOLVE, CHANNEL, VC, NR, NB>, dim3(p.heads, n_entries, (p.vdim + VC - 1) / VC), dim3(COMPUTE + HELPERS), smem, stream, p);
 }
-template <bool FIXED, int VT> int launch_outputs(const Args& p, int n_segments, cudaStream_t stream) {
-  const size_t smem = outputs_smem<VT>(p.dim);
-  const int rc = allow_smem(outputs_kernel<FIXED, VT>, smem);
+template <bool FIXED, bool CHANNEL, int VT> int launch_outputs(const Args& p, int n_segments, cudaStream_t stream) {
+  const size_t smem = outputs_smem<VT>(p.dim, CHANNEL);
+  const int rc = allow_smem(outputs_kernel<FIXED, CHANNEL, VT>, smem);
   if (rc) return rc;
-  return launch_pdl(outputs_kernel<FIXED, VT>, dim3(n_segments, p.heads, (p.vdim + VT - 1) / VT), dim3(COMPUTE), smem, stream, p);
+  return launch_pdl(outputs_kernel<FIXED, CHANNEL, VT>, dim3(n_segments, p.heads, (p.vdim + VT - 1) / VT), dim3(COMPUTE), smem, stream, p);
 }
 
 // Both kernels, one after the other.  Narrow column blocks where they fit the SMs at once.
-template <bool FIXED, bool SOLVE> int launch(const Args& p, int n_entries, int n_segments, cudaStream_t stream) {
+template <bool FIXED, bool SOLVE, bool CHANNEL = false> int launch(const Args& p, int n_entries, int n_segments, cudaStream_t stream) {
   const bool wide = (long long)p.heads * n_entries * ((p.vdim + 7) / 8) > 148;
   int rc;
   if (p.dim <= 128)
-    rc = wide ? launch_carry<FIXED, SOLVE, 16, 1, 4>(p, n_entries, stream) : launch_carry<FIXED, SOLVE, 8, 1, 4>(p, n_entries, stream);
+    rc = wide ? launch_carry<FIXED, SOLVE, CHANNEL, 16, 1, 4>(p, n_entries, stream) : launch_carry<FIXED, SOLVE, CHANNEL, 8, 1, 4>(p, n_entries, stream);
   else
-    rc = wide ? launch_carry<FIXED, SOLVE, 16, 2, 2>(p, n_entries, stream) : launch_carry<FIXED, SOLVE, 8, 2, 2>(p, n_entries, stream);
+    rc = wide ? launch_carry<FIXED, SOLVE, CHANNEL, 16, 2, 2>(p, n_entries, stream) : launch_carry<FIXED, SOLVE, CHANNEL, 8, 2, 2>(p, n_entries, stream);
   if (rc) return rc;
-  return p.vdim > 64 ? launch_outputs<FIXED, 128>(p, n_segments, stream) : launch_outputs<FIXED, 64>(p, n_segments, stream);
+  return p.vdim > 64 ? launch_outputs<FIXED, CHANNEL, 128>(p, n_segments, stream) : launch_outputs<FIXED, CHANNEL, 64>(p, n_segments, stream);
 }
 }  // namespace segscan

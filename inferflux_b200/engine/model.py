@@ -120,9 +120,17 @@ class Model:
             self.state_needs.append(states)
             self.runs.append(info)
 
+        self.embedding_state_needs: List[StateNeed] = list(type(self.embedding).state_needs(spec.embedding.params))
+
+    def slot_needs(self) -> List[List[StateNeed]]:
+        """What a request's state slot holds: a list per run, in schedule order, and one for the embedding."""
+        return [*self.state_needs, self.embedding_state_needs]
+
     def attach_states(self, storage) -> None:
         for info in self.runs:
             info.states = storage.of_run(info.run_index)
+        if self.embedding_state_needs:
+            self.embedding.states = storage.of_run(len(self.runs))
 
     # ---------------------------------------------------------------- weights
     def weight_specs(self) -> List[WeightSpec]:

@@ -58,7 +58,7 @@ class StepRunner:
         self.kv_storage = KVCacheStorage(needs, model.runs_per_group, self.num_pages, self.page_size,
                                          self.dtype, self.device)
         self.slots = StateSlotManager(engine_config.max_seqs)
-        self.state_storage = StateSlotStorage(engine_config.max_seqs, model.state_needs, self.device)
+        self.state_storage = StateSlotStorage(engine_config.max_seqs, model.slot_needs(), self.device)
         model.attach_states(self.state_storage)
         self.slab = MetadataSlab(1 << 16, self.device)
         self._graphs = {}

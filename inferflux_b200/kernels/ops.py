@@ -159,16 +159,16 @@ def _lib():
         lib.ifx_retention_finish.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_ll, c_int, c_int, c_int, c_float,
                                              c_void_p]
         lib.ifx_gelu_tanh.argtypes = [c_void_p, c_int, c_ll, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
-        lib.ifx_moe_route.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p]
+        lib.ifx_moe_route.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.ifx_moe_tile_rows.argtypes = [c_int]
         lib.ifx_moe_experts.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                        c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                        c_void_p]
+                                        c_int, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                                        c_void_p, c_void_p, c_void_p, c_void_p]
         lib.ifx_moe_group.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.ifx_moe_gather_rows.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
-        lib.ifx_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
-        lib.ifx_gemm_umma_grouped.argtypes = [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int,
-                                              c_void_p, c_void_p, c_void_p]
+        lib.ifx_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]
+        lib.ifx_gemm_umma_grouped.argtypes = [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_float,
+                                              c_float, c_float, c_int, c_void_p, c_void_p, c_void_p]
         lib.ifx_activation.argtypes = [c_void_p, c_ll, c_int, c_ll, c_void_p, c_int, c_ll, c_int, c_int, c_int, c_void_p]
         lib.ifx_causal_conv.argtypes = [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                         c_void_p, c_int, c_int, c_void_p, c_ll, c_int, c_int, c_void_p]
@@ -204,7 +204,7 @@ def _lib():
                                              c_void_p, c_void_p, c_ll, c_ll, c_void_p, c_int, c_ll, c_int, c_void_p, c_int,
                                              c_void_p]
         lib.ifx_attn_decode_bf16_ex.argtypes = list(lib.ifx_attn_decode_bf16.argtypes[:-1]) + [
-            c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
+            c_float, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
         lib.ifx_attn_decode_bf16_ex.restype = c_int
         lib.ifx_attn_prefill_bf16_ex2.argtypes = list(lib.ifx_attn_prefill_bf16_ex.argtypes[:-1]) + [
             c_int, c_float, c_int, c_void_p, c_void_p, c_void_p]
@@ -216,10 +216,18 @@ def _lib():
                                                  c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p]
         lib.ifx_causal_conv_heads.argtypes = list(lib.ifx_causal_conv.argtypes[:-1]) + [c_int, c_int, c_int, c_float, c_float, c_void_p]
         lib.ifx_gated_delta_segment.argtypes = []
-        lib.ifx_gated_delta_scan.argtypes = [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p,
+        lib.ifx_gated_delta_scan.argtypes = [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p,
                                              c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+                                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                             c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.ifx_softcap.argtypes = [c_void_p, c_ll, c_float, c_void_p]
+        lib.ifx_max_streams.argtypes = []
+        lib.ifx_stream_mix_norm.argtypes = [c_void_p, c_void_p, c_int, c_int, c_ll, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
+                                            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+        lib.ifx_embed_bigram.argtypes = [c_void_p, c_void_p, c_int, c_ll, c_ll, c_ll, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+        for name in ("ifx_max_streams", "ifx_stream_mix_norm", "ifx_embed_bigram"):
+            getattr(lib, name).restype = c_int
         for name in ("ifx_head_norm_rope_write", "ifx_causal_conv_heads", "ifx_gated_delta_segment", "ifx_gated_delta_scan",
                      "ifx_softcap"):
             getattr(lib, name).restype = c_int
@@ -699,11 +707,11 @@ def attn_decode_bf16(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_layer:
                      entry_q_len: torch.Tensor, entry_ctx_start: torch.Tensor, part_o: Optional[torch.Tensor],
                      part_ml: Optional[torch.Tensor], n_heads: int, n_kv: int, head_dim: int, scale: float,
                      window: int, n_splits: int, q_temp=None, distance_toll=None, gate: Optional[torch.Tensor] = None,
-                     gate_per_head: bool = False) -> torch.Tensor:
+                     gate_per_head: bool = False, softcap: float = 0.0) -> torch.Tensor:
     """Tensor-core attention of single decoded tokens (entries listed in
     dec_entries), the keys split ``n_splits`` ways and merged.  Scratch:
     part_o float32 [n_dec * n_heads * n_splits * head_dim], part_ml float32
-    [n_dec * n_heads * n_splits * 2].  ``window``, ``q_temp``, ``distance_toll``,
+    [n_dec * n_heads * n_splits * 2].  ``window``, ``softcap``, ``q_temp``, ``distance_toll``,
     ``gate`` and ``gate_per_head`` as in :func:`attn_paged_options`."""
     gp, g_parts, g_pstride, g_stride = _gate_slices(gate, n_heads if gate_per_head else n_heads * head_dim, "attn_decode_bf16")
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
@@ -726,7 +734,7 @@ def attn_decode_bf16(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_layer:
                                           page_stride, page_size, _ptr(block_tables), block_tables.stride(0),
                                           _ptr(dec_entries), n_dec, _ptr(entry_q_start), _ptr(entry_q_len),
                                           _ptr(entry_ctx_start), _ptr(part_o), _ptr(part_ml), n_heads, n_kv, head_dim,
-                                          float(scale), int(window), int(n_splits), coef, every, _ptr(r1), _ptr(r2),
+                                          float(scale), int(window), int(n_splits), float(softcap), coef, every, _ptr(r1), _ptr(r2),
                                           gp, g_parts, g_pstride, g_stride, int(bool(gate_per_head)), _stream()),
            "attn_decode_bf16")
     return out
@@ -1470,17 +1478,21 @@ def gelu_tanh(z: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def moe_route(logits: torch.Tensor, top: int, over_all: bool = False, scale: float = 1.0):
+def moe_route(logits: torch.Tensor, top: int, over_all: bool = False, scale: float = 1.0,
+              correction: Optional[torch.Tensor] = None):
     """The ``top`` largest of every row of float32 ``logits [N, E]`` (lowest index first among equals) and their
     weights: the softmax over the chosen logits alone, or, with ``over_all``, the softmax over every expert's
-    logit with the chosen scores divided by their sum (+ 1e-20); either times ``scale``.  Returns (int32
+    logit with the chosen scores divided by their sum (+ 1e-20); either times ``scale``.  ``correction`` (float32 ``[E]``,
+    with ``over_all``): the choice goes by the score plus the correction, the weights by the score alone.  Returns (int32
     ``[N, top]``, float32 ``[N, top]``)."""
     n, experts = logits.shape
     _need(logits.dtype == torch.float32 and logits.is_contiguous(), "moe_route: float32 logits")
     _need(1 <= top <= min(64, experts), f"moe_route: top {top} must be within 1..min(64, experts)")
+    _need(correction is None or (over_all and correction.dtype == torch.float32 and correction.is_contiguous()
+                                 and correction.numel() == experts), "moe_route: correction float32 [E], with over_all")
     chosen = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
-    _check(_lib().ifx_moe_route(_ptr(logits), n, experts, top, int(bool(over_all)), float(scale), _ptr(chosen),
+    _check(_lib().ifx_moe_route(_ptr(logits), n, experts, top, int(bool(over_all)), float(scale), _ptr(correction), _ptr(chosen),
                                 _ptr(weights), _stream()), "moe_route")
     return chosen, weights
 
@@ -1492,7 +1504,7 @@ MOE_TENSOR_CORE_PAIRS = 512
 MOE_UMMA_TILE = 256
 
 
-def _moe_experts_umma(x, w_gate_up, w_down, chosen, weights, n, hidden, ff, experts, top, activation) -> torch.Tensor:
+def _moe_experts_umma(x, w_gate_up, w_down, chosen, weights, n, hidden, ff, experts, top, activation, shape) -> torch.Tensor:
     lib, dev, tile = _lib(), x.device, MOE_UMMA_TILE
     pairs = n * top
     max_tiles = pairs // tile + experts
@@ -1506,35 +1518,39 @@ def _moe_experts_umma(x, w_gate_up, w_down, chosen, weights, n, hidden, ff, expe
     _check(lib.ifx_moe_gather_rows(_ptr(x), _code(x), _ptr(sorted_pair), _ptr(xs), rows, hidden, top, _stream()), "moe_gather_rows")
     act = torch.empty((rows, ff), dtype=x.dtype, device=dev)
     flag = error_flag(dev)
-    _check(lib.ifx_gemm_umma_grouped(_ptr(xs), hidden, _ptr(w_gate_up), _ptr(act), ff, BF16, rows, ff, hidden, activation, experts,
-                                     _ptr(tile_expert), _ptr(flag), _stream()), "gemm_umma_grouped (gate, up)")
+    _check(lib.ifx_gemm_umma_grouped(_ptr(xs), hidden, _ptr(w_gate_up), _ptr(act), ff, BF16, rows, ff, hidden, activation, *shape,
+                                     experts, _ptr(tile_expert), _ptr(flag), _stream()), "gemm_umma_grouped (gate, up)")
     y = torch.empty((rows, hidden), dtype=torch.float32, device=dev)
-    _check(lib.ifx_gemm_umma_grouped(_ptr(act), ff, _ptr(w_down), _ptr(y), hidden, F32, rows, hidden, ff, 0, experts,
-                                     _ptr(tile_expert), _ptr(flag), _stream()), "gemm_umma_grouped (down)")
+    _check(lib.ifx_gemm_umma_grouped(_ptr(act), ff, _ptr(w_down), _ptr(y), hidden, F32, rows, hidden, ff, 0, *shape,
+                                     experts, _ptr(tile_expert), _ptr(flag), _stream()), "gemm_umma_grouped (down)")
     out = torch.empty((n, hidden), dtype=torch.float32, device=dev)
-    _check(lib.ifx_moe_combine(_ptr(y), _ptr(pair_row), _ptr(weights), _ptr(out), n, hidden, top, _stream()), "moe_combine")
+    _check(lib.ifx_moe_combine(_ptr(y), _ptr(pair_row), _ptr(weights), _ptr(x), _code(x), _ptr(out), n, hidden, top, _stream()), "moe_combine")
     return out
 
 
-MOE_SWIGLU, MOE_RELU2 = 1, 2
+MOE_SWIGLU, MOE_RELU2, MOE_CLAMPED_GLU = 1, 2, 3
 
 
 def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor,
-                weights: torch.Tensor, activation: int = MOE_SWIGLU) -> torch.Tensor:
+                weights: torch.Tensor, activation: int = MOE_SWIGLU, limit: float = 0.0, alpha: float = 0.0,
+                shift: float = 0.0) -> torch.Tensor:
     """``out[t] = sum_k weights[t, k] * W_down[e] act_e(x_t)``, ``e = chosen[t, k]``.  ``MOE_SWIGLU``: ``w_gate_up
     [E, 2F, H]`` (gate rows, then up rows) and ``act = silu(W_gate x) * (W_up x)``; ``MOE_RELU2``: ``w_gate_up [E, F, H]``
-    (up rows alone) and ``act = relu(W_up x)^2``.  ``x [N, H]``, ``w_down [E, H, F]`` of one type; float32 ``[N, H]``
+    (up rows alone) and ``act = relu(W_up x)^2``; ``MOE_CLAMPED_GLU``: ``w_gate_up`` as for the first and ``g * sigmoid(alpha g)
+    * (u + shift)`` with ``g = min(W_gate x, limit)``, ``u = clamp(W_up x, -limit, limit)``.  A choice of E or more is one of
+    the identity: it gives ``x_t`` itself.  ``x [N, H]``, ``w_down [E, H, F]`` of one type; float32 ``[N, H]``
     out.  The pairs are sorted by expert on the device and run as tiles of one expert each."""
     n, hidden = x.shape
     experts, up_rows, _ = w_gate_up.shape
-    ff, top = (up_rows // 2 if activation == MOE_SWIGLU else up_rows), chosen.shape[1]
-    _need(activation in (MOE_SWIGLU, MOE_RELU2), "moe_experts: activation")
+    ff, top = (up_rows if activation == MOE_RELU2 else up_rows // 2), chosen.shape[1]
+    shape = (float(limit), float(alpha), float(shift))
+    _need(activation in (MOE_SWIGLU, MOE_RELU2) or (activation == MOE_CLAMPED_GLU and limit > 0), "moe_experts: activation")
     _need(x.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and x.dtype == w_gate_up.dtype == w_down.dtype,
           "moe_experts: contiguous operands of one type")
     _need(tuple(w_down.shape) == (experts, hidden, ff) and w_gate_up.shape[2] == hidden, "moe_experts: weight shapes")
     pairs = n * top
     if (MOE_TENSOR_CORES and x.dtype == torch.bfloat16 and pairs >= MOE_TENSOR_CORE_PAIRS and hidden % 8 == 0 and ff % 8 == 0):
-        return _moe_experts_umma(x, w_gate_up, w_down, chosen, weights, n, hidden, ff, experts, top, activation)
+        return _moe_experts_umma(x, w_gate_up, w_down, chosen, weights, n, hidden, ff, experts, top, activation, shape)
     tile = int(_lib().ifx_moe_tile_rows(pairs))
     max_tiles = pairs // tile + experts
     dev = x.device
@@ -1545,7 +1561,7 @@ def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     y = torch.empty((max_tiles * tile, hidden), dtype=torch.float32, device=dev)
     out = torch.empty((n, hidden), dtype=torch.float32, device=dev)
     _check(_lib().ifx_moe_experts(_ptr(x), _code(x), _ptr(w_gate_up), _ptr(w_down), _ptr(chosen), _ptr(weights), n, hidden, ff,
-                                  experts, top, activation, tile, max_tiles, _ptr(tile_expert), _ptr(sorted_pair), _ptr(pair_row),
+                                  experts, top, activation, *shape, tile, max_tiles, _ptr(tile_expert), _ptr(sorted_pair), _ptr(pair_row),
                                   _ptr(act), _ptr(y), _ptr(out), _stream()), "moe_experts")
     global launch_count
     launch_count += 3
@@ -1553,7 +1569,7 @@ def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
 
 
 # ------------------------------------------------- activations, state-space scan, delta rule, normed q/k/v
-ACT_GELU, ACT_TANH, ACT_RELU2, ACT_SILU, ACT_SIGMOID = 0, 1, 2, 3, 4
+ACT_GELU, ACT_TANH, ACT_RELU2, ACT_SILU, ACT_SIGMOID, ACT_NONE = 0, 1, 2, 3, 4, 5
 
 
 def activation(z: torch.Tensor, out: torch.Tensor, act: int) -> torch.Tensor:
@@ -1871,31 +1887,42 @@ def gated_delta_scan(qkv: torch.Tensor, q_col: int, k_col: int, v_col: int, raw:
                      a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, entry_q_start: torch.Tensor,
                      entry_q_len: torch.Tensor, entry_slot: torch.Tensor, n_entries: int, out: torch.Tensor, heads: int,
                      kv_heads: int, dim: int, vdim: int, seg_entry: torch.Tensor, seg_t0: torch.Tensor,
-                     entry_first_seg: torch.Tensor, n_segments: int) -> torch.Tensor:
+                     entry_first_seg: torch.Tensor, n_segments: int,
+                     decay: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The gated delta rule, float32.  Per head (query and key of head ``h // (heads / kv_heads)``): ``g = exp(-exp(a_log)
     softplus(a + dt_bias))``, ``beta = sigmoid(b)``, ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
     ``o = S^T q``.  ``qkv`` float32 rows hold the prepared q and k (``kv_heads * dim``) and v (``heads * vdim``) from the
     given columns; ``raw`` float32 rows hold a and b (``heads`` each); ``state [slots, heads, dim, vdim]``; ``out``
     float32 ``[N, heads * vdim]``.  The step's entries are cut into segments of :func:`gated_delta_segment` tokens
-    (``n_segments`` 0: every entry brings one token)."""
+    (``n_segments`` 0: every entry brings one token).  With ``decay`` (float32 rows ``[N, heads * dim]``) there is one g per
+    head and key channel, from ``decay`` in a's place and ``dt_bias [heads * dim]``; ``S <- diag(g) S``."""
     n, dev = qkv.shape[0], qkv.device
+    _need(decay is None or (decay.dtype == torch.float32 and decay.stride(1) == 1 and tuple(decay.shape) == (n, heads * dim)),
+          "gated_delta_scan: decay float32 [N, heads * dim]")
     _need(qkv.dtype == torch.float32 and qkv.stride(1) == 1 and raw.dtype == torch.float32 and raw.stride(1) == 1
           and raw.shape[0] == n, "gated_delta_scan: float32 rows")
-    _need(all(v.dtype == torch.float32 and v.numel() == heads and v.is_contiguous() for v in (a_log, dt_bias)),
-          "gated_delta_scan: a_log, dt_bias float32 [heads]")
+    _need(all(v.dtype == torch.float32 and v.numel() == k and v.is_contiguous()
+              for v, k in ((a_log, heads), (dt_bias, heads if decay is None else heads * dim))),
+          "gated_delta_scan: a_log, dt_bias float32 [heads] (dt_bias [heads * dim] with a decay per channel)")
     _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim),
           "gated_delta_scan: state float32 [slots, heads, dim, vdim]")
     _need(out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, heads * vdim), "gated_delta_scan: out")
     _need(n_segments > 0 or n == n_entries, "gated_delta_scan: a step with portions lists its segments")
-    w_rows = u_rows = cum = seg_start = None
+    w_rows = u_rows = cum = seg_start = k_rows = q_rows = seg_decay = scores = None
     if n_segments:
         f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
-        w_rows, u_rows, cum = f32(n, heads * dim), f32(n, heads * vdim), f32(n, heads)
+        w_rows, u_rows = f32(n, heads * dim), f32(n, heads * vdim)
+        if decay is None:
+            cum = f32(n, heads)
+        else:
+            k_rows, q_rows = f32(n, heads * dim), f32(n, heads * dim)
+            seg_decay, scores = f32(n_segments, heads, dim), f32(n_segments, heads, gated_delta_segment(), gated_delta_segment())
         seg_start = f32(n_segments, heads, dim, vdim)
     _check(_lib().ifx_gated_delta_scan(_ptr(qkv), qkv.stride(0), q_col, k_col, v_col, _ptr(raw), raw.stride(0), a_col, b_col,
-                                       _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(entry_q_start), _ptr(entry_q_len),
+                                       _ptr(decay), decay.stride(0) if decay is not None else 0, _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(entry_q_start), _ptr(entry_q_len),
                                        _ptr(entry_slot), n_entries, _ptr(seg_entry), _ptr(seg_t0), _ptr(entry_first_seg),
-                                       n_segments, _ptr(w_rows), _ptr(u_rows), _ptr(cum), _ptr(seg_start), _ptr(out), heads,
+                                       n_segments, _ptr(w_rows), _ptr(u_rows), _ptr(cum), _ptr(k_rows), _ptr(q_rows),
+                                       _ptr(seg_decay), _ptr(scores), _ptr(seg_start), _ptr(out), heads,
                                        kv_heads, dim, vdim, _stream()), "gated_delta_scan")
     if n_segments:
         global launch_count
@@ -1908,3 +1935,53 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
     _need(x.dtype == torch.float32 and x.is_contiguous() and cap > 0, "softcap: float32, a positive cap")
     _check(_lib().ifx_softcap(_ptr(x), x.numel(), float(cap), _stream()), "softcap")
     return x
+
+
+# ------------------------------------------------- a stream of several copies, hashed token pairs
+MAX_STREAMS = 16        # copies that stream_mix_norm takes
+
+
+def stream_mix_norm(x: torch.Tensor, y: Optional[torch.Tensor], mix: Optional[torch.Tensor], w_out: Optional[torch.Tensor],
+                    reads: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                    rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x`` float32 ``[N, S, H]``: with ``y`` (``[N, H]`` or slices ``[P, N, H]``, float32 or bfloat16) pending, ``X_t <- sum_s
+    mix[s, t] X_s + w_out[t] * y``; then ``u = sum_s reads[s] X_s`` and ``out = u / sqrt(mean(u^2) + eps) * weight``.  ``mix``
+    ``[S, S]``, ``w_out``, ``reads`` ``[S]``, ``weight`` ``[H]``: float32.  With ``rows`` (int32) only those rows are worked
+    on, into ``out [R, H]``, and ``x`` is left as it is."""
+    n, s, hidden = x.shape
+    f32 = lambda t, k: t.dtype == torch.float32 and t.is_contiguous() and t.numel() == k
+    _need(x.dtype == torch.float32 and x.is_contiguous() and 1 <= s <= MAX_STREAMS, "stream_mix_norm: x float32 [N, S, H]")
+    _need(f32(reads, s) and f32(weight, hidden), "stream_mix_norm: reads [S], weight [H] float32")
+    n_rows = rows.numel() if rows is not None else n
+    _need(rows is None or rows.dtype == torch.int32, "stream_mix_norm: rows int32")
+    _need(out.is_contiguous() and tuple(out.shape) == (n_rows, hidden), "stream_mix_norm: out [rows, H]")
+    parts = 1
+    if y is not None:
+        _need(y.is_contiguous() and y.dim() in (2, 3) and tuple(y.shape[-2:]) == (n, hidden), "stream_mix_norm: y [N, H] or [P, N, H]")
+        _need(mix is not None and w_out is not None and f32(mix, s * s) and f32(w_out, s), "stream_mix_norm: mix [S, S], w_out [S] float32")
+        parts = y.shape[0] if y.dim() == 3 else 1
+    _check(_lib().ifx_stream_mix_norm(_ptr(x), _ptr(y), _code(y) if y is not None else F32, parts, n * hidden, _ptr(mix),
+                                      _ptr(w_out), _ptr(reads), _ptr(weight), float(eps), _ptr(out), _code(out), _ptr(rows), n_rows,
+                                      hidden, s, 0 if rows is not None else 1, _stream()), "stream_mix_norm")
+    return out
+
+
+def embed_bigram(table: torch.Tensor, pairs: Optional[torch.Tensor], hash_, ids: torch.Tensor, last: Optional[torch.Tensor],
+                 row_entry: torch.Tensor, entry_q_start: torch.Tensor, entry_q_len: torch.Tensor, entry_slot: torch.Tensor,
+                 out: torch.Tensor) -> torch.Tensor:
+    """``out[t, s] = float32(table[ids[t]])`` for every copy s of ``out`` float32 ``[N, S, H]``, plus, with ``hash_`` =
+    ``(buckets, mul_prev, mul_cur)``, ``pairs[(previous * mul_prev + id * mul_cur) mod buckets]`` (``pairs[buckets]`` where a
+    sequence begins).  ``last`` int32 ``[slots, 1]`` holds each request's last token plus one (0: none yet) and is moved on."""
+    n, s, hidden = out.shape
+    vocab = table.shape[0]
+    _need(ids.dtype == torch.int32 and ids.numel() == n and out.dtype == torch.float32 and out.is_contiguous(), "embed_bigram: ids int32, out float32")
+    _need(table.is_contiguous() and table.shape[1] == hidden, "embed_bigram: table [V, H]")
+    buckets, mul_prev, mul_cur = hash_ if hash_ else (0, 0, 0)
+    if hash_:
+        _need(pairs is not None and pairs.is_contiguous() and pairs.dtype == table.dtype and tuple(pairs.shape) == (buckets + 1, hidden),
+              "embed_bigram: pairs [buckets + 1, H] of the table's type")
+        _need(last is not None and last.dtype == torch.int32 and last.is_contiguous(), "embed_bigram: last int32 [slots, 1]")
+    _check(_lib().ifx_embed_bigram(_ptr(table), _ptr(pairs) if hash_ else None, _code(table), buckets, mul_prev, mul_cur, _ptr(ids),
+                                   _ptr(last), _ptr(row_entry), _ptr(entry_q_start), _ptr(entry_q_len), _ptr(entry_slot), _ptr(out),
+                                   n, hidden, vocab, s, _stream()), "embed_bigram")
+    return out

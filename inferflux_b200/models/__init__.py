@@ -5,3 +5,4 @@ from . import pemorax  # noqa: F401
 from . import tekosun  # noqa: F401
 from . import malazen  # noqa: F401
 from . import zetivik  # noqa: F401
+from . import kibilix  # noqa: F401

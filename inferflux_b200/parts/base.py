@@ -99,6 +99,15 @@ class JoinedSum:
         self.value, self.rows, self.vector = value, rows, vector
 
 
+class StreamMix:
+    """A sublayer's result on its way into a stream of several copies: ``X_t <- sum_s mix[s, t] X_s + out[t] * value``,
+    all copies at once from the old ones; ``value`` a tensor or :class:`PartialSums`, ``mix`` float32 ``[S, S]`` (from, to),
+    ``out`` float32 ``[S]``.  The norm that comes next mixes the copies while it reads them."""
+
+    def __init__(self, value, mix: torch.Tensor, out: torch.Tensor):
+        self.value, self.mix, self.out = value, mix, out
+
+
 class NormedDelta:
     """A sublayer's result that is to be normed before it joins the stream: ``N(value) * weight`` with ``value``
     a tensor, :class:`PartialSums` or :class:`BranchMean`.  Blocks with a norm behind every sublayer hand this
@@ -134,7 +143,8 @@ class Part:
       object and says so in its docstring.
     * ``embedding``: ``forward_step(ctx) -> float32 [N, hidden]`` (the default
       calls ``forward(token_ids)``; one that adds positions reads them from
-      ``ctx``); ``lm_head``: ``forward(x) -> float32 [rows, vocab]``.
+      ``ctx``; one for a stream of several copies gives ``[N, copies, hidden]``,
+      and its :meth:`state_needs` are tensors it finds in ``self.states``); ``lm_head``: ``forward(x) -> float32 [rows, vocab]``.
     * ``shift``: ``forward(h32, ctx, run) -> Tensor``: mixes every row of the
       float32 normed rows with the row before it (the request's state slot
       holds the last row of the step before).

@@ -254,6 +254,39 @@ class PostNormBlock:
         return NormedDelta(self.ff.forward(x2, ctx), self.ff_post.weight, self.ff_post.eps)
 
 
+class StreamsBlock:
+    """Pre-norm over a stream of several copies ``X_1 .. X_S`` (``residual`` is float32 ``[N, S, hidden]``): each sublayer
+    has a norm that reads a weighted sum of the copies and a join that mixes them anew while its result comes in,
+
+        y = mixer(norm_1(sum_s in_1[s] X_s));   X_t <- sum_s mix_1[s, t] X_s + out_1[t] * y
+        then the same with the feed-forward                          (a layer may have no feed-forward)
+
+    Nothing is mixed here: a sublayer's result goes on as a :class:`~inferflux_b200.parts.base.StreamMix`, and the next
+    norm mixes the copies, sums what it reads and norms it in one kernel."""
+
+    family = "arrangement"
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "mixer_join": "junction",
+             "feed_forward_norm": "norm", "feed_forward": "feed_forward", "feed_forward_join": "junction"}
+    optional_roles = frozenset({"feed_forward_norm", "feed_forward", "feed_forward_join"})
+
+    def __init__(self, parts: Dict[str, object], position_name: Optional[str]):
+        self.mixer_norm, self.mixer, self.mixer_join = parts["mixer_norm"], parts["mixer"], parts["mixer_join"]
+        self.ff_norm, self.ff, self.ff_join = (parts.get(r) for r in ("feed_forward_norm", "feed_forward", "feed_forward_join"))
+        if (self.ff is None) != (self.ff_norm is None) or (self.ff is None) != (self.ff_join is None):
+            raise ValueError("a streams block has a feed-forward with its norm and its join or none of the three")
+        self.position_name = position_name
+
+    def forward(self, residual: torch.Tensor, delta, ctx, run: RunInfo):
+        x = self.mixer_norm.forward(residual, delta)
+        position = ctx.position_tables.get(self.position_name) if self.position_name else None
+        a = self.mixer_join.pending(self.mixer.forward(x, ctx, run, position), ctx, run)
+        if self.ff is None:
+            return a
+        x2 = self.ff_norm.forward(residual, a)
+        return self.ff_join.pending(self.ff.forward(x2, ctx), ctx, run)
+
+
+register_part("arrangement", "streams", StreamsBlock)
 register_part("arrangement", "pre_post_norm", PrePostNormBlock)
 register_part("arrangement", "post_norm", PostNormBlock)
 register_part("arrangement", "parallel", ParallelBlock)

@@ -24,7 +24,12 @@ state lives in the request's state slot.
     o_t = S^T q_t
 
 every head's o is divided by its root mean square, multiplied by a weight ``vdim`` long that the heads share and by
-silu(W_g h), and projected.  All input projections are one stacked product whose sums stay float32, and so does
+silu(W_g h) (or sigmoid of it), and projected.  With ``decay`` ``channel`` there is one decay per head and key channel,
+
+    g_t = exp(-exp(A_log) softplus(W_a2 W_a1 h_t + dt_bias))         heads x dim;   S <- diag(g_t) S
+
+(A_log one a head).  The decays and, with ``two_step``, the gate (W_g2 W_g1 h) are projected in two steps: the two inner
+products are rows of the stacked one, and both outer products are one product over the inner rows side by side.  All input projections are one stacked product whose sums stay float32, and so does
 everything up to the output projection's input.  The state and the last ``taps - 1`` inputs of the convolutions live in
 the request's state slot, so a prompt may be cut anywhere; a portion is cut into segments whose part that does not
 depend on the state is worked out side by side.
@@ -140,9 +145,10 @@ class GatedDeltaStep:
 
 class GatedDelta(Part):
     """params: ``hidden``, ``heads``, ``kv_heads`` (default ``heads``), ``dim``, ``vdim``, ``conv`` (taps), ``eps`` (of the
-    per-head norm), ``q_scale`` (default ``dim^-1/2``), ``key_eps`` (default 1e-6), ``name`` (tensors
+    per-head norm), ``q_scale`` (default ``dim^-1/2``), ``key_eps`` (default 1e-6), ``decay`` (``head`` or ``channel``, the
+    latter projected in two steps), ``gate`` (``silu`` or ``sigmoid``), ``two_step`` (the gate's projection), ``name`` (tensors
     ``<prefix>.<name>.{q,k,v,a,b,g,o,A_log,dt_bias,norm}`` and ``.{q,k,v}.conv`` ``[channels, taps]``; ``b`` is the rate's
-    projection).  State: ``gated_delta`` float32 ``[heads, dim, vdim]``, ``gated_delta_tail`` float32 ``[taps - 1,
+    projection; a projection in two steps is ``{a1,a2}`` or ``{g1,g2}``, its inner size the stored tensors' own).  State: ``gated_delta`` float32 ``[heads, dim, vdim]``, ``gated_delta_tail`` float32 ``[taps - 1,
     channels of q, k and v]``."""
 
     family = "mixer"
@@ -162,8 +168,14 @@ class GatedDelta(Part):
             raise ValueError("gated_delta: dim must be within 1..256")
         if not 1 <= self.taps <= 16:
             raise ValueError("gated_delta: conv must be within 1..16 taps")
+        self.by_channel = {"head": False, "channel": True}.get(p.get("decay", "head"))
+        self.gate = {"silu": ops.GATE_SILU, "sigmoid": ops.GATE_SIGMOID}.get(p.get("gate", "silu"))
+        if self.by_channel is None or self.gate is None:
+            raise ValueError("gated_delta: decay is 'head' or 'channel', gate is 'silu' or 'sigmoid'")
+        self.two_step = bool(p.get("two_step"))
         self.channels = self._channels(p)
-        self.stacked: Linear = None         # [q; k; v; g; a; b]
+        self.stacked: Linear = None         # [q; k; v; the one-step ones of g and a; the inner ones of a and g; b]
+        self.outer: Linear = None           # the outer steps of a and g over the inner rows
         self.o: Linear = None
 
     @classmethod
@@ -179,9 +191,19 @@ class GatedDelta(Part):
         rows = {"q": nk * d, "k": nk * d, "v": nh * vd}
         return ([WeightSpec(n(x), (r, h), MATRIX) for x, r in rows.items()]
                 + [WeightSpec(n(f"{x}.conv"), (r, taps), VECTOR, std=0.5) for x, r in rows.items()]
-                + [WeightSpec(n("g"), (nh * vd, h), MATRIX), WeightSpec(n("a"), (nh, h), MATRIX), WeightSpec(n("b"), (nh, h), MATRIX),
-                   WeightSpec(n("A_log"), (nh,), VECTOR, std=0.5), WeightSpec(n("dt_bias"), (nh,), VECTOR, std=0.5),
+                + cls._projection(params, n, "g", params.get("two_step"), nh * vd, h)
+                + cls._projection(params, n, "a", params.get("decay") == "channel", nh * d if params.get("decay") == "channel" else nh, h)
+                + [WeightSpec(n("b"), (nh, h), MATRIX), WeightSpec(n("A_log"), (nh,), VECTOR, std=0.5),
+                   WeightSpec(n("dt_bias"), (nh * d if params.get("decay") == "channel" else nh,), VECTOR, std=0.5),
                    WeightSpec(n("norm"), (vd,), VECTOR, init="one_plus_normal"), WeightSpec(n("o"), (h, nh * vd), MATRIX)])
+
+    @staticmethod
+    def _projection(params, n, leaf: str, two_step: bool, rows: int, hidden: int) -> List[WeightSpec]:
+        if not two_step:
+            return [WeightSpec(n(leaf), (rows, hidden), MATRIX)]
+        rank = int(params.get("rank") or 128)              # of random weights; stored ones have their own
+        return [WeightSpec(n(leaf + "1"), (-1, hidden), MATRIX, free_size=rank),
+                WeightSpec(n(leaf + "2"), (rows, -1), MATRIX, std=rank ** -0.5, free_size=rank)]
 
     @classmethod
     def state_needs(cls, params: Dict[str, Any]) -> List[StateNeed]:
@@ -193,11 +215,36 @@ class GatedDelta(Part):
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         n = lambda leaf: self.full_name(self.prefix, self.params, leaf)
         f32 = lambda leaf: tensors.pop(n(leaf)).to(torch.float32).contiguous()
-        mats = [tensors.pop(n(x)) for x in ("q", "k", "v", "g", "a", "b")]
-        if len({m.dtype for m in mats}) > 1:
-            mats = [m.float() for m in mats]
-        self.stacked = Linear(torch.cat(mats, dim=0))
-        del mats
+        mats = {x: tensors.pop(n(x)) for x in (["q", "k", "v"] + ([] if self.two_step else ["g"]) + ([] if self.by_channel else ["a"]))}
+        outer = []                                         # (second step, its inner size), the decays' first
+        for leaf, on in (("a", self.by_channel), ("g", self.two_step)):
+            if on:
+                mats[leaf + "1"], second = tensors.pop(n(leaf + "1")), tensors.pop(n(leaf + "2"))
+                if second.shape[1] != mats[leaf + "1"].shape[0]:
+                    raise ValueError(f"{n(leaf + '2')} takes {second.shape[1]} inputs but {n(leaf + '1')} gives {mats[leaf + '1'].shape[0]}")
+                outer.append(second)
+        mats["b"] = tensors.pop(n("b"))
+        if len({m.dtype for m in (*mats.values(), *outer)}) > 1:
+            mats, outer = {k: m.float() for k, m in mats.items()}, [m.float() for m in outer]
+        self.inner_cols = -(-sum(m.shape[1] for m in outer) // 8) * 8          # rows of zeros fill the inner ones up to eights
+        if outer:
+            like = mats["b"]
+            fill = like.new_zeros((self.inner_cols - sum(m.shape[1] for m in outer), self.hidden))
+            b = mats.pop("b")
+            mats.update(fill=fill, b=b)
+            joint, row, col = like.new_zeros((sum(m.shape[0] for m in outer), self.inner_cols)), 0, 0
+            for m in outer:
+                joint[row:row + m.shape[0], col:col + m.shape[1]] = m
+                row, col = row + m.shape[0], col + m.shape[1]
+            self.outer = Linear(joint)
+        self.at, row = {}, 0                               # where each block of the stacked product begins
+        for k, m in mats.items():
+            self.at[k], row = row, row + m.shape[0]
+        self.at["inner"] = self.at.get("a1", self.at.get("g1", 0))
+        if outer and row % 4:                              # rows of float32 sums that start on 16-byte boundaries
+            mats["end"] = mats["b"].new_zeros((4 - row % 4, self.hidden))
+        self.stacked = Linear(torch.cat(list(mats.values()), dim=0))
+        del mats, outer
         self.conv_w = torch.cat([f32(f"{x}.conv") for x in ("q", "k", "v")]).contiguous()
         self.a_log, self.dt_bias = f32("A_log"), f32("dt_bias")
         self.norm_w = f32("norm").repeat(self.heads).contiguous()
@@ -225,19 +272,26 @@ class GatedDelta(Part):
         n, dev = x.shape[0], x.device
         kd, hv, c = self.kv_heads * self.dim, self.heads * self.vdim, self.channels
         step: GatedDeltaStep = ctx.extras[self.describe_key]
-        proj = self.stacked.forward(x, out_dtype=torch.float32)               # [q | k | v | g | a | b]
+        proj = self.stacked.forward(x, out_dtype=torch.float32)
+        outer = None                                       # [decays | gate] of what is projected in two steps
+        if self.outer is not None:
+            rows = torch.empty((n, self.inner_cols), dtype=x.dtype, device=dev)
+            ops.activation(proj[:, self.at["inner"]:self.at["inner"] + self.inner_cols], rows, ops.ACT_NONE)
+            outer = self.outer.forward(rows, out_dtype=torch.float32)
+        decay = outer[:, :self.heads * self.dim] if self.by_channel else None
+        gate = outer[:, outer.shape[1] - hv:] if self.two_step else proj[:, self.at["g"]:self.at["g"] + hv]
         qkv = torch.empty((n, c), dtype=torch.float32, device=dev)
         ops.causal_conv_heads(proj, 0, c, self.conv_w, None, run.states["gated_delta_tail"] if self.taps > 1 else None,
                               step.row_entry, ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, qkv,
                               2 * self.kv_heads, self.dim, self.kv_heads, self.q_scale, self.key_eps)
         o = torch.empty((n, hv), dtype=torch.float32, device=dev)
-        ops.gated_delta_scan(qkv, 0, kd, 2 * kd, proj, c + hv, c + hv + self.heads, self.a_log, self.dt_bias,
+        ops.gated_delta_scan(qkv, 0, kd, 2 * kd, proj, self.at.get("a", 0), self.at["b"], self.a_log, self.dt_bias,
                              run.states["gated_delta"], ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, ctx.n_entries, o,
                              self.heads, self.kv_heads, self.dim, self.vdim, step.seg_entry, step.seg_t0, step.entry_first_seg,
-                             step.n_segments)
+                             step.n_segments, decay)
         if out is None:
             out = torch.empty((n, hv), dtype=x.dtype, device=dev)
-        return ops.head_norm_gate(o, proj[:, c:c + hv], self.norm_w, out, self.heads, self.vdim, self.eps, ops.GATE_SILU)
+        return ops.head_norm_gate(o, gate, self.norm_w, out, self.heads, self.vdim, self.eps, self.gate)
 
     def forward(self, x: torch.Tensor, ctx, run: RunInfo, position):
         return self.o.forward(self.inner(x, ctx, run), allow_partials=True, f32_sums=True, out_dtype=torch.float32)

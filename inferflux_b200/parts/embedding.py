@@ -17,8 +17,9 @@ import torch
 from ..config.registry import register_part
 from ..kernels import ops
 from ..weights.loader import IGNORED, MATRIX, VECTOR, WeightSpec
-from .base import Part
+from .base import Part, StateNeed
 from .linear import Linear
+from .state_space import describe_row_entries
 
 
 class TokenEmbedding(Part):
@@ -87,6 +88,54 @@ class SinusoidNormEmbedding(Part):
         return ops.embed_sinusoid_layernorm(self.table, ctx.token_ids, ctx.positions, self.weight, self.eps, self.base, out)
 
 
+class BigramEmbedding(Part):
+    """Token embedding plus, with ``bigram``, a hashed embedding of the token pair, for a stream of several copies:
+
+        x = E[id] + B[(previous * mul_prev + id * mul_cur) mod buckets]      B[buckets] for a sequence's first token
+
+    written to every copy of the stream.  Ids and the hash are 64-bit integers, the sum float32.  The last token of a
+    portion waits in the request's state slot (stored one up, so that a zeroed slot says that there is none yet).
+    params: ``vocab``, ``hidden``, ``table`` and ``pairs`` (the full names of the two tensors), ``bigram`` (None, or
+    {buckets, mul_prev, mul_cur}), ``streams`` (default 1).  State: ``last_token`` int32 ``[1]``."""
+
+    family = "embedding"
+    describe_key = "row_entries"
+
+    def __init__(self, params, prefix, dtype, device):
+        super().__init__(params, prefix, dtype, device)
+        self.vocab, self.hidden, self.streams = int(params["vocab"]), int(params["hidden"]), int(params.get("streams") or 1)
+        b = params.get("bigram")
+        self.hash = (int(b["buckets"]), int(b["mul_prev"]), int(b["mul_cur"])) if b else None
+        self.table: torch.Tensor = None
+        self.pairs: torch.Tensor = None
+        self.states: Dict[str, torch.Tensor] = {}
+
+    @classmethod
+    def weight_specs(cls, params, prefix) -> List[WeightSpec]:
+        h = int(params["hidden"])
+        specs = [WeightSpec(params["table"], (int(params["vocab"]), h), MATRIX)]
+        if params.get("bigram"):
+            specs.append(WeightSpec(params["pairs"], (int(params["bigram"]["buckets"]) + 1, h), MATRIX))
+        return specs
+
+    @classmethod
+    def state_needs(cls, params) -> List[StateNeed]:
+        return [StateNeed("last_token", (1,), torch.int32)] if params.get("bigram") else []
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.table = tensors[self.params["table"]].contiguous()
+        if self.hash:
+            self.pairs = tensors.pop(self.params["pairs"]).to(self.table.dtype).contiguous()
+
+    def describe_step(self, layout, put) -> torch.Tensor:
+        return describe_row_entries(layout, put)
+
+    def forward_step(self, ctx) -> torch.Tensor:
+        out = torch.empty((ctx.token_ids.numel(), self.streams, self.hidden), dtype=torch.float32, device=ctx.token_ids.device)
+        return ops.embed_bigram(self.table, self.pairs, self.hash, ctx.token_ids, self.states.get("last_token"),
+                                ctx.extras[self.describe_key], ctx.entry_q_start, ctx.entry_q_len, ctx.entry_slot, out)
+
+
 class LinearHead(Part):
     """params: ``vocab``, ``hidden``, ``name``, ``tied_to`` (None, or the full
     name of the embedding table to use instead of a weight of its own),
@@ -129,4 +178,5 @@ class LinearHead(Part):
 
 register_part("embedding", "token_embedding", TokenEmbedding)
 register_part("embedding", "sinusoid_norm_embedding", SinusoidNormEmbedding)
+register_part("embedding", "bigram_embedding", BigramEmbedding)
 register_part("lm_head", "linear_head", LinearHead)

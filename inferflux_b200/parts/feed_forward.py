@@ -234,14 +234,20 @@ class RoutedExperts(Part):
         ``route`` ``chosen``:  weights = softmax over the chosen logits alone
         ``route`` ``all``:     s = softmax(z) over every expert; weights = the chosen s over their sum (+ 1e-20)
         either times ``scale``
+        ``correction``: a stored number per expert joins its score s (``route`` ``all``) for the choice, not for the weight
         expert e, ``activation`` ``swiglu``:  W_down_e ( silu(W_gate_e x) * (W_up_e x) )
                   ``activation`` ``relu2``:   W_down_e ( relu(W_up_e x)^2 )                      no biases
+                  ``activation`` ``clamped_glu``:  W_down_e ( g * sigmoid(alpha g) * (u + shift) ),  g = min(W_gate_e x, limit),
+                                          u = clamp(W_up_e x, -limit, limit)
+        ``identity``: so many more outputs of the router, behind the experts', stand for the identity: a token that
+                  chooses one adds its own row, weighted
         ``shared`` (an intermediate size): one more expert of the ``relu2`` form that every token runs, added unweighted
 
     The experts' matrices are stacked at load; the (token, expert) pairs are sorted by expert on the device and
     run as tiles of one expert each, so nothing waits for the host and a step of single tokens is captured like
-    any other.  params: ``hidden``, ``intermediate`` (of one expert), ``experts``, ``top``, ``activation``, ``route``,
-    ``scale``, ``router_bias`` (default true), ``shared``, ``name`` (tensors ``<prefix>.<name>.router``, ``.router.b``,
+    any other.  params: ``hidden``, ``intermediate`` (of one expert), ``experts``, ``identity`` (default 0), ``top``,
+    ``activation`` (``clamped_glu`` with ``limit``, ``alpha``, ``shift``), ``route``, ``scale``, ``correction``, ``router_bias``
+    (default true), ``shared``, ``name`` (tensors ``<prefix>.<name>.router``, ``.router.b``, ``.correction``,
     ``.e<i>.{gate,up,down}``, ``.shared.{up,down}``)."""
 
     family = "feed_forward"
@@ -250,12 +256,19 @@ class RoutedExperts(Part):
         super().__init__(params, prefix, dtype, device)
         self.hidden, self.intermediate = int(params["hidden"]), int(params["intermediate"])
         self.experts, self.top = int(params["experts"]), int(params["top"])
-        if not 1 <= self.top <= min(self.experts, 64):
+        self.outputs = self.experts + int(params.get("identity") or 0)          # of the router
+        if not 1 <= self.top <= min(self.outputs, 64):
             raise ValueError(f"routed_experts: top {self.top} must be within 1..min(experts, 64)")
-        self.activation = {"swiglu": ops.MOE_SWIGLU, "relu2": ops.MOE_RELU2}.get(params.get("activation", "swiglu"))
+        self.activation = {"swiglu": ops.MOE_SWIGLU, "relu2": ops.MOE_RELU2,
+                           "clamped_glu": ops.MOE_CLAMPED_GLU}.get(params.get("activation", "swiglu"))
         self.over_all = {"chosen": False, "all": True}.get(params.get("route", "chosen"))
         if self.activation is None or self.over_all is None:
-            raise ValueError("routed_experts: activation is 'swiglu' or 'relu2', route is 'chosen' or 'all'")
+            raise ValueError("routed_experts: activation is 'swiglu', 'relu2' or 'clamped_glu', route is 'chosen' or 'all'")
+        self.limits = (float(params["limit"]), float(params.get("alpha", 1.702)), float(params.get("shift", 1.0))) \
+            if self.activation == ops.MOE_CLAMPED_GLU else (0.0, 0.0, 0.0)
+        if params.get("correction") and not self.over_all:
+            raise ValueError("routed_experts: a correction of the choice joins the scores of route 'all'")
+        self.correction: torch.Tensor = None
         self.scale = float(params.get("scale", 1.0))
         self.shared = self._shared(params, prefix, dtype, device)
         self.router: Linear = None
@@ -277,10 +290,13 @@ class RoutedExperts(Part):
     def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
         h, i, e = int(params["hidden"]), int(params["intermediate"]), int(params["experts"])
         n = lambda leaf: cls.full_name(prefix, params, leaf)
-        specs = [WeightSpec(n("router"), (e, h), MATRIX, std=0.5)]
+        outputs = e + int(params.get("identity") or 0)
+        specs = [WeightSpec(n("router"), (outputs, h), MATRIX, std=0.5)]
         if params.get("router_bias", True):
-            specs.append(WeightSpec(n("router.b"), (e,), VECTOR, std=0.5))
-        mats = ("gate", "up") if params.get("activation", "swiglu") == "swiglu" else ("up",)
+            specs.append(WeightSpec(n("router.b"), (outputs,), VECTOR, std=0.5))
+        if params.get("correction"):
+            specs.append(WeightSpec(n("correction"), (outputs,), VECTOR, std=0.1))
+        mats = ("up",) if params.get("activation", "swiglu") == "relu2" else ("gate", "up")
         for k in range(e):
             specs += [WeightSpec(n(f"e{k}.{x}"), (i, h), MATRIX) for x in mats] + [WeightSpec(n(f"e{k}.down"), (h, i), MATRIX)]
         sp = cls._shared(params, prefix)
@@ -293,7 +309,9 @@ class RoutedExperts(Part):
         # The router's products are 32-bit whatever the engine: a bfloat16 weight times a bfloat16 input is exact
         # in float32, and the sums are float32 (the library's product or the weight-streaming kernel).
         self.router = Linear(tensors.pop(n("router")), tensors.pop(n("router.b")) if self.params.get("router_bias", True) else None)
-        ups = ("gate", "up") if self.activation == ops.MOE_SWIGLU else ("up",)
+        if self.params.get("correction"):
+            self.correction = tensors.pop(n("correction")).to(torch.float32).contiguous()
+        ups = ("up",) if self.activation == ops.MOE_RELU2 else ("gate", "up")
         mats = [[tensors.pop(n(f"e{k}.{x}")) for x in (*ups, "down")] for k in range(self.experts)]
         kinds = {m.dtype for row in mats for m in row}
         cast = (lambda m: m.float()) if len(kinds) > 1 else (lambda m: m)
@@ -304,11 +322,11 @@ class RoutedExperts(Part):
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         logits = self.router.forward(x, out_dtype=torch.float32)
-        chosen, weights = ops.moe_route(logits, self.top, self.over_all, self.scale)
+        chosen, weights = ops.moe_route(logits, self.top, self.over_all, self.scale, self.correction)
         xe = x
         if x.dtype != self.gate_up.dtype:
             xe = ops.convert(x.contiguous(), torch.empty(x.shape, dtype=self.gate_up.dtype, device=x.device))
-        out = ops.moe_experts(xe.contiguous(), self.gate_up, self.down, chosen, weights, self.activation)
+        out = ops.moe_experts(xe.contiguous(), self.gate_up, self.down, chosen, weights, self.activation, *self.limits)
         if self.shared is not None:
             y = self.shared.forward(x, ctx)
             y, parts = (y.tensor, y.count) if isinstance(y, PartialSums) else (y, 1)

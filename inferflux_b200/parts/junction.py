@@ -14,6 +14,10 @@ is the same in every pass and is made once per step; the sum is float32.
 ``loop_step``: ``x <- x + x0 + step[t]``, without ``x0`` ahead of the first
 pass.  It rewrites nothing itself: it hands what it adds on with the pending
 sum, and the norm that comes next adds it all.
+
+``stream_join``: how a sublayer's result joins a stream of several copies; like
+``loop_step`` it only says what is to be done, and the norm that comes next
+does it.
 """
 from __future__ import annotations
 
@@ -24,7 +28,7 @@ import torch
 from ..config.registry import register_part
 from ..kernels import ops
 from ..weights.loader import MATRIX, VECTOR, WeightSpec
-from .base import JoinedSum, Part, RunInfo
+from .base import JoinedSum, Part, RunInfo, StreamMix
 from .linear import Linear
 
 
@@ -100,6 +104,35 @@ class LoopStep(Part):
         return JoinedSum(delta, ctx.embedding_output if t > 0 else None, self.step[t])
 
 
+class StreamJoin(Part):
+    """``X_t <- sum_s mix[s, t] X_s + factor * out[t] * y`` for a sublayer's result ``y`` and the stream's copies ``X_s``.
+    params: ``streams``, ``factor`` (default 1; it joins ``out`` at load, in float32), ``name`` (tensors
+    ``<prefix>.<name>.mix`` ``[streams, streams]`` and ``.out`` ``[streams]``)."""
+
+    family = "junction"
+
+    def __init__(self, params, prefix, dtype, device):
+        super().__init__(params, prefix, dtype, device)
+        self.streams, self.factor = int(params["streams"]), float(params.get("factor", 1.0))
+        self.mix: torch.Tensor = None
+        self.out: torch.Tensor = None
+
+    @classmethod
+    def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
+        s = int(params["streams"])
+        return [WeightSpec(cls.full_name(prefix, params, "mix"), (s, s), VECTOR, std=s ** -0.5),
+                WeightSpec(cls.full_name(prefix, params, "out"), (s,), VECTOR, init="one_plus_normal", std=0.1)]
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        f32 = lambda leaf: tensors.pop(self.full_name(self.prefix, self.params, leaf)).to(torch.float32)
+        self.mix = f32("mix").contiguous()
+        self.out = (f32("out") * self.factor).contiguous()
+
+    def pending(self, delta, ctx, run: RunInfo) -> StreamMix:
+        return StreamMix(delta, self.mix, self.out)
+
+
+register_part("junction", "stream_join", StreamJoin)
 register_part("junction", "loop_entry", LoopEntry)
 register_part("junction", "loop_step", LoopStep)
 register_part("junction", "add_embedding", AddEmbedding)

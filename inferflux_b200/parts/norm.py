@@ -15,7 +15,7 @@ import torch
 from ..config.registry import register_part
 from ..kernels import ops
 from ..weights.loader import VECTOR, WeightSpec
-from .base import BranchMean, JoinedSum, NormedDelta, Part, PartialSums, ScaledSum
+from .base import BranchMean, JoinedSum, NormedDelta, Part, PartialSums, ScaledSum, StreamMix
 
 
 class RMSNorm(Part):
@@ -167,6 +167,53 @@ class GroupRMSNorm(RMSNorm):
         return ops.add_group_rmsnorm(residual, a, self.weight, self.eps, self.groups, out, rows, fa, b, fb, x, vec)
 
 
+class StreamRMSNorm(RMSNorm):
+    """RMS norm of a weighted sum of the stream's copies, fused with what is pending for them: with ``X`` float32
+    ``[N, streams, hidden]`` and a :class:`StreamMix` pending,
+
+        X_t <- sum_s mix[s, t] X_s + out[t] * value;   u = sum_s reads[s] X_s;   result = u / sqrt(mean(u^2) + eps) * weight
+
+    in one pass over the row.  params: those of ``rmsnorm``, ``streams``, and ``reads``: the leaf name of the weights
+    ``[streams]`` (None = ones: the plain sum)."""
+
+    family = "norm"
+
+    def __init__(self, params, prefix, dtype, device):
+        super().__init__(params, prefix, dtype, device)
+        self.streams = int(params["streams"])
+        if not 1 <= self.streams <= ops.MAX_STREAMS:
+            raise ValueError(f"stream_rmsnorm: {self.streams} streams are not within 1..{ops.MAX_STREAMS}")
+        self.reads: Optional[torch.Tensor] = None
+
+    @classmethod
+    def weight_specs(cls, params: Dict[str, Any], prefix: str) -> List[WeightSpec]:
+        specs = super().weight_specs(params, prefix)
+        if params.get("reads"):
+            specs.append(WeightSpec(cls.full_name(prefix, {}, params["reads"]), (int(params["streams"]),), VECTOR, std=0.5))
+        return specs
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        super().load(tensors)
+        if self.params.get("reads"):
+            self.reads = tensors.pop(self.full_name(self.prefix, {}, self.params["reads"])).to(torch.float32).contiguous()
+        else:
+            self.reads = torch.ones(self.streams, dtype=torch.float32, device=self.weight.device)
+
+    def forward(self, residual: torch.Tensor, delta, out: Optional[torch.Tensor] = None,
+                rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        n_rows = rows.numel() if rows is not None else residual.shape[0]
+        if out is None:
+            out = torch.empty((n_rows, self.hidden), dtype=self.dtype, device=residual.device)
+        value = mix = out_w = None
+        if delta is not None:
+            if not isinstance(delta, StreamMix):
+                raise TypeError("stream_rmsnorm takes what a stream_join made of a sublayer's result")
+            value, mix, out_w = delta.value, delta.mix, delta.out
+            value = value.tensor if isinstance(value, PartialSums) else value
+        return ops.stream_mix_norm(residual, value, mix, out_w, self.reads, self.weight, self.eps, out, rows)
+
+
+register_part("norm", "stream_rmsnorm", StreamRMSNorm)
 register_part("norm", "rmsnorm", RMSNorm)
 register_part("norm", "group_rmsnorm", GroupRMSNorm)
 register_part("norm", "layernorm", LayerNorm)

@@ -302,7 +302,7 @@ class WindowAttention(Part):
         fast = (self.TENSOR_CORES and x.dtype == torch.bfloat16 and self.dim == self.vdim and out.is_contiguous()
                 and self.dim in ops.FAST_ATTENTION_HEAD_DIMS)
         singles = (step.single_entry, step.single_q0, step.n_single)
-        if fast and step.n_dec and not (self.softcap or self.keep_first or self.sink):
+        if fast and step.n_dec and not (self.keep_first or self.sink):
             # entries of one token: the split tensor-core kernel, which reads a key once for all the heads that share it
             max_keys = min(ctx.max_ctx_len, abs(self.reach)) if self.reach else ctx.max_ctx_len
             n_splits = ops.attn_decode_splits(step.n_dec, self.heads, self.kv_heads, self.dim, max_keys)
@@ -312,7 +312,7 @@ class WindowAttention(Part):
                 part_ml = torch.empty(step.n_dec * self.heads * n_splits * 2, dtype=torch.float32, device=x.device)
             ops.attn_decode_bf16(q, q.stride(0), out, *pages, step.dec_entry, step.n_dec, ctx.entry_q_start, ctx.entry_q_len,
                                  ctx.entry_ctx_start, part_o, part_ml, self.heads, self.kv_heads, self.dim, self.scale,
-                                 self.reach, n_splits, gate=gate, **more)
+                                 self.reach, n_splits, gate=gate, softcap=self.softcap, **more)
             singles = (step.short_entry, step.short_q0, step.n_short)
         if singles[2]:          # decoded tokens and the shortest portions: a block a token and head
             ops.attn_paged_options(q, q.stride(0), out, *pages, *singles, *common, *rest, single_tokens=True, **more)
