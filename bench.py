@@ -256,9 +256,29 @@ def zetivik_config(size: str, layers: int):
                 layers=[pair if i % 2 == 0 else lightning for i in range(layers)])
 
 
+def kibilix_config(size: str, layers: int):
+    """A Kibilix config.json at the widths of one of the family sizes above: layers in turn attention (the family's heads and
+    kv heads of 128 in chunks of 8,192, capped scores, band-scaled rotary positions) and the delta rule with a decay per key
+    channel (half as many value heads of 128 x 128, two to a query and key head, four taps, inner projections of 128); every
+    second pair of layers with a squared-relu feed-forward of one and a half times the family's width, the others with 16
+    clamped gated experts of a quarter of that width and two identity experts of which a token takes 4; four streams; hashed
+    token pairs; no loop."""
+    _, hidden, heads, kv_heads, inter, vocab, _ = SIZES[size]
+    dense = dict(kind="dense", ff=inter * 3 // 2)                # as many weights as a gated one of the family's width
+    moe = dict(kind="moe", expert=dict(ff=inter // 4 // 8 * 8, limit=7.0), router=dict(experts=16, identity=2, top=4))
+    attn = dict(type="attention", mixer=dict(
+        heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=8192),
+        rot=dict(dims=128, base=500000.0, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))))
+    delta = dict(type="channel_delta", mixer=dict(heads=heads // 2, kv_heads=heads // 4, dim=128, vdim=128, conv=4))
+    return dict(architecture="Kibilix", width=hidden, vocab=vocab, norm=dict(eps=1e-6), streams=4, residual_mult=0.7,
+                embedding=dict(bigram=dict(buckets=vocab // 2 + 1, mul_prev=31, mul_cur=17)),
+                layers=[dict(delta if i % 2 else attn, mlp=moe if i % 4 >= 2 else dense) for i in range(layers)])
+
+
 #: --arch: the design's config.json at a size, and the design it is timed beside (the closest one that was there)
 DESIGNS = {"kunonex": (kunonex_config, "qwen2"), "pemorax": (pemorax_config, "qwen2"), "tekosun": (tekosun_config, "pemorax"),
-           "malazen": (malazen_config, "pemorax"), "zetivik": (zetivik_config, "malazen")}
+           "malazen": (malazen_config, "pemorax"), "zetivik": (zetivik_config, "malazen"),
+           "kibilix": (kibilix_config, "zetivik")}
 
 
 def architecture_workload(args) -> int:
