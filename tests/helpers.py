@@ -545,3 +545,110 @@ def make_zetivik_folder(cfg: dict, seed: int, folder: Optional[str] = None, **kw
         json.dump(cfg, f)
     write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
     return folder
+
+
+def _kb_attn(heads, dim, kv_heads=None, vdim=None, scale=None, chunk=None, softcap=None, rot=None, mlp=None):
+    m = dict(heads=heads, dim=dim)
+    for key, v in (("kv_heads", kv_heads), ("vdim", vdim), ("scale", scale), ("softcap", softcap), ("rot", rot)):
+        if v is not None:
+            m[key] = v
+    if chunk is not None:
+        m["mask"] = dict(size=chunk)
+    return dict(type="attention", mixer=m, mlp=mlp)
+
+
+def _kb_delta(heads, dim, conv, kv_heads=None, vdim=None, mlp=None):
+    m = dict(heads=heads, dim=dim, conv=conv)
+    for key, v in (("kv_heads", kv_heads), ("vdim", vdim)):
+        if v is not None:
+            m[key] = v
+    return dict(type="channel_delta", mixer=m, mlp=mlp)
+
+
+def _kb_moe(ff, limit, experts, top, identity=0):
+    router = dict(experts=experts, top=top)
+    if identity:
+        router["identity"] = identity
+    return dict(kind="moe", expert=dict(ff=ff, limit=limit), router=router)
+
+
+# Tiny Kibilix configurations that differ in every size, option and order of layers.  A: three streams, key, value and
+# state sizes all different, shared key/value heads in both mixers, chunks of 20 and 33, partly rotated heads with scaled
+# and unscaled frequencies, identity experts, a layer without feed-forward, a loop from layer 0 that runs three times.
+KB_A = dict(architecture="Kibilix", width=64, vocab=300, norm=dict(eps=1e-5), streams=3, residual_mult=0.8,
+            embedding=dict(bigram=dict(buckets=101, mul_prev=53, mul_cur=11)), layers=[
+    _kb_attn(4, 16, kv_heads=2, vdim=24, scale=0.3, chunk=20, softcap=6.0,
+             rot=dict(dims=12, base=1000.0, scaling=dict(factor=4.0, low=1.0, high=8.0, original=64)), mlp=dict(kind="dense", ff=96)),
+    _kb_delta(4, 12, 4, kv_heads=2, vdim=20, mlp=_kb_moe(40, 1.0, 5, 3, identity=2)),
+    _kb_attn(2, 32, kv_heads=1, scale=0.2, chunk=33, softcap=9.0, rot=dict(dims=32, base=500.0))], loop=dict(start=0, stop=2, times=3))
+# B: sizes that are no multiple of 4 or 8 anywhere, two streams, no token pairs, chunks shorter than a page and none, no
+# rotation, no cap and no scale in one layer, one tap and two, as many key/value heads as heads, no identity experts, one
+# expert a token, layers without feed-forward, no loop
+KB_B = dict(architecture="Kibilix", width=50, vocab=77, norm=dict(eps=3e-6), streams=2, residual_mult=1.0, layers=[
+    _kb_delta(2, 6, 1, vdim=10), _kb_attn(3, 10, vdim=6, chunk=7, mlp=_kb_moe(35, 0.5, 3, 2)),
+    _kb_delta(6, 10, 2, kv_heads=3, vdim=6, mlp=_kb_moe(18, 2.0, 2, 1)),
+    _kb_attn(5, 6, kv_heads=1, vdim=10, scale=0.5, softcap=4.0, rot=dict(dims=2, base=50.0), mlp=dict(kind="dense", ff=45))])
+# C: heads of 64 (the size tensor-core kernels take), chunks longer than several pages, four streams, five taps, states of
+# 64 x 64, experts whose sizes the tensor-core products take, a loop over the last two layers
+KB_C = dict(architecture="Kibilix", width=128, vocab=200, norm=dict(eps=1e-6), streams=4, residual_mult=0.6,
+            embedding=dict(bigram=dict(buckets=64, mul_prev=7, mul_cur=3)), layers=[
+    _kb_delta(2, 64, 5, mlp=_kb_moe(64, 1.5, 4, 2, identity=1)),
+    _kb_attn(4, 64, kv_heads=2, scale=0.125, chunk=70, softcap=8.0, rot=dict(dims=64, base=200000.0), mlp=dict(kind="dense", ff=160)),
+    _kb_attn(2, 64, scale=0.1, chunk=48, softcap=15.0,
+             rot=dict(dims=16, base=1e4, scaling=dict(factor=8.0, low=1.0, high=4.0, original=128)), mlp=_kb_moe(96, 0.8, 6, 3, identity=3)),
+    _kb_delta(4, 32, 4, kv_heads=2, vdim=48, mlp=None)], loop=dict(start=2, stop=4, times=2))
+KB = {"A": KB_A, "B": KB_B, "C": KB_C}
+
+
+def kibilix_tensors(cfg: dict, seed: int, sharpen: float = 6.0):
+    """Random tensors (bfloat16 matrices) for a Kibilix configuration.  ``sharpen`` multiplies the attentions' query and
+    key projections, so that the softmax is peaked on single keys wherever they lie in the chunk (a lost key would hide
+    below the bfloat16 tolerance otherwise); the other projections are enlarged so that every sublayer carries weight in
+    the streams and the experts' clamps bite, and the decays' sizes are set so that a state lost many tokens back would show."""
+    from inferflux_b200.config import load_config
+    from inferflux_b200.config.registry import build_spec
+    from inferflux_b200.engine.model import Model
+    from inferflux_b200.weights.random_init import random_tensors
+    config = load_config(json.loads(json.dumps(cfg)))
+    specs = Model(build_spec(config), torch.float32, "cpu").weight_specs()
+    tensors = random_tensors(specs, seed, torch.bfloat16, None, "cpu")
+    attention = {f"l{i}" for i, l in enumerate(cfg["layers"]) if l["type"] == "attention"}
+    for name in tensors:
+        f, add = 1.0, 0.0
+        if name.endswith((".mix.q", ".mix.k")):
+            f = sharpen if name.split(".")[0] in attention else 5.0
+        elif name.endswith((".mix.v", ".mix.o", ".mix.b", ".mix.a1", ".mix.g1", ".up", ".down", ".gate")):
+            f = 5.0
+        elif name.endswith((".a2", ".g2")):
+            f = 4.0
+        elif name.endswith(".router"):
+            f = 0.3
+        elif name.endswith(".correction"):
+            f = 2.0
+        elif name.endswith(".A_log"):
+            add = -2.0
+        elif name.endswith(".conv"):
+            add = 0.3
+        elif name in ("embed", "bigram"):
+            f = 20.0
+        elif name == "head":
+            f = 5.0
+        if f != 1.0 or add:
+            tensors[name] = (tensors[name].float() * f + add).to(tensors[name].dtype)
+        # the two-step projections' inner sizes are the tensors' own: two odd ones, which differ
+        for leaf, rank in (("a", 21), ("g", 14)):
+            if name.endswith(f".mix.{leaf}1"):
+                tensors[name] = tensors[name][:rank].contiguous()
+            elif name.endswith(f".mix.{leaf}2"):
+                tensors[name] = tensors[name][:, :rank].contiguous()
+    return config, tensors
+
+
+def make_kibilix_folder(cfg: dict, seed: int, folder: Optional[str] = None, **kw) -> str:
+    from inferflux_b200.weights.safetensors_io import write_safetensors
+    folder = folder or tempfile.mkdtemp(prefix="ifx_kb_")
+    config, tensors = kibilix_tensors(cfg, seed, **kw)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
+    return folder
