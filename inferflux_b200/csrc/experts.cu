@@ -26,12 +26,12 @@ template <int MODE> __device__ __forceinline__ float glu(float g, float u, const
 }
 
 __global__ void __launch_bounds__(256)
-moe_route_kernel(const float* __restrict__ logits, int n_tokens, int experts, int top, int over_all, float scale,
+moe_route_kernel(const float* __restrict__ logits, long long stride, int n_tokens, int experts, int top, int over_all, float scale,
                  const float* __restrict__ correction, int* __restrict__ chosen, float* __restrict__ weights) {
   pdl_enter();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= n_tokens) return;
-  const float* z = logits + (size_t)t * experts;
+  const float* z = logits + (size_t)t * stride;
   int ids[MAX_TOP]; float vals[MAX_TOP];
   float most = -INFINITY, all = 0.0f;
   if (over_all) {                        // the scores' softmax over every expert
@@ -73,6 +73,68 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int experts, in
   for (int k = lane; k < top; k += 32) {
     chosen[(size_t)t * top + k] = ids[k];
     weights[(size_t)t * top + k] = expf(vals[k] - vals[0]) / sum * scale;
+  }
+}
+
+// The same with a lane's share of the router's outputs in registers (EPL of them a lane: lane, lane + 32, ...).
+template <int EPL>
+__global__ void __launch_bounds__(256)
+moe_route_regs_kernel(const float* __restrict__ logits, long long stride, int n_tokens, int experts, int top, int over_all, float scale,
+                      const float* __restrict__ correction, int* __restrict__ chosen, float* __restrict__ weights) {
+  pdl_enter();
+  const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= n_tokens) return;
+  float score[EPL], by[EPL];             // what weighs, what the choice goes by
+  float most = -INFINITY;
+#pragma unroll
+  for (int i = 0; i < EPL; ++i) {
+    const int e = lane + 32 * i;
+    score[i] = by[i] = e < experts ? logits[(size_t)t * stride + e] : -INFINITY;
+    most = fmaxf(most, score[i]);
+  }
+  most = warp_max(most);
+  float all = 0.0f;
+#pragma unroll
+  for (int i = 0; i < EPL; ++i) {
+    score[i] = expf(score[i] - most);
+    all += score[i];
+  }
+  if (over_all) {
+    all = warp_sum(all);
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+      const int e = lane + 32 * i;
+      score[i] = score[i] / all;
+      if (correction && e < experts) by[i] = score[i] + correction[e];
+    }
+  }
+  int my_id[2] = {0, 0};                 // lane k holds choices k and k + 32
+  float my_score[2] = {0.0f, 0.0f}, sum = 0.0f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY, s = 0.0f; int arg = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < EPL; ++i)
+      if (by[i] > best) { best = by[i]; s = score[i]; arg = lane + 32 * i; }
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, s, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; s = os; }
+    }
+#pragma unroll
+    for (int i = 0; i < EPL; ++i)
+      if (lane + 32 * i == arg) by[i] = -INFINITY;
+    sum += s;
+    if ((k & 31) == lane) {
+      if (k < 32) { my_id[0] = arg; my_score[0] = s; }
+      else { my_id[1] = arg; my_score[1] = s; }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int k = lane + 32 * i;
+    if (k >= top) continue;
+    chosen[(size_t)t * top + k] = my_id[i];
+    weights[(size_t)t * top + k] = my_score[i] / (over_all ? sum + 1e-20f : sum) * scale;
   }
 }
 
@@ -201,12 +263,17 @@ moe_product_kernel(const TA* __restrict__ A, long long lda, int gather_div /* 0:
 
 // The same tile product for bfloat16 and short tiles (16 rows: steps of single tokens) on tensor cores: the 16 rows
 // are the rows of one m16n8k16 MMA, a warp owns 16 of the block's 64 rows of W_e (SwiGLU: 8 gate rows and the 8 up
-// rows that belong to them), operands go through shared memory 64 K at a time by 16-byte loads.  Such a step is
+// rows that belong to them), operands go through a ring in shared memory 64 K at a time by 16-byte asynchronous copies.  Such a step is
 // bound by reading the chosen experts' weights once; the arithmetic of the FFMA tiles above took three times as long.
 __device__ __forceinline__ void moe_mma_bf16(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+__device__ __forceinline__ void moe_cp_async16(void* dst_shared, const void* src, bool valid) {
+  const unsigned dst = (unsigned)__cvta_generic_to_shared(dst_shared);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
 }
 
 template <typename TO, int MODE>
@@ -217,8 +284,9 @@ moe_product_mma_kernel(const bf16* __restrict__ A, long long lda, int gather_div
   constexpr bool SWIGLU = MODE == MODE_SWIGLU || MODE == MODE_CLAMPED;
   constexpr int BM = 16, BN = 64, BK = 64, LD = BK + 8;
   pdl_enter();
-  __shared__ __align__(16) bf16 As[BM][LD];
-  __shared__ __align__(16) bf16 Ws[BN][LD];
+  constexpr int STAGES = 4;                          // operands of so many steps of BK are here or on their way
+  __shared__ __align__(16) bf16 As[STAGES][BM][LD];
+  __shared__ __align__(16) bf16 Ws[STAGES][BN][LD];
   __shared__ int rows[BM];
   const int tile = blockIdx.y;
   const int e = tile_expert[tile];
@@ -236,37 +304,49 @@ moe_product_mma_kernel(const bf16* __restrict__ A, long long lda, int gather_div
   const int r0 = SWIGLU ? 8 * warp + g : 16 * warp + g;
   const int r1 = SWIGLU ? cols + 8 * warp + g : 16 * warp + 8 + g;
   float acc0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, acc1[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-  for (int k0 = 0; k0 < K; k0 += BK) {
-    {
-      const int r = tid >> 3, c8 = (tid & 7) * 8;
-      const int src = rows[r];
-      *reinterpret_cast<uint4*>(&As[r][c8]) = (src >= 0 && k0 + c8 < K)
-          ? *reinterpret_cast<const uint4*>(A + (size_t)src * lda + k0 + c8) : zero;
-    }
+  // what this thread copies of every step: 16 bytes of a row of A and of four rows of W_e
+  const int c8 = (tid & 7) * 8, ra = tid >> 3;
+  const bf16* a_src = rows[ra] >= 0 ? A + (size_t)rows[ra] * lda : nullptr;
+  const bf16* w_src[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int v = tid + 128 * i, c = v >> 3, c8 = (v & 7) * 8;
-      const int col = SWIGLU ? (c < cols ? n0 + c : n0 + c - cols) : n0 + c;        // the output column this row of the tile feeds
-      const int wrow = SWIGLU && c >= cols ? n_out + col : col;
-      *reinterpret_cast<uint4*>(&Ws[c][c8]) = (col < n_out && k0 + c8 < K)
-          ? *reinterpret_cast<const uint4*>(We + (size_t)wrow * K + k0 + c8) : zero;
-    }
-    __syncthreads();
+  for (int i = 0; i < 4; ++i) {
+    const int c = ra + 16 * i;
+    const int col = SWIGLU ? (c < cols ? n0 + c : n0 + c - cols) : n0 + c;          // the output column this row of the tile feeds
+    w_src[i] = col < n_out ? We + (size_t)(SWIGLU && c >= cols ? n_out + col : col) * K : nullptr;
+  }
+  auto stage = [&](int s, int k0) {                  // sources that do not exist give zeros
+    const bool in = k0 + c8 < K;
+    moe_cp_async16(&As[s][ra][c8], a_src && in ? a_src + k0 + c8 : A, a_src && in);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) moe_cp_async16(&Ws[s][ra + 16 * i][c8], w_src[i] && in ? w_src[i] + k0 + c8 : W, w_src[i] && in);
+  };
+  const int steps = (K + BK - 1) / BK;
+#pragma unroll
+  for (int s = 0; s < STAGES - 1; ++s) {
+    if (s < steps) stage(s, s * BK);
+    cp_async_commit();
+  }
+  for (int i = 0; i < steps; ++i) {
+    asm volatile("cp.async.wait_group %0;\n" ::"n"(STAGES - 2) : "memory");
+    __syncthreads();                                 // step i is here for everyone, and the place of step i - 1 is free
+    const int nx = i + STAGES - 1;
+    if (nx < steps) stage(nx % STAGES, nx * BK);
+    cp_async_commit();
+    const int s = i % STAGES;
 #pragma unroll
     for (int kk = 0; kk < BK; kk += 16) {
       unsigned a[4];
-      a[0] = *reinterpret_cast<const unsigned*>(&As[g][kk + 2 * t]);
-      a[1] = *reinterpret_cast<const unsigned*>(&As[g + 8][kk + 2 * t]);
-      a[2] = *reinterpret_cast<const unsigned*>(&As[g][kk + 8 + 2 * t]);
-      a[3] = *reinterpret_cast<const unsigned*>(&As[g + 8][kk + 8 + 2 * t]);
-      moe_mma_bf16(acc0, a, *reinterpret_cast<const unsigned*>(&Ws[r0][kk + 2 * t]),
-                   *reinterpret_cast<const unsigned*>(&Ws[r0][kk + 8 + 2 * t]));
-      moe_mma_bf16(acc1, a, *reinterpret_cast<const unsigned*>(&Ws[r1][kk + 2 * t]),
-                   *reinterpret_cast<const unsigned*>(&Ws[r1][kk + 8 + 2 * t]));
+      a[0] = *reinterpret_cast<const unsigned*>(&As[s][g][kk + 2 * t]);
+      a[1] = *reinterpret_cast<const unsigned*>(&As[s][g + 8][kk + 2 * t]);
+      a[2] = *reinterpret_cast<const unsigned*>(&As[s][g][kk + 8 + 2 * t]);
+      a[3] = *reinterpret_cast<const unsigned*>(&As[s][g + 8][kk + 8 + 2 * t]);
+      moe_mma_bf16(acc0, a, *reinterpret_cast<const unsigned*>(&Ws[s][r0][kk + 2 * t]),
+                   *reinterpret_cast<const unsigned*>(&Ws[s][r0][kk + 8 + 2 * t]));
+      moe_mma_bf16(acc1, a, *reinterpret_cast<const unsigned*>(&Ws[s][r1][kk + 2 * t]),
+                   *reinterpret_cast<const unsigned*>(&Ws[s][r1][kk + 8 + 2 * t]));
     }
-    __syncthreads();
   }
+  cp_async_wait_all();
   // accumulator layout: [0], [1] = row g, columns 2t and 2t + 1; [2], [3] = row g + 8, the same columns
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
@@ -389,6 +469,18 @@ int launch_products(const void* x, const void* w_up, const void* w_down, const i
 }
 }  // namespace
 
+// The same 16 bytes a thread at a time (rows on 16-byte boundaries); elements of any type, `units` of 16 bytes a row.
+__global__ void __launch_bounds__(256)
+moe_gather_rows_vec_kernel(const uint4* __restrict__ x, const int* __restrict__ sorted_pair, uint4* __restrict__ xs, int units, int top) {
+  pdl_enter();
+  const int r = blockIdx.x;
+  const int pair = sorted_pair[r];
+  const uint4* src = pair >= 0 ? x + (size_t)(pair / top) * units : nullptr;
+  uint4* dst = xs + (size_t)r * units;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < units; i += blockDim.x) dst[i] = src ? src[i] : make_uint4(0u, 0u, 0u, 0u);
+}
+
 // xs[r] = x[pair / top] for the pair at sorted row r, zeros where a row holds no pair
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -414,6 +506,13 @@ IFX_API int ifx_moe_group(const int* chosen, int pairs, int experts, int tile, i
 IFX_API int ifx_moe_gather_rows(const void* x, int dtype, const int* sorted_pair, void* xs, int rows, int hidden, int top,
                                 cudaStream_t stream) {
   if (rows <= 0) return 0;
+  const size_t bytes = (size_t)hidden * (dtype == IFX_BF16 ? 2 : 4);
+  if (!(bytes & 15) && !(((uintptr_t)x | (uintptr_t)xs) & 15)) {
+    const int units = (int)(bytes / 16);
+    const int rc = launch_pdl(moe_gather_rows_vec_kernel, dim3(rows), dim3(units >= 256 ? 256 : units >= 128 ? 128 : 64), 0, stream,
+                              (const uint4*)x, sorted_pair, (uint4*)xs, units, top);
+    return rc ? rc : IFX_LAUNCH_CHECK();
+  }
   const int rc = dtype == IFX_BF16
       ? launch_pdl(moe_gather_rows_kernel<bf16>, dim3(rows), dim3(256), 0, stream, (const bf16*)x, sorted_pair, (bf16*)xs, hidden, top)
       : launch_pdl(moe_gather_rows_kernel<float>, dim3(rows), dim3(256), 0, stream, (const float*)x, sorted_pair, (float*)xs, hidden, top);
@@ -429,16 +528,18 @@ IFX_API int ifx_moe_combine(const float* y, const int* pair_row, const float* we
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 
-// over_all 0: weights are the softmax over the chosen logits alone; 1: the softmax over every expert's logit, the
+// logits: rows of `experts` numbers, `stride` apart.  over_all 0: weights are the softmax over the chosen logits alone; 1: the softmax over every expert's logit, the
 // chosen ones' scores divided by their sum (+ 1e-20).  Either is multiplied by scale.  correction (float32 [experts] or null;
 // with over_all): the choice goes by score + correction, the weights by the score.
-IFX_API int ifx_moe_route(const float* logits, int n_tokens, int experts, int top, int over_all, float scale,
+IFX_API int ifx_moe_route(const float* logits, long long stride, int n_tokens, int experts, int top, int over_all, float scale,
                           const float* correction, int* chosen, float* weights, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (correction && !over_all) return IFX_ERR_UNSUPPORTED;
   if (top < 1 || top > MAX_TOP || top > experts) return IFX_ERR_UNSUPPORTED;
-  const int rc = launch_pdl(moe_route_kernel, dim3((n_tokens + 7) / 8), dim3(256), 0, stream, logits, n_tokens, experts, top,
-                            over_all, scale, correction, chosen, weights);
+  auto kern = experts <= 32 ? moe_route_regs_kernel<1> : experts <= 64 ? moe_route_regs_kernel<2> : experts <= 128 ? moe_route_regs_kernel<4>
+            : experts <= 256 ? moe_route_regs_kernel<8> : moe_route_kernel;
+  const int rc = launch_pdl(kern, dim3((n_tokens + 7) / 8), dim3(256), 0, stream, logits, stride, n_tokens, experts, top, over_all, scale,
+                            correction, chosen, weights);
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
 

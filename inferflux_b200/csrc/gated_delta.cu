@@ -216,16 +216,22 @@ gated_delta_step_kernel(GdArgs p) {
   }
 }
 
-// One decay per key channel.  The logarithms' running sums are kept to base two.
+// One decay per key channel.  The logarithms' running sums c are kept to base two.  Between the segment's halves the
+// exponentials factor: with m the sum at the first half's end, e^(c_i - c_j) = e^(c_i - m) e^(m - c_j) for i in the second and
+// j in the first half, neither factor above one, so a quarter of the pairs' square is a product of scaled rows; inside the
+// halves the differences are taken pair by pair.
 __global__ void __launch_bounds__(THREADS, 2)
 channel_delta_segments_kernel(GdArgs p) {
   extern __shared__ __align__(16) float sm[];
   pdl_enter();
+  constexpr int HALF = SEG / 2, EACH = SEG / (THREADS / 32);
   const int D = p.dim, V = p.vdim, DP = segscan::pad4(D), LD = row_ld(D);
   float* ks = sm;                          // [SEG][LD]
   float* qs = ks + SEG * LD;               // [SEG][LD]
   float* cs = qs + SEG * LD;               // [SEG][LD] running sums of log2 g per channel
-  float* L = cs + SEG * LD;                // [SEG][LLD]
+  float* km = cs + SEG * LD;               // [SEG][LD] keys: times e^(m - c) in the first half, e^(c - m) in the second
+  float* qm = km + SEG * LD;               // [HALF][LD] the second half's queries times e^(c - m)
+  float* L = qm + HALF * LD;               // [SEG][LLD]
   float* A = L + SEG * LLD;                // [SEG j][LLD] scores, transposed
   float* be = A + SEG * LLD;               // [SEG] beta
   const int seg = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
@@ -239,77 +245,117 @@ channel_delta_segments_kernel(GdArgs p) {
     const float rate = -1.4426950408889634f * expf(p.a_log[h]);
     const float* dec = p.dec + (size_t)row0 * p.dec_stride + h * D;
     const float* bias = p.dt_bias + h * D;
-    for (int i = tid >> 5; i < SEG; i += THREADS / 32)
-      for (int d = tid & 31; d < DP; d += 32)
-        cs[i * LD + d] = i < n && d < D ? rate * softplus(dec[(size_t)i * p.dec_stride + d] + bias[d]) : 0.0f;
+    const int i0 = tid >> 5;
+    for (int d = tid & 31; d < DP; d += 32) {
+      float x[EACH];
+#pragma unroll
+      for (int u = 0; u < EACH; ++u) {
+        const int i = i0 + u * (THREADS / 32);
+        x[u] = i < n && d < D ? dec[(size_t)i * p.dec_stride + d] : 0.0f;
+      }
+      const float bd = d < D ? bias[d] : 0.0f;
+#pragma unroll
+      for (int u = 0; u < EACH; ++u) {
+        const int i = i0 + u * (THREADS / 32);
+        cs[i * LD + d] = i < n && d < D ? rate * softplus(x[u] + bd) : 0.0f;
+      }
+    }
   }
   if (tid < SEG) be[tid] = tid < n ? write_rate(p, row0 + tid, h) : 0.0f;
   for (int idx = tid; idx < SEG * LLD; idx += THREADS) L[idx] = A[idx] = 0.0f;
   __syncthreads();
   for (int d = tid; d < DP; d += THREADS) {
-    float c = 0.0f;
+    float x[SEG];
 #pragma unroll
-    for (int i = 0; i < SEG; ++i) {
-      c += cs[i * LD + d];
-      cs[i * LD + d] = c;
-    }
+    for (int i = 0; i < SEG; ++i) x[i] = cs[i * LD + d];
+#pragma unroll
+    for (int i = 1; i < SEG; ++i) x[i] += x[i - 1];
+#pragma unroll
+    for (int i = 0; i < SEG; ++i) cs[i * LD + d] = x[i];
   }
   cp_async_wait_all();
   __syncthreads();
+  auto at = [&](const float* b, int i, int d) { return *reinterpret_cast<const float4*>(b + i * LD + d); };
+  auto put = [&](float* b, int i, int d, float4 v) { *reinterpret_cast<float4*>(b + i * LD + d) = v; };
+  auto times = [](float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); };
+  auto apart = [](float4 a, float4 b) { return make_float4(exp2f(a.x - b.x), exp2f(a.y - b.y), exp2f(a.z - b.z), exp2f(a.w - b.w)); };
+  auto dot = [](float4 a, float4 b, float s) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s)))); };
+  // the scaled rows; eight neighbouring threads walk a row
+  for (int i = tid >> 3; i < SEG; i += THREADS / 8)
+    for (int d = 4 * (tid & 7); d < DP; d += 32) {
+      const float4 c = at(cs, i, d), m = at(cs, HALF - 1, d);
+      if (i < HALF) {
+        put(km, i, d, times(at(ks, i, d), apart(m, c)));
+      } else {
+        const float4 g = apart(c, m);
+        put(km, i, d, times(at(ks, i, d), g));
+        put(qm, i - HALF, d, times(at(qs, i, d), g));
+      }
+    }
   {
-    // rows bi and 31 - bi with columns bj and 16 + bj, as far as the column is not behind the row
-    const int bi = tid >> 4, bj = tid & 15, i0 = bi, i1 = SEG - 1 - bi, j0 = bj, j1 = bj + 16;
-    const bool low = j0 <= i0, high = j1 <= i1;
-    float kk[3] = {}, qk[3] = {};          // (i1, j0), (i0, j0), (i1, j1)
-    auto pair = [](float4 k, float4 q, float4 c, float4 kj, float4 cj, float& sk, float& sq) {
-      float t;
-      t = kj.x * exp2f(c.x - cj.x); sk = fmaf(k.x, t, sk); sq = fmaf(q.x, t, sq);
-      t = kj.y * exp2f(c.y - cj.y); sk = fmaf(k.y, t, sk); sq = fmaf(q.y, t, sq);
-      t = kj.z * exp2f(c.z - cj.z); sk = fmaf(k.z, t, sk); sq = fmaf(q.z, t, sq);
-      t = kj.w * exp2f(c.w - cj.w); sk = fmaf(k.w, t, sk); sq = fmaf(q.w, t, sq);
-    };
-#pragma unroll 1
+    // inside the halves: the pair (bi, bj) of the first half where bj <= bi, else (bj, bi) of the second, a thread one pair;
+    // the second half's diagonal (scores only, no decay in them) by sixteen threads a row
+    const int bi = tid >> 4, bj = tid & 15;
+    const bool first = bj <= bi;
+    const int i = first ? bi : HALF + bj, j = first ? bj : HALF + bi;
+    float kk = 0.0f, qk = 0.0f, own = 0.0f;
+#pragma unroll 4
     for (int d = 0; d < DP; d += 4) {
-      auto at = [&](const float* b, int i) { return *reinterpret_cast<const float4*>(b + i * LD + d); };
-      const float4 k1 = at(ks, i1), q1 = at(qs, i1), c1 = at(cs, i1), kj = at(ks, j0), cj = at(cs, j0);
-      pair(k1, q1, c1, kj, cj, kk[0], qk[0]);
-      if (low) pair(at(ks, i0), at(qs, i0), at(cs, i0), kj, cj, kk[1], qk[1]);
-      if (high) pair(k1, q1, c1, at(ks, j1), at(cs, j1), kk[2], qk[2]);
+      const float4 t = times(at(ks, j, d), apart(at(cs, i, d), at(cs, j, d)));
+      kk = dot(at(ks, i, d), t, kk);
+      qk = dot(at(qs, i, d), t, qk);
     }
-    L[i1 * LLD + j0] = be[i1] * kk[0];     // i1 >= 16 > j0
-    A[j0 * LLD + i1] = qk[0];
-    if (low) {
-      if (j0 < i0) L[i0 * LLD + j0] = be[i0] * kk[1];
-      A[j0 * LLD + i0] = qk[1];
-    }
-    if (high) {
-      if (j1 < i1) L[i1 * LLD + j1] = be[i1] * kk[2];
-      A[j1 * LLD + i1] = qk[2];
-    }
+    for (int d = 4 * bj; d < DP; d += 64) own = dot(at(ks, HALF + bi, d), at(qs, HALF + bi, d), own);
+    for (int o = 8; o > 0; o >>= 1) own += __shfl_xor_sync(0xffffffffu, own, o);
+    if (j < i) L[i * LLD + j] = be[i] * kk;
+    A[j * LLD + i] = qk;
+    if (bj == 0) A[(HALF + bi) * LLD + HALF + bi] = own;
   }
   __syncthreads();
+  {
+    // the second half's rows with the first half's
+    const int bi = tid >> 4, bj = tid & 15, i = HALF + bi;
+    float kk = 0.0f, qk = 0.0f;
+#pragma unroll 4
+    for (int d = 0; d < DP; d += 4) {
+      const float4 kj = at(km, bj, d);
+      kk = dot(at(km, i, d), kj, kk);
+      qk = dot(at(qm, bi, d), kj, qk);
+    }
+    L[i * LLD + bj] = be[i] * kk;
+    A[bj * LLD + i] = qk;
+  }
+  __syncthreads();                         // km has been read: its place takes the keys times e^c
+  for (int i = tid >> 3; i < SEG; i += THREADS / 8)
+    for (int d = 4 * (tid & 7); d < DP; d += 32) {
+      const float4 c = at(cs, i, d), last = at(cs, n - 1, d), k = at(ks, i, d);
+      const float4 g = apart(c, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+      put(km, i, d, times(k, g));
+      if (i >= n) continue;
+      const float4 kr = times(k, apart(last, c)), qr = times(at(qs, i, d), g);
+      const size_t to = ((size_t)(row0 + i) * p.heads + h) * D + d;
+      if (p.vec) {
+        *reinterpret_cast<float4*>(p.k_rows + to) = kr;
+        *reinterpret_cast<float4*>(p.q_rows + to) = qr;
+      } else {
+        const float kv[4] = {kr.x, kr.y, kr.z, kr.w}, qv[4] = {qr.x, qr.y, qr.z, qr.w};
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          if (d + x < D) { p.k_rows[to + x] = kv[x]; p.q_rows[to + x] = qv[x]; }
+      }
+    }
+  for (int d = tid; d < D; d += THREADS) p.seg_decay[((size_t)seg * p.heads + h) * D + d] = exp2f(cs[(n - 1) * LD + d]);
   {
     float* dst = p.scores + ((size_t)seg * p.heads + h) * SEG * SEG;
     const int j = tid >> 3, i = 4 * (tid & 7);
     *reinterpret_cast<float4*>(dst + j * SEG + i) = *reinterpret_cast<const float4*>(A + j * LLD + i);
   }
+  __syncthreads();
   for (int c = tid; c < D + V; c += THREADS) {
     float x[SEG];
     if (c < D) {
-      // this channel's keys and queries with their decays, and what is left of the state at the segment's end
-      const float last = cs[(n - 1) * LD + c];
-      float* kr = p.k_rows + ((size_t)row0 * p.heads + h) * D + c;
-      float* qr = p.q_rows + ((size_t)row0 * p.heads + h) * D + c;
-      p.seg_decay[((size_t)seg * p.heads + h) * D + c] = exp2f(last);
 #pragma unroll
-      for (int i = 0; i < SEG; ++i) {
-        const float ci = cs[i * LD + c], k = ks[i * LD + c], g = exp2f(ci);
-        x[i] = be[i] * g * k;
-        if (i < n) {
-          kr[(size_t)i * p.heads * D] = exp2f(last - ci) * k;
-          qr[(size_t)i * p.heads * D] = g * qs[i * LD + c];
-        }
-      }
+      for (int i = 0; i < SEG; ++i) x[i] = be[i] * km[i * LD + c];
     } else {
       const float* v = p.qkv + (size_t)row0 * p.stride + p.v_col + h * V + (c - D);
 #pragma unroll
@@ -326,7 +372,7 @@ channel_delta_segments_kernel(GdArgs p) {
   }
 }
 
-size_t channel_segments_smem(int D) { return ((size_t)3 * SEG * row_ld(D) + 2 * SEG * LLD + SEG) * sizeof(float); }
+size_t channel_segments_smem(int D) { return ((size_t)(4 * SEG + SEG / 2) * row_ld(D) + 2 * SEG * LLD + SEG) * sizeof(float); }
 size_t segments_smem(int D) { return ((size_t)SEG * row_ld(D) + SEG * LLD + 3 * SEG) * sizeof(float); }
 }  // namespace
 

@@ -475,10 +475,11 @@ int pick_tile_n(int M, int n_out, int pairs) {
   return best;
 }
 
-template <bool SWIGLU, typename TOut>
+template <int MODE, typename TOut>
 int launch_gemm_pair(const void* A, long long lda, const void* W, const float* bias, void* out, long long ldo, int M, int n_out,
                      int K, int* error_flag, cudaStream_t stream) {
-  auto kern = gemm_umma_pair_kernel<SWIGLU ? 1 : 0, TOut>;
+  constexpr bool SWIGLU = MODE == 1;
+  auto kern = gemm_umma_pair_kernel<MODE, TOut>;
   static int sms = 0;
   if (!sms) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, P_SMEM);
@@ -601,22 +602,23 @@ int launch_gemm_skinny(const void* X, long long ldx, const void* W, float* out, 
 }
 }  // namespace
 
-// out[M, n_out] = A[M, K] * W^T (+ bias), W [n_out, K] contiguous; or, with swiglu != 0, W [2 * n_out, K] =
-// [gate; up] and out = silu(A gate^T) * (A up^T).  A rows lda elements apart; K and lda multiples of 8;
+// out[M, n_out] = A[M, K] * W^T (+ bias), W [n_out, K] contiguous; or, with act 1, W [2 * n_out, K] =
+// [gate; up] and out = silu(A gate^T) * (A up^T), or, with act 2, out = relu(A W^T)^2.  A rows lda elements apart; K and lda multiples of 8;
 // A and W 16-byte aligned.  out_dtype: float32 or bfloat16.  error_flag: a device word set if a bounded
 // wait inside the kernel runs out.
 IFX_API int ifx_gemm_umma(const void* A, long long lda, const void* W, const float* bias, void* out, long long ldo,
-                          int out_dtype, int M, int n_out, int K, int swiglu, int* error_flag, cudaStream_t stream) {
+                          int out_dtype, int M, int n_out, int K, int act, int* error_flag, cudaStream_t stream) {
   if (M <= 0 || n_out <= 0) return 0;
-  if (K <= 0 || (K & 7) || (lda & 7) || !error_flag) return IFX_ERR_UNSUPPORTED;
+  if (act < 0 || act > 2 || K <= 0 || (K & 7) || (lda & 7) || !error_flag) return IFX_ERR_UNSUPPORTED;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return IFX_ERR_ALIGNMENT;
-  if (swiglu && bias) return IFX_ERR_UNSUPPORTED;
+  if (act && bias) return IFX_ERR_UNSUPPORTED;
   if (out_dtype == IFX_BF16)
-    return swiglu ? launch_gemm_pair<true, bf16>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream)
-                  : launch_gemm_pair<false, bf16>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream);
-  if (out_dtype == IFX_F32)
-    return swiglu ? launch_gemm_pair<true, float>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream)
-                  : launch_gemm_pair<false, float>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream);
+    return act == 1 ? launch_gemm_pair<1, bf16>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream)
+         : act == 2 ? launch_gemm_pair<4, bf16>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream)
+                    : launch_gemm_pair<0, bf16>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream);
+  if (out_dtype == IFX_F32 && act < 2)
+    return act ? launch_gemm_pair<1, float>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream)
+               : launch_gemm_pair<0, float>(A, lda, W, bias, out, ldo, M, n_out, K, error_flag, stream);
   return IFX_ERR_UNSUPPORTED;
 }
 

@@ -66,7 +66,7 @@ template <int NT, bool SWIGLU, typename TOut, int RT, int KW>
 __global__ void __launch_bounds__(KW * 32)
 gemv_bf16_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, const float* __restrict__ bias,
                  TOut* __restrict__ out, int M, int n_out, int K, long long ldx, long long ldo,
-                 long long partial_stride, int n_groups) {
+                 long long partial_stride, int n_groups, int relu2) {
   constexpr int THREADS = KW * 32;
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint4 ring[];                 // [NST][2 * RT][threads]: a thread's slots are [..][..][tid]
@@ -208,8 +208,10 @@ gemv_bf16_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, const f
           if (o < n_out) dst[(size_t)token * ldo + o] = to_out<TOut>(lo / (1.0f + expf(-lo)) * hi);
         } else {
           const int ra = tile * 16 + g, rb2 = ra + 8;
-          if (ra < n_out) dst[(size_t)token * ldo + ra] = to_out<TOut>(lo + (add_bias ? bias[ra] : 0.0f));
-          if (rb2 < n_out) dst[(size_t)token * ldo + rb2] = to_out<TOut>(hi + (add_bias ? bias[rb2] : 0.0f));
+          float va = lo + (add_bias && ra < n_out ? bias[ra] : 0.0f), vb = hi + (add_bias && rb2 < n_out ? bias[rb2] : 0.0f);
+          if (relu2) { va = fmaxf(va, 0.0f); va *= va; vb = fmaxf(vb, 0.0f); vb *= vb; }
+          if (ra < n_out) dst[(size_t)token * ldo + ra] = to_out<TOut>(va);
+          if (rb2 < n_out) dst[(size_t)token * ldo + rb2] = to_out<TOut>(vb);
         }
       }
     }
@@ -247,7 +249,7 @@ inline int grid_width(int resident, int n_groups, int k_splits) {
 
 template <int NT, bool SWIGLU, typename TOut, int RT, int KW>
 int launch(const void* X, const void* W, const float* bias, void* out, int M, int n_out, int K, long long ldx,
-           long long ldo, int k_splits, long long partial_stride, cudaStream_t stream) {
+           long long ldo, int k_splits, long long partial_stride, int relu2, cudaStream_t stream) {
   const int tiles = SWIGLU ? (n_out + 7) / 8 : (n_out + 15) / 16;
   const int n_groups = (tiles + RT - 1) / RT;
   const size_t smem = (size_t)NST * 2 * RT * KW * 32 * sizeof(uint4);
@@ -255,7 +257,7 @@ int launch(const void* X, const void* W, const float* bias, void* out, int M, in
   if (resident < 0) return -resident;
   dim3 grid(grid_width(resident, n_groups, k_splits), k_splits);
   int ifx_rc = launch_pdl(gemv_bf16_kernel<NT, SWIGLU, TOut, RT, KW>, grid, dim3(KW * 32), smem, stream, (const bf16*)X,
-                          (const bf16*)W, bias, (TOut*)out, M, n_out, K, ldx, ldo, partial_stride, n_groups);
+                          (const bf16*)W, bias, (TOut*)out, M, n_out, K, ldx, ldo, partial_stride, n_groups, relu2);
   return ifx_rc ? ifx_rc : IFX_LAUNCH_CHECK();
 }
 
@@ -271,43 +273,46 @@ inline BlockShape block_shape(int tiles, int K, int k_splits) {
 
 template <int NT, bool SWIGLU, typename TOut>
 int by_shape(const void* X, const void* W, const float* bias, void* out, int M, int n_out, int K, long long ldx,
-             long long ldo, int k_splits, long long partial_stride, cudaStream_t stream) {
+             long long ldo, int k_splits, long long partial_stride, int relu2, cudaStream_t stream) {
   const BlockShape bs = block_shape(SWIGLU ? (n_out + 7) / 8 : (n_out + 15) / 16, K, k_splits);
-  if (bs.rt == 2) return launch<NT, SWIGLU, TOut, 2, 8>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, stream);
-  if (bs.kw == 8) return launch<NT, SWIGLU, TOut, 1, 8>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, stream);
-  return launch<NT, SWIGLU, TOut, 1, 4>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, stream);
+  if (bs.rt == 2) return launch<NT, SWIGLU, TOut, 2, 8>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, relu2, stream);
+  if (bs.kw == 8) return launch<NT, SWIGLU, TOut, 1, 8>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, relu2, stream);
+  return launch<NT, SWIGLU, TOut, 1, 4>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, relu2, stream);
 }
 
 template <bool SWIGLU, typename TOut>
 int by_tiles(const void* X, const void* W, const float* bias, void* out, int M, int n_out, int K, long long ldx,
-             long long ldo, int k_splits, long long partial_stride, cudaStream_t stream) {
-  if (M <= 8) return by_shape<1, SWIGLU, TOut>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, stream);
-  return by_shape<2, SWIGLU, TOut>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, stream);
+             long long ldo, int k_splits, long long partial_stride, int relu2, cudaStream_t stream) {
+  if (M <= 8) return by_shape<1, SWIGLU, TOut>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, relu2, stream);
+  return by_shape<2, SWIGLU, TOut>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, partial_stride, relu2, stream);
 }
 }  // namespace
 
-// out[M, n_out] = X[M, K] * W^T (+ bias), W [n_out, K]; or, with swiglu != 0, W [2 * n_out, K] = [gate; up]
-// and out = silu(X gate^T) * (X up^T).  M <= 16; K a multiple of 8; X rows and W 16-byte aligned.
-// k_splits > 1 (float32 output, no swiglu): out is [k_splits, M, n_out], slice s holding the sum over
+// out[M, n_out] = X[M, K] * W^T (+ bias), W [n_out, K]; or, with act 1, W [2 * n_out, K] = [gate; up]
+// and out = silu(X gate^T) * (X up^T), or, with act 2, out = relu(X W^T)^2.  M <= 16; K a multiple of 8; X rows and W 16-byte aligned.
+// k_splits > 1 (float32 output, no activation): out is [k_splits, M, n_out], slice s holding the sum over
 // the s-th part of K; the caller adds the slices (the fused residual-add + norm kernel does).
 // W is read before the kernel has waited for the kernel launched before it in the stream, so W must
 // not be the output of a kernel of this library launched directly before (weights are parameters).
 IFX_API int ifx_gemv_bf16(const void* X, const void* W, const float* bias, void* out, int out_dtype, int M,
-                          int n_out, int K, long long ldx, long long ldo, int swiglu, int k_splits,
+                          int n_out, int K, long long ldx, long long ldo, int act, int k_splits,
                           cudaStream_t stream) {
   if (M <= 0 || n_out <= 0) return 0;
+  if (act < 0 || act > 2) return IFX_ERR_UNSUPPORTED;
+  const bool swiglu = act == 1;
+  const int relu2 = act == 2;
   if (M > 16 || K <= 0 || (K & 7)) return IFX_ERR_UNSUPPORTED;
   if (((uintptr_t)X & 15) || ((uintptr_t)W & 15) || (ldx & 7)) return IFX_ERR_ALIGNMENT;
-  if (swiglu && bias) return IFX_ERR_UNSUPPORTED;
+  if (act && bias) return IFX_ERR_UNSUPPORTED;
   if (k_splits < 1 || k_splits > 64) return IFX_ERR_UNSUPPORTED;
-  if (k_splits > 1 && (swiglu || out_dtype != IFX_F32)) return IFX_ERR_UNSUPPORTED;
+  if (k_splits > 1 && (act || out_dtype != IFX_F32)) return IFX_ERR_UNSUPPORTED;
   const long long ps = (long long)M * ldo;
   if (out_dtype == IFX_BF16)
-    return swiglu ? by_tiles<true, bf16>(X, W, bias, out, M, n_out, K, ldx, ldo, 1, 0, stream)
-                  : by_tiles<false, bf16>(X, W, bias, out, M, n_out, K, ldx, ldo, 1, 0, stream);
+    return swiglu ? by_tiles<true, bf16>(X, W, bias, out, M, n_out, K, ldx, ldo, 1, 0, relu2, stream)
+                  : by_tiles<false, bf16>(X, W, bias, out, M, n_out, K, ldx, ldo, 1, 0, relu2, stream);
   if (out_dtype == IFX_F32)
-    return swiglu ? by_tiles<true, float>(X, W, bias, out, M, n_out, K, ldx, ldo, 1, 0, stream)
-                  : by_tiles<false, float>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, ps, stream);
+    return swiglu ? by_tiles<true, float>(X, W, bias, out, M, n_out, K, ldx, ldo, 1, 0, relu2, stream)
+                  : by_tiles<false, float>(X, W, bias, out, M, n_out, K, ldx, ldo, k_splits, ps, relu2, stream);
   return IFX_ERR_UNSUPPORTED;
 }
 

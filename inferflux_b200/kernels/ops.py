@@ -159,7 +159,7 @@ def _lib():
         lib.ifx_retention_finish.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_ll, c_int, c_int, c_int, c_float,
                                              c_void_p]
         lib.ifx_gelu_tanh.argtypes = [c_void_p, c_int, c_ll, c_void_p, c_int, c_ll, c_int, c_int, c_void_p]
-        lib.ifx_moe_route.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p]
+        lib.ifx_moe_route.argtypes = [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.ifx_moe_tile_rows.argtypes = [c_int]
         lib.ifx_moe_experts.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                         c_int, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
@@ -414,11 +414,11 @@ GEMV_MAX_ROWS = 16
 
 
 def gemv_bf16(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-              swiglu: bool = False, k_splits: int = 1) -> torch.Tensor:
+              swiglu: bool = False, k_splits: int = 1, relu2: bool = False) -> torch.Tensor:
     """out[M, N] = x[M, K] @ w[N, K]^T (+ bias) for M <= 16, bfloat16 operands,
     float32 accumulation, bfloat16 or float32 result.  With ``swiglu`` w is
-    [2N, K] = [gate; up] and out = silu(x gate^T) * (x up^T).  With
-    ``k_splits`` > 1 out is float32 [k_splits, M, N]: slice s is the sum over the
+    [2N, K] = [gate; up] and out = silu(x gate^T) * (x up^T); with ``relu2`` out =
+    relu(x w^T)^2.  With ``k_splits`` > 1 out is float32 [k_splits, M, N]: slice s is the sum over the
     s-th part of K and the caller adds the slices.  ``w`` is a parameter: the
     kernel starts to read it before the kernel launched before it has finished,
     so it must not be that kernel's output."""
@@ -429,27 +429,27 @@ def gemv_bf16(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ou
     _need(m <= GEMV_MAX_ROWS and k % 8 == 0, f"gemv_bf16: at most {GEMV_MAX_ROWS} rows and K a multiple of 8")
     if k_splits > 1:
         _need(tuple(out.shape) == (k_splits, m, n) and out.is_contiguous() and out.dtype == torch.float32
-              and not swiglu, "gemv_bf16: partial sums are float32 [k_splits, M, N]")
+              and not swiglu and not relu2, "gemv_bf16: partial sums are float32 [k_splits, M, N]")
         ldo = n
     else:
         _need(out.dim() == 2 and out.shape[0] == m and out.stride(1) == 1, "gemv_bf16: out [M, N]")
         ldo = out.stride(0) if m > 1 else n
     _need(x.stride(1) == 1, "gemv_bf16: unit inner strides")
     if bias is not None:
-        _need(bias.dtype == torch.float32 and bias.numel() == n and not swiglu, "gemv_bf16: bias float32 [N]")
+        _need(bias.dtype == torch.float32 and bias.numel() == n and not swiglu and not relu2, "gemv_bf16: bias float32 [N]")
     _check(_lib().ifx_gemv_bf16(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), _code(out), m, n, k,
-                                x.stride(0) if m > 1 else k, ldo, 1 if swiglu else 0, int(k_splits),
+                                x.stride(0) if m > 1 else k, ldo, 1 if swiglu else 2 if relu2 else 0, int(k_splits),
                                 _stream()), "gemv_bf16")
     return out
 
 
 def gemm_umma(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-              swiglu: bool = False) -> torch.Tensor:
+              swiglu: bool = False, relu2: bool = False) -> torch.Tensor:
     """out[M, N] = x[M, K] @ w[N, K]^T (+ bias) for many rows, on the tcgen05 tensor
     cores (TMA operands, accumulators in tensor memory), bfloat16 operands, float32
     accumulation, bfloat16 or float32 result.  With ``swiglu`` w is [2N, K] =
     [gate; up] and out = silu(x gate^T) * (x up^T), the activation applied in the
-    product's epilogue.  Two SMs share each tile (cta_group::2).  A bounded wait
+    product's epilogue; with ``relu2`` (bfloat16 out) out = relu(x w^T)^2 likewise.  Two SMs share each tile (cta_group::2).  A bounded wait
     that runs out sets the device's error flag (see :func:`check_device_errors`)."""
     m, k = x.shape
     n = out.shape[-1]
@@ -459,9 +459,9 @@ def gemm_umma(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ou
           "gemm_umma: out [M, N], unit inner strides")
     _need(k % 8 == 0 and (m == 1 or x.stride(0) % 8 == 0), "gemm_umma: K and the row stride of x must be multiples of 8")
     if bias is not None:
-        _need(bias.dtype == torch.float32 and bias.numel() == n and not swiglu, "gemm_umma: bias float32 [N]")
+        _need(bias.dtype == torch.float32 and bias.numel() == n and not swiglu and not relu2, "gemm_umma: bias float32 [N]")
     _check(_lib().ifx_gemm_umma(_ptr(x), x.stride(0) if m > 1 else k, _ptr(w), _ptr(bias), _ptr(out), out.stride(0),
-                                _code(out), m, n, k, 1 if swiglu else 0, _ptr(error_flag(x.device)), _stream()),
+                                _code(out), m, n, k, 1 if swiglu else 2 if relu2 else 0, _ptr(error_flag(x.device)), _stream()),
            "gemm_umma")
     return out
 
@@ -1486,13 +1486,13 @@ def moe_route(logits: torch.Tensor, top: int, over_all: bool = False, scale: flo
     with ``over_all``): the choice goes by the score plus the correction, the weights by the score alone.  Returns (int32
     ``[N, top]``, float32 ``[N, top]``)."""
     n, experts = logits.shape
-    _need(logits.dtype == torch.float32 and logits.is_contiguous(), "moe_route: float32 logits")
+    _need(logits.dtype == torch.float32 and logits.stride(1) == 1, "moe_route: float32 rows")
     _need(1 <= top <= min(64, experts), f"moe_route: top {top} must be within 1..min(64, experts)")
     _need(correction is None or (over_all and correction.dtype == torch.float32 and correction.is_contiguous()
                                  and correction.numel() == experts), "moe_route: correction float32 [E], with over_all")
     chosen = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
-    _check(_lib().ifx_moe_route(_ptr(logits), n, experts, top, int(bool(over_all)), float(scale), _ptr(correction), _ptr(chosen),
+    _check(_lib().ifx_moe_route(_ptr(logits), logits.stride(0), n, experts, top, int(bool(over_all)), float(scale), _ptr(correction), _ptr(chosen),
                                 _ptr(weights), _stream()), "moe_route")
     return chosen, weights
 

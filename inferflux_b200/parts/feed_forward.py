@@ -20,7 +20,7 @@ from ..config.registry import register_part
 from ..kernels import ops
 from ..weights.loader import MATRIX, VECTOR, WeightSpec
 from .base import Part, PartialSums
-from .linear import Linear
+from .linear import GEMV_ROWS, Linear
 
 
 FUSED_PRODUCT_ROWS = 128   # above this many rows gate/up + activation run as one tcgen05 product (measured: 256 rows 63 us
@@ -198,8 +198,9 @@ class ClampedGLU(Part):
 
 
 class SquaredReluMLP(Part):
-    """``down( relu(up(x))^2 )``, no biases.  The up projection leaves float32 sums; the activation rounds once into
-    the engine's type.  params: ``hidden``, ``intermediate``, ``name`` (tensors ``<prefix>.<name>.{up,down}``)."""
+    """``down( relu(up(x))^2 )``, no biases.  The activation is computed on the up projection's float32 sums and rounds
+    once into the engine's type; in bfloat16 it sits in the product's epilogue for few rows (the weight-streaming kernel)
+    and for many (the tcgen05 product).  params: ``hidden``, ``intermediate``, ``name`` (tensors ``<prefix>.<name>.{up,down}``)."""
 
     family = "feed_forward"
 
@@ -220,9 +221,16 @@ class SquaredReluMLP(Part):
         self.up, self.down = Linear(tensors.pop(n("up"))), Linear(tensors.pop(n("down")))
 
     def forward(self, x: torch.Tensor, ctx):
-        z = self.up.forward(x, out_dtype=torch.float32, allow_partials=True, f32_sums=True)
+        w = self.up.weight
         act = torch.empty((x.shape[0], self.intermediate), dtype=x.dtype, device=x.device)
-        ops.activation(z.tensor if isinstance(z, PartialSums) else z, act, ops.ACT_RELU2)
+        fused = w.dtype == torch.bfloat16 and x.dtype == torch.bfloat16 and self.hidden % 8 == 0
+        if fused and x.shape[0] <= GEMV_ROWS:
+            ops.gemv_bf16(x, w, None, act, relu2=True)
+        elif fused and x.is_contiguous() and x.shape[0] > FUSED_PRODUCT_ROWS:
+            ops.gemm_umma(x, w, None, act, relu2=True)
+        else:
+            z = self.up.forward(x, out_dtype=torch.float32, allow_partials=True, f32_sums=True)
+            ops.activation(z.tensor if isinstance(z, PartialSums) else z, act, ops.ACT_RELU2)
         return self.down.forward(act, out_dtype=torch.float32, allow_partials=True, f32_sums=True)
 
 
@@ -308,7 +316,11 @@ class RoutedExperts(Part):
         n = lambda leaf: self.full_name(self.prefix, self.params, leaf)
         # The router's products are 32-bit whatever the engine: a bfloat16 weight times a bfloat16 input is exact
         # in float32, and the sums are float32 (the library's product or the weight-streaming kernel).
-        self.router = Linear(tensors.pop(n("router")), tensors.pop(n("router.b")) if self.params.get("router_bias", True) else None)
+        # Rows of zeros fill the weight up to a multiple of 8 (the library's products are quick at such widths only).
+        def filled(t):
+            return t if t.shape[0] % 8 == 0 else torch.cat([t, t.new_zeros((-t.shape[0] % 8, *t.shape[1:]))])
+        self.router = Linear(filled(tensors.pop(n("router"))),
+                             filled(tensors.pop(n("router.b"))) if self.params.get("router_bias", True) else None)
         if self.params.get("correction"):
             self.correction = tensors.pop(n("correction")).to(torch.float32).contiguous()
         ups = ("up",) if self.activation == ops.MOE_RELU2 else ("gate", "up")
@@ -321,7 +333,7 @@ class RoutedExperts(Part):
             self.shared.load(tensors)
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
-        logits = self.router.forward(x, out_dtype=torch.float32)
+        logits = self.router.forward(x, out_dtype=torch.float32)[:, :self.outputs]
         chosen, weights = ops.moe_route(logits, self.top, self.over_all, self.scale, self.correction)
         xe = x
         if x.dtype != self.gate_up.dtype:
