@@ -56,27 +56,30 @@ template <> struct Vec<4> {
 
 // S: the number of copies, or 0 for any number up to MAX_STREAMS.  W: columns a thread takes at a time.
 template <int S, int W, typename TY, typename TO>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(512, 2)
 stream_mix_norm_kernel(StreamArgs p, const TY* __restrict__ y, TO* __restrict__ out) {
-  pdl_enter();
+  pdl_launch_dependents();
   extern __shared__ __align__(16) float u_buf[];            // [hidden]
   __shared__ float scratch[32];
   constexpr int SM = S ? S : MAX_STREAMS;
   const int ns = S ? S : p.streams, hidden = p.hidden;
+  // volatile, in shared memory: kept in registers these would halve the occupancy.  They are parameters, so they are
+  // read before the kernel ahead has finished.
+  __shared__ volatile float reads[SM], w_out[SM], mix[SM * SM];
+  for (int i = threadIdx.x; i < ns * ns; i += blockDim.x) {
+    if (i < ns) {
+      reads[i] = p.reads[i];
+      if (y) w_out[i] = p.w_out[i];
+    }
+    if (y) mix[i] = p.mix[i];
+  }
+  __syncthreads();
+  pdl_wait();
   const int src = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
   float* xr = p.x + (size_t)src * ns * hidden;
   const TY* yr = y ? y + (size_t)src * hidden : nullptr;
-  float reads[SM], w_out[SM], mix[S ? S * S : 1];
-#pragma unroll
-  for (int s = 0; s < SM; ++s) {
-    reads[s] = s < ns ? p.reads[s] : 0.0f;
-    w_out[s] = yr && s < ns ? p.w_out[s] : 0.0f;
-  }
-  if (S && yr) {
-#pragma unroll
-    for (int i = 0; i < S * S; ++i) mix[i] = p.mix[i];
-  }
   float ss = 0.0f;
+#pragma unroll 1
   for (int i = W * threadIdx.x; i < hidden; i += W * blockDim.x) {
     Vec<W> x[SM], u;
 #pragma unroll
@@ -91,7 +94,7 @@ stream_mix_norm_kernel(StreamArgs p, const TY* __restrict__ y, TO* __restrict__ 
 #pragma unroll
         for (int c = 0; c < W; ++c) d.v[c] += more.v[c];
       }
-#pragma unroll
+#pragma unroll (S ? S : 1)
       for (int t = 0; t < SM; ++t) {
         if (t >= ns) break;
         Vec<W> a;
@@ -100,7 +103,7 @@ stream_mix_norm_kernel(StreamArgs p, const TY* __restrict__ y, TO* __restrict__ 
 #pragma unroll
         for (int s = 0; s < SM; ++s) {
           if (s >= ns) break;
-          const float m = S ? mix[s * S + t] : p.mix[s * ns + t];
+          const float m = mix[s * ns + t];
 #pragma unroll
           for (int c = 0; c < W; ++c) a.v[c] = fmaf(m, x[s].v[c], a.v[c]);
         }
@@ -150,9 +153,10 @@ int launch_mix_out(const StreamArgs& p, const void* y, void* out, int out_dtype,
 }
 template <int S>
 int launch_mix_types(const StreamArgs& p, const void* y, int y_dtype, void* out, int out_dtype, int vec, int n_rows, cudaStream_t stream) {
+  constexpr int W = S ? 4 : 1;             // many copies leave no registers for four columns
   if (y_dtype == IFX_BF16)
-    return vec ? launch_mix_out<S, 4, bf16>(p, y, out, out_dtype, n_rows, stream) : launch_mix_out<S, 1, bf16>(p, y, out, out_dtype, n_rows, stream);
-  return vec ? launch_mix_out<S, 4, float>(p, y, out, out_dtype, n_rows, stream) : launch_mix_out<S, 1, float>(p, y, out, out_dtype, n_rows, stream);
+    return vec ? launch_mix_out<S, W, bf16>(p, y, out, out_dtype, n_rows, stream) : launch_mix_out<S, 1, bf16>(p, y, out, out_dtype, n_rows, stream);
+  return vec ? launch_mix_out<S, W, float>(p, y, out, out_dtype, n_rows, stream) : launch_mix_out<S, 1, float>(p, y, out, out_dtype, n_rows, stream);
 }
 
 struct BigramArgs {
@@ -217,7 +221,7 @@ IFX_API int ifx_stream_mix_norm(float* x, const void* y, int y_dtype, int parts,
     case 2: rc = launch_mix_types<2>(p, y, yd, out, out_dtype, vec, n_rows, stream); break;
     case 3: rc = launch_mix_types<3>(p, y, yd, out, out_dtype, vec, n_rows, stream); break;
     case 4: rc = launch_mix_types<4>(p, y, yd, out, out_dtype, vec, n_rows, stream); break;
-    default: rc = launch_mix_types<0>(p, y, yd, out, out_dtype, 0, n_rows, stream); break;
+    default: rc = launch_mix_types<0>(p, y, yd, out, out_dtype, vec, n_rows, stream); break;
   }
   return rc ? rc : IFX_LAUNCH_CHECK();
 }
