@@ -270,7 +270,7 @@ def kibilix_config(size: str, layers: int):
         heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=8192),
         rot=dict(dims=128, base=500000.0, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))))
     delta = dict(type="channel_delta", mixer=dict(heads=heads // 2, kv_heads=heads // 4, dim=128, vdim=128, conv=4))
-    return dict(architecture="Kibilix", width=hidden, vocab=vocab, norm=dict(eps=1e-6), streams=4, residual_mult=0.7,
+    return dict(architecture="Kibilix", width=hidden, vocab=vocab, norm=dict(eps=1e-6), streams=4, residual_mult=0.8,
                 embedding=dict(bigram=dict(buckets=vocab // 2 + 1, mul_prev=31, mul_cur=17)),
                 layers=[dict(delta if i % 2 else attn, mlp=moe if i % 4 >= 2 else dense) for i in range(layers)])
 

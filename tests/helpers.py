@@ -595,7 +595,7 @@ KB_C = dict(architecture="Kibilix", width=128, vocab=200, norm=dict(eps=1e-6), s
     _kb_delta(2, 64, 5, mlp=_kb_moe(64, 1.5, 4, 2, identity=1)),
     _kb_attn(4, 64, kv_heads=2, scale=0.125, chunk=70, softcap=8.0, rot=dict(dims=64, base=200000.0), mlp=dict(kind="dense", ff=160)),
     _kb_attn(2, 64, scale=0.1, chunk=48, softcap=15.0,
-             rot=dict(dims=16, base=1e4, scaling=dict(factor=8.0, low=1.0, high=4.0, original=128)), mlp=_kb_moe(96, 0.8, 6, 3, identity=3)),
+             rot=dict(dims=16, base=1e4, scaling=dict(factor=6.0, low=1.0, high=3.0, original=128)), mlp=_kb_moe(96, 0.8, 6, 3, identity=3)),
     _kb_delta(4, 32, 4, kv_heads=2, vdim=48, mlp=None)], loop=dict(start=2, stop=4, times=2))
 KB = {"A": KB_A, "B": KB_B, "C": KB_C}
 

@@ -250,7 +250,7 @@ def test_streams_mixed_and_read_by_the_norm(dtype, hidden, streams):
     from inferflux_b200.parts.base import PartialSums
     from inferflux_b200.parts.junction import StreamJoin
     from inferflux_b200.parts.norm import StreamRMSNorm
-    eps, tol, factor = 3e-6, (2e-6 if dtype == torch.float32 else 5e-3), 0.7
+    eps, tol, factor = 3e-6, (2e-6 if dtype == torch.float32 else 5e-3), 0.6
     part = StreamRMSNorm(dict(weight_name="norm1", reads="hc1.in", hidden=hidden, streams=streams, eps=eps), "l0", dtype, DEV)
     last = StreamRMSNorm(dict(weight_name="norm1", reads=None, hidden=hidden, streams=streams, eps=eps), "l0", dtype, DEV)
     join = StreamJoin(dict(name="hc1", streams=streams, factor=factor), "l0", dtype, DEV)
